@@ -31,6 +31,13 @@ int hb_add_rmsnorm(void* out, int out_dtype, void* h, int h_dtype, const void* d
                    int weight_dtype, float eps, float offset, const int32_t* index, int rows, int dim,
                    hb_stream stream);
 
+// The same with a layer norm, out = (v - mean v) / sqrt(mean((v - mean v)^2) + eps) * weight, and a factor on what is added
+// (csrc/layernorm.cu): v = h[row] + scale * delta[row], or with `place` (int32 [tokens, top]) v = h[row] + scale * sum_k
+// delta[place[row, k]]: the rows that `top` experts left for a token (negative places are skipped).
+int hb_add_layernorm(void* out, int out_dtype, void* h, int h_dtype, const void* delta, float scale, const int32_t* place,
+                     int top, const void* weight, int weight_dtype, float eps, const int32_t* index, int rows, int dim,
+                     hb_stream stream);
+
 // out[t, i] = silu(gate_up[t, i]) * gate_up[t, inter + i], in 32-bit, rounded once.
 int hb_silu_mul(void* out, const void* gate_up, int dtype, int tokens, int inter, hb_stream stream);
 
@@ -135,15 +142,19 @@ int hb_hyper_mix_norm(void* out, int out_dtype, float* xs, const float* src, con
 // qa[:, :, rank:] (the first rot_dims entries turn, half-split pairs, angles from table [max_positions, rot_dims],
 // cosines then sines) and, with dkv_at >= 0, [RMSNorm(latent) · norm_weight | rotated key part] into cache row
 // write_index[t] (negative or out of range: skipped).
+// `neighbours`: pairs (2i, 2i + 1) turn instead of (i, i + rot_dims / 2). qa null: no queries here. cq [tokens, q_rank]
+// (null: none) receives RMSNorm(columns cq_at .. of `first`) · cq_weight, the latent that queries are then made from (with
+// the latent's eps; cq_weight of norm_weight's dtype).
 int hb_latent_prepare(void* qa, const void* first, int dtype, int ld, int tokens, int heads, int dim, int rot, int rank,
-                      int dkv_at, const int32_t* positions, const float* table, int rot_dims, int max_positions,
-                      const void* norm_weight, int weight_dtype, float eps, void* cache, const int32_t* write_index,
+                      int dkv_at, void* cq, int cq_at, int q_rank, const void* cq_weight, const int32_t* positions,
+                      const float* table, int rot_dims, int max_positions, int neighbours, const void* norm_weight, int weight_dtype, float eps, void* cache, const int32_t* write_index,
                       int pages, int page_size, hb_stream stream);
-// out [tokens, heads, rank] = softmax_j(scale · qa · row_j) · latent_j over the keys a query sees (as hb_attention_generic).
+// out [tokens, heads, rank] = softmax_j(scale · qa · row_j) · latent_j over the keys a query sees (as hb_attention_generic);
+// sinks (float [heads] or null): exp(sinks[h]) stands in the softmax's denominator besides.
 int hb_latent_attention_generic(void* out, const void* qa, const void* cache, int dtype, const int32_t* block_table,
                                 int table_stride, const int32_t* row_slot, const int32_t* query_start,
                                 const int32_t* kv_len, int rows, int tokens, int heads, int rank, int rot, int pages,
-                                int page_size, float scale, int window, hb_stream stream);
+                                int page_size, float scale, int window, const float* sinks, hb_stream stream);
 
 // The same on tensor cores in bfloat16 (csrc/latent_bf16.cu) for rows row0 .. row1 - 1 of the batch, which bring `tokens`
 // tokens in all, the first of them token `first_token` of the step; rank and rot multiples of 16, rank up to 512.
@@ -153,7 +164,7 @@ size_t hb_latent_attention_scratch_floats(int tokens, int heads, int rank, int s
 int hb_latent_attention_bf16(void* out, float* scratch, const void* qa, const void* cache, const int32_t* block_table,
                              int table_stride, const int32_t* row_slot, const int32_t* query_start, const int32_t* kv_len,
                              int row0, int row1, int first_token, int tokens, int heads, int rank, int rot, int pages,
-                             int page_size, float scale, int window, int splits, hb_stream stream);
+                             int page_size, float scale, int window, int splits, const float* sinks, hb_stream stream);
 
 // Routed experts (csrc/experts.cu). z [tokens, ld]: 32-bit router logits in columns 0 .. experts - 1. chosen / weight
 // [tokens, top]: the experts with the largest softmax scores (equal ones by ascending expert) and score · scale
@@ -167,16 +178,19 @@ int hb_latent_attention_bf16(void* out, float* scratch, const void* qa, const vo
 // The choice may run on other numbers than the weights: `correction` (float [experts] or null) is added to the softmax
 // scores for the choice alone; with `groups` > 1 the experts form that many equal groups of neighbours, a group counts by
 // its best choice score and only experts of the `keep` best groups can be chosen; `tiny` is added to the chosen scores'
-// sum before `renormalize` divides by it.
+// sum before `renormalize` divides by it. `sigmoid`: a score is its own logit's sigmoid instead of a share of the softmax.
+// row_weight (float [tokens top] or null): the weight of each row's pair, for products that scale their rows.
+// hb_expert_combine with weight null: every weight is 1.
 int hb_route_top(int32_t* chosen, float* weight, int32_t* counts, const float* z, const float* bias, int ld, int tokens, int experts,
-                 int top, float scale, int renormalize, const float* correction, int groups, int keep, float tiny, hb_stream stream);
+                 int top, float scale, int renormalize, const float* correction, int groups, int keep, float tiny, int sigmoid,
+                 hb_stream stream);
 int hb_expert_rows(int32_t* place, int32_t* token_of, int32_t* counts, const int32_t* chosen, int tokens, int top,
-                   int experts, hb_stream stream);
+                   int experts, const float* weight, float* row_weight, hb_stream stream);
 // hb_route_top and hb_expert_rows as one call (one launch for up to 256 tokens and 1,024 experts). counts [2 experts + 3]
 // need not be zeroed; afterwards counts[2 experts + 1 ..] = (0, tokens): the `starts` of one expert that takes every token.
 int hb_route_rows(int32_t* chosen, float* weight, int32_t* counts, int32_t* place, int32_t* token_of, const float* z,
                   const float* bias, int ld, int tokens, int experts, int top, float scale, int renormalize,
-                  const float* correction, int groups, int keep, float tiny, hb_stream stream);
+                  const float* correction, int groups, int keep, float tiny, int sigmoid, float* row_weight, hb_stream stream);
 int hb_expert_linear(void* out, const void* x, int dtype, const int32_t* token_of, const void* w, const int32_t* starts,
                      int rows, int experts, int n, int k, int act, hb_stream stream);
 int hb_expert_combine(void* out, const void* y, int dtype, const int32_t* place, const float* weight, const void* shared,
@@ -356,8 +370,11 @@ int hb_sum_norm(float* h, const void* x0, const void* x1, const void* x2, const 
                 float offset, int tokens, int hidden, hb_stream stream);
 // out [tokens, inter] = g sigmoid(alpha g) (u + 1), g = min(gate + b, limit), u = clamp(up + b, -limit, limit), from
 // gate_up [tokens, 2 inter] (gate first) and bias [2 inter] (or null).
-int hb_glu_clamped(void* out, const void* gate_up, const void* bias, int dtype, float limit, float alpha, int tokens,
-                   int inter, hb_stream stream);
+// row_scale (float [tokens] or null): a factor on each row of gate_up, before the bias.
+int hb_glu_clamped(void* out, const void* gate_up, const void* bias, const float* row_scale, int dtype, float limit, float alpha,
+                   int tokens, int inter, hb_stream stream);
+// x = cap tanh(x / cap) in place.
+int hb_softcap(float* x, long count, float cap, hb_stream stream);
 
 // ---- mixers with a matrix state per head (csrc/recurrent.cu). Rows as for attention: row b brings tokens
 // query_start[b] .. query_start[b + 1] and lives in slot row_slot[b].
@@ -392,7 +409,7 @@ int hb_conv_carry(void* conv_state, const void* first, int dtype, int ld, int ch
 // position (as hb_qk_norm_rope_kv_write turns them), k times k_scale, all to 32-bit.
 int hb_retention_prepare(float* qk, float* v, const void* first, int dtype, int ld, const int32_t* positions,
                          const float* table, int rot_dims, int max_positions, int tokens, int heads, int dim, int vdim,
-                         float k_scale, hb_stream stream);
+                         float k_scale, int silu, hb_stream stream);
 // out [tokens, heads, vdim] (`dtype`) = o / sqrt(mean(o^2) + eps) * weight (float [vdim], with `weight_heads` [heads
 // vdim], or null) * gate, the gate a 32-bit multiplier gate_mul [tokens, heads vdim], or silu (`gate_sigmoid`: sigmoid)
 // of gate_pre (rows `ld` apart, `dtype`), or none.

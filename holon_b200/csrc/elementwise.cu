@@ -72,24 +72,6 @@ extern "C" int hb_embed(float* out, const void* table, int table_dtype, const in
 // ---------------------------------------------------------------- (add +) RMSNorm
 // One block per output row. The row is kept in shared memory as 32-bit between the two passes.
 // VEC: dim is a multiple of 4 and every pointer is 16-byte aligned per row, so a thread moves 4 values at a time.
-template <typename T> struct Vec4;
-template <> struct Vec4<float> {
-    static __device__ __forceinline__ void load(const float* p, float (&v)[4]) { const float4 x = *(const float4*)p; v[0] = x.x; v[1] = x.y; v[2] = x.z; v[3] = x.w; }
-    static __device__ __forceinline__ void store(float* p, const float (&v)[4]) { *(float4*)p = make_float4(v[0], v[1], v[2], v[3]); }
-};
-template <> struct Vec4<bf16> {
-    static __device__ __forceinline__ void load(const bf16* p, float (&v)[4]) {
-        const uint2 x = *(const uint2*)p;
-        const float2 a = __bfloat1622float2(*(const __nv_bfloat162*)&x.x), b = __bfloat1622float2(*(const __nv_bfloat162*)&x.y);
-        v[0] = a.x; v[1] = a.y; v[2] = b.x; v[3] = b.y;
-    }
-    static __device__ __forceinline__ void store(bf16* p, const float (&v)[4]) {
-        __nv_bfloat162 a = __floats2bfloat162_rn(v[0], v[1]), b = __floats2bfloat162_rn(v[2], v[3]);
-        uint2 x; x.x = *(uint32_t*)&a; x.y = *(uint32_t*)&b;
-        *(uint2*)p = x;
-    }
-};
-
 template <typename TH, typename TD, typename TW, bool VEC>
 __global__ void add_rmsnorm_kernel(TD* __restrict__ out, TH* h, const TD* __restrict__ delta,
                                    const TW* __restrict__ weight, float eps, float offset,
@@ -381,15 +363,17 @@ extern "C" int hb_sum_into(float* h, const void* x0, const void* x1, const void*
 }
 
 // ---------------------------------------------------------------- a gated unit with clamped inputs
-// gate_up [tokens, 2 inter] (gate columns first), bias [2 inter] or null: g = min(gate + b, limit),
-// u = clamp(up + b, -limit, limit), out = g sigmoid(alpha g) (u + 1), in 32-bit with one rounding.
+// gate_up [tokens, 2 inter] (gate columns first), bias [2 inter] or null, row_scale [tokens] or null (a factor on the row
+// of gate_up, before the bias): g = min(gate + b, limit), u = clamp(up + b, -limit, limit), out = g sigmoid(alpha g) (u + 1),
+// in 32-bit with one rounding. grid (rows, column segments).
 template <typename T>
 __global__ void glu_clamped_kernel(T* __restrict__ out, const T* __restrict__ gate_up, const T* __restrict__ bias,
-                                   float limit, float alpha, int inter) {
-    const size_t t = blockIdx.y;
-    const int i = blockIdx.x * blockDim.x + threadIdx.x;
+                                   const float* __restrict__ row_scale, float limit, float alpha, int inter) {
+    const size_t t = blockIdx.x;
+    const int i = blockIdx.y * blockDim.x + threadIdx.x;
     if (i >= inter) return;
-    float g = to_f32(gate_up[t * 2 * inter + i]), u = to_f32(gate_up[t * 2 * inter + inter + i]);
+    const float f = row_scale ? row_scale[t] : 1.f;
+    float g = f * to_f32(gate_up[t * 2 * inter + i]), u = f * to_f32(gate_up[t * 2 * inter + inter + i]);
     if (bias) { g += to_f32(bias[i]); u += to_f32(bias[inter + i]); }
     g = fminf(g, limit);
     u = fminf(fmaxf(u, -limit), limit);
@@ -399,13 +383,16 @@ __global__ void glu_clamped_kernel(T* __restrict__ out, const T* __restrict__ ga
 // The same, four neighbouring values a thread (inter a multiple of 4, pointers on 16-byte boundaries).
 template <typename T>
 __global__ void glu_clamped4_kernel(T* __restrict__ out, const T* __restrict__ gate_up, const T* __restrict__ bias,
-                                    float limit, float alpha, int inter) {
-    const size_t t = blockIdx.y;
-    const int i = (blockIdx.x * blockDim.x + threadIdx.x) * 4;
+                                    const float* __restrict__ row_scale, float limit, float alpha, int inter) {
+    const size_t t = blockIdx.x;
+    const int i = (blockIdx.y * blockDim.x + threadIdx.x) * 4;
     if (i >= inter) return;
+    const float f = row_scale ? row_scale[t] : 1.f;
     float g[4], u[4], b[4], y[4];
     Vec4<T>::load(gate_up + t * 2 * inter + i, g);
     Vec4<T>::load(gate_up + t * 2 * inter + inter + i, u);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) { g[e] *= f; u[e] *= f; }
     if (bias) {
         Vec4<T>::load(bias + i, b);
 #pragma unroll
@@ -422,21 +409,21 @@ __global__ void glu_clamped4_kernel(T* __restrict__ out, const T* __restrict__ g
     Vec4<T>::store(out + t * inter + i, y);
 }
 
-extern "C" int hb_glu_clamped(void* out, const void* gate_up, const void* bias, int dtype, float limit, float alpha,
-                              int tokens, int inter, hb_stream stream) {
+extern "C" int hb_glu_clamped(void* out, const void* gate_up, const void* bias, const float* row_scale, int dtype, float limit,
+                              float alpha, int tokens, int inter, hb_stream stream) {
     if (tokens == 0 || inter == 0) return 0;
-    if (tokens > 65535) HB_REFUSE("glu_clamped: %d rows are above 65535", tokens);
+    if (inter > 65535 * 256) HB_REFUSE("glu_clamped: rows of %d columns", inter);
     cudaStream_t s = (cudaStream_t)stream;
     if (inter % 4 == 0 && aligned16(out) && aligned16(gate_up) && aligned16(bias) && (dtype == HB_F32 || dtype == HB_BF16)) {
-        dim3 grid4((inter / 4 + 255) / 256, tokens);
-        if (dtype == HB_F32) glu_clamped4_kernel<float><<<grid4, 256, 0, s>>>((float*)out, (const float*)gate_up, (const float*)bias, limit, alpha, inter);
-        else glu_clamped4_kernel<bf16><<<grid4, 256, 0, s>>>((bf16*)out, (const bf16*)gate_up, (const bf16*)bias, limit, alpha, inter);
+        dim3 grid4(tokens, (inter / 4 + 255) / 256);
+        if (dtype == HB_F32) glu_clamped4_kernel<float><<<grid4, 256, 0, s>>>((float*)out, (const float*)gate_up, (const float*)bias, row_scale, limit, alpha, inter);
+        else glu_clamped4_kernel<bf16><<<grid4, 256, 0, s>>>((bf16*)out, (const bf16*)gate_up, (const bf16*)bias, row_scale, limit, alpha, inter);
         HB_LAUNCH_CHECK("glu_clamped");
         return 0;
     }
-    dim3 grid((inter + 255) / 256, tokens);
-    if (dtype == HB_F32) glu_clamped_kernel<float><<<grid, 256, 0, s>>>((float*)out, (const float*)gate_up, (const float*)bias, limit, alpha, inter);
-    else if (dtype == HB_BF16) glu_clamped_kernel<bf16><<<grid, 256, 0, s>>>((bf16*)out, (const bf16*)gate_up, (const bf16*)bias, limit, alpha, inter);
+    dim3 grid(tokens, (inter + 255) / 256);
+    if (dtype == HB_F32) glu_clamped_kernel<float><<<grid, 256, 0, s>>>((float*)out, (const float*)gate_up, (const float*)bias, row_scale, limit, alpha, inter);
+    else if (dtype == HB_BF16) glu_clamped_kernel<bf16><<<grid, 256, 0, s>>>((bf16*)out, (const bf16*)gate_up, (const bf16*)bias, row_scale, limit, alpha, inter);
     else HB_REFUSE("glu_clamped: dtype %d", dtype);
     HB_LAUNCH_CHECK("glu_clamped");
     return 0;
@@ -606,5 +593,29 @@ extern "C" int hb_out_norm_add(float* dst, const float* src, const void* y, int 
             weight_dtype == HB_F32, eps, offset, hist, hist_stride, n_hist, coef, avg, cast, cast_dtype, dim);
     } else HB_REFUSE("out_norm_add: dtype %d", y_dtype);
     HB_LAUNCH_CHECK("out_norm_add");
+    return 0;
+}
+
+// ---------------------------------------------------------------- a soft limit on logits
+// x = cap tanh(x / cap) in place, 32-bit.
+__global__ void softcap_kernel(float* __restrict__ x, long count, float cap) {
+    const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i < count) x[i] = cap * tanhf(x[i] / cap);
+}
+__global__ void softcap4_kernel(float4* __restrict__ x, long quads, float cap) {
+    const long i = (long)blockIdx.x * blockDim.x + threadIdx.x;
+    if (i >= quads) return;
+    float4 v = x[i];
+    v.x = cap * tanhf(v.x / cap); v.y = cap * tanhf(v.y / cap); v.z = cap * tanhf(v.z / cap); v.w = cap * tanhf(v.w / cap);
+    x[i] = v;
+}
+
+extern "C" int hb_softcap(float* x, long count, float cap, hb_stream stream) {
+    if (count == 0) return 0;
+    if (!(cap > 0.f)) HB_REFUSE("softcap: the cap must be positive");
+    cudaStream_t s = (cudaStream_t)stream;
+    if (count % 4 == 0 && aligned16(x)) softcap4_kernel<<<(unsigned)((count / 4 + 255) / 256), 256, 0, s>>>((float4*)x, count / 4, cap);
+    else softcap_kernel<<<(unsigned)((count + 255) / 256), 256, 0, s>>>(x, count, cap);
+    HB_LAUNCH_CHECK("softcap");
     return 0;
 }

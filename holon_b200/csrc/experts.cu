@@ -9,12 +9,16 @@
 // hb_expert_combine  out[t] = sum_k weight[t, k] · y[place[t, k]] (+ sigmoid(gate_t) · shared[t]); rows of identity experts read x[t]
 #include "common.cuh"
 
+// A logit's score up to the factor that all experts share: exp(z - max) (the factor is one over their sum) or sigmoid(z) (one).
+__device__ __forceinline__ float route_score(float z, float m, int sigmoid) { return sigmoid ? 1.f / (1.f + expf(-z)) : expf(z - m); }
+
 // ---------------------------------------------------------------- the router's choice
-// One block per token. softmax over all experts in 32-bit; the `top` largest scores, equal scores by ascending
-// expert; weight = score · scale, with `renormalize` divided by the chosen scores' sum first.
+// One block per token. The scores, in 32-bit, are the softmax over all experts or, with `sigmoid`, each logit's own
+// sigmoid; the `top` largest scores, equal scores by ascending expert; weight = score · scale, with `renormalize` divided
+// by the chosen scores' sum first.
 __global__ void route_top_kernel(int32_t* __restrict__ chosen, float* __restrict__ weight, int32_t* __restrict__ counts,
                                  const float* __restrict__ z, int ld, int experts, int top, float scale, int renormalize,
-                                 const float* __restrict__ bias) {
+                                 const float* __restrict__ bias, int sigmoid) {
     extern __shared__ float sc[];                       // experts scores
     __shared__ float scratch[33];
     __shared__ float best_v[32];
@@ -25,9 +29,9 @@ __global__ void route_top_kernel(int32_t* __restrict__ chosen, float* __restrict
     for (int e = threadIdx.x; e < experts; e += blockDim.x) m = fmaxf(m, zr[e] + (bias ? bias[e] : 0.f));
     m = block_max(m, scratch);
     float sum = 0.f;
-    for (int e = threadIdx.x; e < experts; e += blockDim.x) { const float p = expf(zr[e] + (bias ? bias[e] : 0.f) - m); sc[e] = p; sum += p; }
+    for (int e = threadIdx.x; e < experts; e += blockDim.x) { const float p = route_score(zr[e] + (bias ? bias[e] : 0.f), m, sigmoid); sc[e] = p; sum += p; }
     sum = block_sum(sum, scratch);
-    const float inv = 1.f / sum;
+    const float inv = sigmoid ? 1.f : 1.f / sum;
     float taken = 0.f;
     for (int k = 0; k < top; ++k) {
         float bv = -1.f; int bi = 0x7fffffff;
@@ -129,7 +133,7 @@ __global__ void __launch_bounds__(256) route_choice_kernel(int32_t* __restrict__
                                                            int32_t* __restrict__ counts, const float* __restrict__ z, int ld,
                                                            int tokens, int experts, int top, float scale, int renormalize,
                                                            const float* __restrict__ bias, const float* __restrict__ correction,
-                                                           int groups, int keep, float tiny) {
+                                                           int groups, int keep, float tiny, int sigmoid) {
     extern __shared__ float rc_smem[];
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
     const int t = blockIdx.x * 8 + warp;
@@ -142,16 +146,16 @@ __global__ void __launch_bounds__(256) route_choice_kernel(int32_t* __restrict__
     for (int e = lane; e < experts; e += 32) m = fmaxf(m, zr[e] + (bias ? bias[e] : 0.f));
     m = warp_max(m);
     float sum = 0.f;
-    for (int e = lane; e < experts; e += 32) { const float p = expf(zr[e] + (bias ? bias[e] : 0.f) - m); my[e] = p; sum += p; }
+    for (int e = lane; e < experts; e += 32) { const float p = route_score(zr[e] + (bias ? bias[e] : 0.f), m, sigmoid); my[e] = p; sum += p; }
     sum = warp_sum(sum);
     __syncwarp();
-    route_choice_warp(lane, my, ch, gm, 1.f / sum, correction, experts, top, groups, keep, chosen + (size_t)t * top,
+    route_choice_warp(lane, my, ch, gm, sigmoid ? 1.f : 1.f / sum, correction, experts, top, groups, keep, chosen + (size_t)t * top,
                       weight + (size_t)t * top, counts, scale, renormalize, tiny);
 }
 
 extern "C" int hb_route_top(int32_t* chosen, float* weight, int32_t* counts, const float* z, const float* bias, int ld,
                             int tokens, int experts, int top, float scale, int renormalize, const float* correction,
-                            int groups, int keep, float tiny, hb_stream stream) {
+                            int groups, int keep, float tiny, int sigmoid, hb_stream stream) {
     if (tokens == 0) return 0;
     if (experts < 1 || top < 1 || top > experts || ld < experts) HB_REFUSE("route_top: top %d of %d experts in rows of %d", top, experts, ld);
     if (experts > 8192) HB_REFUSE("route_top: %d experts are above 8192", experts);
@@ -162,13 +166,13 @@ extern "C" int hb_route_top(int32_t* chosen, float* weight, int32_t* counts, con
         if (smem > 200 * 1024) HB_REFUSE("route_top: a choice in groups takes up to 2133 experts, not %d", experts);
         if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(route_choice_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         route_choice_kernel<<<(tokens + 7) / 8, 256, smem, (cudaStream_t)stream>>>(chosen, weight, counts, z, ld, tokens, experts, top,
-                                                                                  scale, renormalize, bias, correction, groups, keep, tiny);
+                                                                                  scale, renormalize, bias, correction, groups, keep, tiny, sigmoid);
         HB_LAUNCH_CHECK("route_choice");
         return 0;
     }
     const int threads = experts > 256 ? 256 : experts > 64 ? 128 : 64;
     route_top_kernel<<<tokens, threads, (size_t)experts * sizeof(float), (cudaStream_t)stream>>>(
-        chosen, weight, counts, z, ld, experts, top, scale, renormalize, bias);
+        chosen, weight, counts, z, ld, experts, top, scale, renormalize, bias, sigmoid);
     HB_LAUNCH_CHECK("route_top");
     return 0;
 }
@@ -207,7 +211,8 @@ __global__ void expert_starts_kernel(int32_t* counts, int experts) {
 }
 
 __global__ void expert_scatter_kernel(int32_t* __restrict__ place, int32_t* __restrict__ token_of, int32_t* counts,
-                                      const int32_t* __restrict__ chosen, int pairs, int top, int experts) {
+                                      const int32_t* __restrict__ chosen, int pairs, int top, int experts,
+                                      const float* __restrict__ weight, float* __restrict__ row_weight) {
     const int i = blockIdx.x * blockDim.x + threadIdx.x;
     if (i >= pairs) return;
     const int e = chosen[i];
@@ -215,16 +220,17 @@ __global__ void expert_scatter_kernel(int32_t* __restrict__ place, int32_t* __re
     const int p = counts[experts + e] + atomicAdd(counts + e, 1);
     place[i] = p;
     token_of[p] = i / top;
+    if (row_weight) row_weight[p] = weight[i];
 }
 
 extern "C" int hb_expert_rows(int32_t* place, int32_t* token_of, int32_t* counts, const int32_t* chosen, int tokens,
-                              int top, int experts, hb_stream stream) {
+                              int top, int experts, const float* weight, float* row_weight, hb_stream stream) {
     if (tokens == 0) return 0;
     cudaStream_t s = (cudaStream_t)stream;
     expert_starts_kernel<<<1, 256, 0, s>>>(counts, experts);
     HB_LAUNCH_CHECK("expert_starts");
     const int pairs = tokens * top;
-    expert_scatter_kernel<<<(pairs + 255) / 256, 256, 0, s>>>(place, token_of, counts, chosen, pairs, top, experts);
+    expert_scatter_kernel<<<(pairs + 255) / 256, 256, 0, s>>>(place, token_of, counts, chosen, pairs, top, experts, weight, row_weight);
     HB_LAUNCH_CHECK("expert_scatter");
     return 0;
 }
@@ -242,7 +248,8 @@ __global__ void __launch_bounds__(256) route_rows_small_kernel(int32_t* __restri
                                                                int ld, int tokens, int experts, int top, float scale,
                                                                int renormalize, const float* __restrict__ bias,
                                                                const float* __restrict__ correction, int groups, int keep,
-                                                               float tiny, int grouped) {
+                                                               float tiny, int grouped, int sigmoid,
+                                                               float* __restrict__ row_weight) {
     extern __shared__ float rs_smem[];
     float* sc = rs_smem;                                   // [8][experts]
     int* cnt = (int*)(sc + 8 * (size_t)experts);           // [experts]: counts, then cursors
@@ -257,10 +264,10 @@ __global__ void __launch_bounds__(256) route_rows_small_kernel(int32_t* __restri
         for (int e = lane; e < experts; e += 32) m = fmaxf(m, zr[e] + (bias ? bias[e] : 0.f));
         m = warp_max(m);
         float sum = 0.f;
-        for (int e = lane; e < experts; e += 32) { const float p = expf(zr[e] + (bias ? bias[e] : 0.f) - m); my[e] = p; sum += p; }
+        for (int e = lane; e < experts; e += 32) { const float p = route_score(zr[e] + (bias ? bias[e] : 0.f), m, sigmoid); my[e] = p; sum += p; }
         sum = warp_sum(sum);
         __syncwarp();
-        const float inv = 1.f / sum;
+        const float inv = sigmoid ? 1.f : 1.f / sum;
         if (grouped) {                                      // (scratch behind the first rows: [8][experts] twice)
             float* extra = (float*)(start + experts + 1);
             route_choice_warp(lane, my, extra + (size_t)warp * experts, extra + (size_t)(8 + warp) * experts, inv, correction,
@@ -305,6 +312,7 @@ __global__ void __launch_bounds__(256) route_rows_small_kernel(int32_t* __restri
         const int p = start[e] + atomicAdd(cnt + e, 1);
         place[i] = p;
         token_of[p] = i / top;
+        if (row_weight) row_weight[p] = weight[i];
     }
 }
 
@@ -314,10 +322,11 @@ __global__ void expert_whole_kernel(int32_t* counts, int experts, int tokens) {
 }
 
 // hb_route_top and hb_expert_rows as one call. counts [2 experts + 3] need not be zeroed; afterwards it also holds, at
-// 2 experts + 1, the pair (0, tokens).
+// 2 experts + 1, the pair (0, tokens). row_weight [tokens top] (or null): the weight of each row's pair.
 extern "C" int hb_route_rows(int32_t* chosen, float* weight, int32_t* counts, int32_t* place, int32_t* token_of,
                              const float* z, const float* bias, int ld, int tokens, int experts, int top, float scale,
-                             int renormalize, const float* correction, int groups, int keep, float tiny, hb_stream stream) {
+                             int renormalize, const float* correction, int groups, int keep, float tiny, int sigmoid,
+                             float* row_weight, hb_stream stream) {
     if (tokens == 0) return 0;
     if (experts < 1 || top < 1 || top > experts || ld < experts) HB_REFUSE("route_rows: top %d of %d experts in rows of %d", top, experts, ld);
     if (groups < 1 || experts % groups || keep < 1 || keep > groups || (long)keep * (experts / groups) < top)
@@ -328,15 +337,15 @@ extern "C" int hb_route_rows(int32_t* chosen, float* weight, int32_t* counts, in
         const size_t smem = ((size_t)(grouped ? 24 : 8) * experts + 2 * experts + 1) * sizeof(float);
         if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(route_rows_small_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         route_rows_small_kernel<<<1, 256, smem, s>>>(chosen, weight, counts, place, token_of, z, ld, tokens, experts, top, scale,
-                                                     renormalize, bias, correction, groups, keep, tiny, grouped);
+                                                     renormalize, bias, correction, groups, keep, tiny, grouped, sigmoid, row_weight);
         HB_LAUNCH_CHECK("route_rows_small");
         return 0;
     }
     HB_CUDA(cudaMemsetAsync(counts, 0, (size_t)(2 * experts + 3) * sizeof(int32_t), s));
     int rc = hb_route_top(chosen, weight, counts, z, bias, ld, tokens, experts, top, scale, renormalize, correction, groups, keep,
-                          tiny, stream);
+                          tiny, sigmoid, stream);
     if (rc) return rc;
-    rc = hb_expert_rows(place, token_of, counts, chosen, tokens, top, experts, stream);
+    rc = hb_expert_rows(place, token_of, counts, chosen, tokens, top, experts, weight, row_weight, stream);
     if (rc) return rc;
     expert_whole_kernel<<<1, 1, 0, s>>>(counts, experts, tokens);
     HB_LAUNCH_CHECK("expert_whole");
@@ -531,7 +540,7 @@ extern "C" int hb_sigmoid_gate(void* o, const void* g, int dtype, int tokens, in
     return 0;
 }
 
-// ---------------------------------------------------------------- the weighted sum per token
+// ---------------------------------------------------------------- the weighted sum per token (weight null: every weight is 1)
 #define XC_TOP 64
 template <typename T>
 __global__ void expert_combine_kernel(T* __restrict__ out, const T* __restrict__ y, const int32_t* __restrict__ place,
@@ -543,14 +552,14 @@ __global__ void expert_combine_kernel(T* __restrict__ out, const T* __restrict__
     __shared__ float wgt[XC_TOP];
     const size_t t = blockIdx.x;
     const bool kept = top <= XC_TOP;
-    if (kept && threadIdx.x < top) { rows[threadIdx.x] = place[t * top + threadIdx.x]; wgt[threadIdx.x] = weight[t * top + threadIdx.x]; }
+    if (kept && threadIdx.x < top) { rows[threadIdx.x] = place[t * top + threadIdx.x]; wgt[threadIdx.x] = weight ? weight[t * top + threadIdx.x] : 1.f; }
     __syncthreads();
     const float gate = shared ? (z ? 1.f / (1.f + expf(-z[t * ldz + gate_at])) : 1.f) : 0.f;
     for (int i = blockIdx.y * blockDim.x + threadIdx.x; i < hidden; i += gridDim.y * blockDim.x) {
         float acc = 0.f;
         for (int k = 0; k < top; ++k) {
             const int p = kept ? rows[k] : place[t * top + k];
-            if (p >= 0) acc = fmaf(kept ? wgt[k] : weight[t * top + k],
+            if (p >= 0) acc = fmaf(kept ? wgt[k] : weight ? weight[t * top + k] : 1.f,
                                    to_f32(p >= ident ? x[t * hidden + i] : y[(size_t)p * hidden + i]), acc);
         }
         if (shared) acc = fmaf(gate, to_f32(shared[t * hidden + i]), acc);
@@ -567,7 +576,7 @@ __global__ void expert_combine_bf16x8_kernel(bf16* __restrict__ out, const bf16*
     __shared__ float wgt[XC_TOP];
     const int ident = identity_from ? *identity_from : 0x7fffffff;
     const size_t t = blockIdx.x;
-    if (threadIdx.x < top) { rows[threadIdx.x] = place[t * top + threadIdx.x]; wgt[threadIdx.x] = weight[t * top + threadIdx.x]; }
+    if (threadIdx.x < top) { rows[threadIdx.x] = place[t * top + threadIdx.x]; wgt[threadIdx.x] = weight ? weight[t * top + threadIdx.x] : 1.f; }
     __syncthreads();
     const float gate = shared ? (z ? 1.f / (1.f + expf(-z[t * ldz + gate_at])) : 1.f) : 0.f;
     for (int i = (blockIdx.y * blockDim.x + threadIdx.x) * 8; i < hidden; i += gridDim.y * blockDim.x * 8) {

@@ -6,16 +6,32 @@
 //
 // hb_latent_prepare: per token, the rotation of each head's rotated query part into the folded queries, and (for a
 // layer that fills its cache entry) RMSNorm of the latent, rotation of the shared key part, and the write of both into
-// the token's cache row. hb_latent_attention_generic: one warp per (query token, head) on CUDA cores, the float32
+// the token's cache row; for queries that come from a latent of their own, that latent's RMSNorm. hb_latent_attention_generic: one warp per (query token, head) on CUDA cores, the float32
 // engine's attention and the bfloat16 engine's for sizes its tensor-core kernel refuses.
 #include "common.cuh"
 
+// Entry d of a part of which the first 2 half entries turn: pairs (d, d + half), or with `neighbours` (2i, 2i + 1); cs holds
+// the cosines of the half angles, then the sines.
+template <typename T>
+__device__ __forceinline__ float turned(const T* __restrict__ x, int d, const float* __restrict__ cs, int half, bool turn, int neighbours) {
+    const float v = to_f32(x[d]);
+    if (!turn || d >= 2 * half) return v;
+    const bool second = neighbours ? d & 1 : d >= half;
+    const int j = neighbours ? d >> 1 : second ? d - half : d;
+    const float c = cs[j], s = cs[half + j];
+    const float other = to_f32(x[neighbours ? d ^ 1 : second ? d - half : d + half]);
+    return second ? v * c + other * s : v * c - other * s;
+}
+
+// grid (tokens, segments): first the heads' rotated query parts, an element a thread; then a block for the token's cache
+// row (dkv_at >= 0) and one for the normed query latent (cq given).
 template <typename T, typename TW>
 __global__ void latent_prepare_kernel(T* __restrict__ qa, const T* __restrict__ first, int ld, int heads, int dim,
-                                      int rot, int rank, int dkv_at, const int32_t* __restrict__ positions,
-                                      const float* __restrict__ table, int rot_dims, int max_positions,
+                                      int rot, int rank, int dkv_at, T* __restrict__ cq, int cq_at, int q_rank,
+                                      const TW* __restrict__ cq_weight, const int32_t* __restrict__ positions,
+                                      const float* __restrict__ table, int rot_dims, int max_positions, int neighbours,
                                       const TW* __restrict__ norm_weight, float eps, T* __restrict__ cache,
-                                      const int32_t* __restrict__ write_index, long cache_rows) {
+                                      const int32_t* __restrict__ write_index, long cache_rows, int head_segments) {
     __shared__ float scratch[33];
     const int t = blockIdx.x;
     const T* fr = first + (size_t)t * ld;
@@ -24,56 +40,54 @@ __global__ void latent_prepare_kernel(T* __restrict__ qa, const T* __restrict__ 
     const bool turn = half > 0 && p >= 0 && p < max_positions;
     const float* cs = table + (size_t)(turn ? p : 0) * rot_dims;           // cosines, then sines
     const int dk = rank + rot;
-    if ((int)blockIdx.y < heads) {                     // this head's rotated query part -> qa[t, h, rank:]
-        const int h = blockIdx.y;
-        const T* q = fr + (size_t)h * (dim + rot) + dim;
-        for (int d = threadIdx.x; d < rot; d += blockDim.x) {
-            float v = to_f32(q[d]);
-            if (turn && d < rot_dims) {
-                const int j = d < half ? d : d - half;
-                const float c = cs[j], s = cs[half + j];
-                v = d < half ? v * c - to_f32(q[d + half]) * s : v * c + to_f32(q[d - half]) * s;
-            }
-            qa[((size_t)t * heads + h) * dk + rank + d] = from_f32<T>(v);
-        }
+    int seg = blockIdx.y;
+    if (seg < head_segments) {                         // rotated query parts -> qa[t, h, rank:]
+        const int e = seg * blockDim.x + threadIdx.x;
+        if (e >= heads * rot) return;
+        const int h = e / rot, d = e - h * rot;
+        qa[((size_t)t * heads + h) * dk + rank + d] = from_f32<T>(turned(fr + (size_t)h * (dim + rot) + dim, d, cs, half, turn, neighbours));
         return;
     }
-    if (dkv_at < 0) return;
-    const long w = write_index[t];
-    const T* d = fr + dkv_at;
+    seg -= head_segments;
+    const bool latent = dkv_at >= 0 && seg == 0;       // else: the query latent
+    const T* d = fr + (latent ? dkv_at : cq_at);
+    const int n = latent ? rank : q_rank;
     float ss = 0.f;
-    for (int i = threadIdx.x; i < rank; i += blockDim.x) { const float v = to_f32(d[i]); ss += v * v; }
-    const float rstd = rsqrtf(block_sum(ss, scratch) / (float)rank + eps);
+    for (int i = threadIdx.x; i < n; i += blockDim.x) { const float v = to_f32(d[i]); ss += v * v; }
+    const float rstd = rsqrtf(block_sum(ss, scratch) / (float)n + eps);
+    if (!latent) {
+        for (int i = threadIdx.x; i < n; i += blockDim.x) cq[(size_t)t * n + i] = from_f32<T>(to_f32(d[i]) * rstd * to_f32(cq_weight[i]));
+        return;
+    }
+    const long w = write_index[t];
     if (w < 0 || w >= cache_rows) return;
     T* row = cache + (size_t)w * dk;
     for (int i = threadIdx.x; i < rank; i += blockDim.x) row[i] = from_f32<T>(to_f32(d[i]) * rstd * to_f32(norm_weight[i]));
-    const T* kr = d + rank;
-    for (int i = threadIdx.x; i < rot; i += blockDim.x) {
-        float v = to_f32(kr[i]);
-        if (turn && i < rot_dims) {
-            const int j = i < half ? i : i - half;
-            const float c = cs[j], s = cs[half + j];
-            v = i < half ? v * c - to_f32(kr[i + half]) * s : v * c + to_f32(kr[i - half]) * s;
-        }
-        row[rank + i] = from_f32<T>(v);
-    }
+    for (int i = threadIdx.x; i < rot; i += blockDim.x) row[rank + i] = from_f32<T>(turned(d + rank, i, cs, half, turn, neighbours));
 }
 
 extern "C" int hb_latent_prepare(void* qa, const void* first, int dtype, int ld, int tokens, int heads, int dim, int rot,
-                                 int rank, int dkv_at, const int32_t* positions, const float* table, int rot_dims,
-                                 int max_positions, const void* norm_weight, int weight_dtype, float eps, void* cache,
+                                 int rank, int dkv_at, void* cq, int cq_at, int q_rank, const void* cq_weight,
+                                 const int32_t* positions, const float* table, int rot_dims, int max_positions, int neighbours,
+                                 const void* norm_weight, int weight_dtype, float eps, void* cache,
                                  const int32_t* write_index, int pages, int page_size, hb_stream stream) {
     if (tokens == 0) return 0;
     if (rot_dims % 2 || rot_dims > rot || rot_dims < 0) HB_REFUSE("latent_prepare: %d of %d dimensions turn", rot_dims, rot);
     if (rot_dims && !table) HB_REFUSE("latent_prepare: a rotation needs its table");
     if (dkv_at >= 0 && (!cache || !write_index || !norm_weight)) HB_REFUSE("latent_prepare: a layer that fills its cache needs cache, write_index and the latent's norm weight");
     if (dkv_at >= 0 && dkv_at + rank + rot > ld) HB_REFUSE("latent_prepare: the down-projection's columns end past the row");
+    if (qa && (long)heads * (dim + rot) > ld) HB_REFUSE("latent_prepare: the queries' columns end past the row");
+    if (cq && (!cq_weight || cq_at < 0 || q_rank < 1 || cq_at + q_rank > ld)) HB_REFUSE("latent_prepare: the query latent's columns end past the row, or its norm has no weight");
     cudaStream_t s = (cudaStream_t)stream;
     const long cache_rows = (long)pages * page_size;
-    if (heads + 1 > 65535) HB_REFUSE("latent_prepare: %d heads", heads);
-    dim3 grid(tokens, heads + (dkv_at >= 0 ? 1 : 0));      // a block a head, and one for the token's cache row
+    const long head_segments = qa ? ((long)heads * rot + 127) / 128 : 0;
+    const long segments = head_segments + (dkv_at >= 0 ? 1 : 0) + (cq ? 1 : 0);
+    if (segments == 0) return 0;
+    if (segments > 65535) HB_REFUSE("latent_prepare: %d heads", heads);
+    dim3 grid(tokens, (unsigned)segments);
 #define LP_GO(T_, TW_) latent_prepare_kernel<T_, TW_><<<grid, 128, 0, s>>>((T_*)qa, (const T_*)first, ld, heads, dim, rot, \
-        rank, dkv_at, positions, table, rot_dims, max_positions, (const TW_*)norm_weight, eps, (T_*)cache, write_index, cache_rows)
+        rank, dkv_at, (T_*)cq, cq_at, q_rank, (const TW_*)cq_weight, positions, table, rot_dims, max_positions, neighbours, \
+        (const TW_*)norm_weight, eps, (T_*)cache, write_index, cache_rows, (int)head_segments)
     if (dtype == HB_F32) LP_GO(float, float);
     else if (dtype == HB_BF16 && weight_dtype == HB_F32) LP_GO(bf16, float);
     else if (dtype == HB_BF16) LP_GO(bf16, bf16);
@@ -92,7 +106,8 @@ __global__ void latent_attention_generic_kernel(T* __restrict__ out, const T* __
                                                 const int32_t* __restrict__ block_table, int table_stride,
                                                 const int32_t* __restrict__ row_slot, const int32_t* __restrict__ query_start,
                                                 const int32_t* __restrict__ kv_len, int rows, int tokens, int heads,
-                                                int rank, int dk, int pages, int page_size, float scale, int window) {
+                                                int rank, int dk, int pages, int page_size, float scale, int window,
+                                                const float* __restrict__ sinks) {
     extern __shared__ float smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const long item = (long)blockIdx.x * LAT_WARPS + warp;
@@ -157,7 +172,11 @@ __global__ void latent_attention_generic_kernel(T* __restrict__ out, const T* __
             }
         }
     }
-    const float inv = l > 0.f ? 1.f / l : 0.f;
+    float inv = l > 0.f ? 1.f / l : 0.f;
+    if (sinks) {                                      // a weight exp(sink) in the denominator, without key or value
+        const float sink = sinks[h], top = fmaxf(m, sink), c = expf(m - top);
+        inv = c / (l * c + expf(sink - top));
+    }
 #pragma unroll
     for (int i = 0; i < LAT_MAX_PER_LANE; ++i) {
         const int d = lane + 32 * i;
@@ -169,7 +188,7 @@ extern "C" int hb_latent_attention_generic(void* out, const void* qa, const void
                                            const int32_t* block_table, int table_stride, const int32_t* row_slot,
                                            const int32_t* query_start, const int32_t* kv_len, int rows, int tokens,
                                            int heads, int rank, int rot, int pages, int page_size, float scale,
-                                           int window, hb_stream stream) {
+                                           int window, const float* sinks, hb_stream stream) {
     if (tokens == 0 || rows == 0) return 0;
     if (rank > 32 * LAT_MAX_PER_LANE) HB_REFUSE("latent attention: rank %d is above %d", rank, 32 * LAT_MAX_PER_LANE);
     cudaStream_t s = (cudaStream_t)stream;
@@ -180,11 +199,11 @@ extern "C" int hb_latent_attention_generic(void* out, const void* qa, const void
     if (dtype == HB_F32)
         latent_attention_generic_kernel<float><<<blocks, LAT_WARPS * 32, smem, s>>>(
             (float*)out, (const float*)qa, (const float*)cache, block_table, table_stride, row_slot, query_start, kv_len,
-            rows, tokens, heads, rank, dk, pages, page_size, scale, window);
+            rows, tokens, heads, rank, dk, pages, page_size, scale, window, sinks);
     else if (dtype == HB_BF16)
         latent_attention_generic_kernel<bf16><<<blocks, LAT_WARPS * 32, smem, s>>>(
             (bf16*)out, (const bf16*)qa, (const bf16*)cache, block_table, table_stride, row_slot, query_start, kv_len,
-            rows, tokens, heads, rank, dk, pages, page_size, scale, window);
+            rows, tokens, heads, rank, dk, pages, page_size, scale, window, sinks);
     else HB_REFUSE("latent attention: dtype %d", dtype);
     HB_LAUNCH_CHECK("latent_attention_generic");
     return 0;

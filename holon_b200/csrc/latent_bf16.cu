@@ -43,12 +43,19 @@ __device__ __forceinline__ uint32_t lb_pack(float lo, float hi) {
     return *(const uint32_t*)&v;
 }
 
+// 1 / (l + 2^(sink' - m)) for sums l relative to a base-2 maximum m, sink' = sink in base 2; written so that neither
+// exponential overflows.
+__device__ __forceinline__ float lb_sink_inverse(float m, float l, float sink) {
+    const float s2 = sink * 1.4426950408889634f, top = fmaxf(m, s2), c = exp2f(m - top);
+    return c / (l * c + exp2f(s2 - top));
+}
+
 template <int R, int W>
 __global__ void __launch_bounds__(W * 32, 1) latent_attention_bf16_kernel(
         bf16* __restrict__ out, float* __restrict__ scratch, const bf16* __restrict__ qa, const bf16* __restrict__ cache,
         const int32_t* __restrict__ block_table, int table_stride, const int32_t* __restrict__ row_slot,
         const int32_t* __restrict__ query_start, const int32_t* __restrict__ kv_len, int row0, int row1, int heads,
-        int rank, int dk, int pages, int page_size, float scale, int window, int splits) {
+        int rank, int dk, int pages, int page_size, float scale, int window, int splits, const float* __restrict__ sinks) {
     constexpr int MT = 16 * W / R;                         // query rows a CTA
     constexpr int LB_THREADS = W * 32;
     extern __shared__ __align__(16) unsigned char lb_smem[];
@@ -265,7 +272,11 @@ __global__ void __launch_bounds__(W * 32, 1) latent_attention_bf16_kernel(
 
     const int cq = (lane & 3) * 2;
     if (splits == 1) {
-        const float i_lo = l_lo > 0.f ? 1.f / l_lo : 0.f, i_hi = l_hi > 0.f ? 1.f / l_hi : 0.f;
+        float i_lo = l_lo > 0.f ? 1.f / l_lo : 0.f, i_hi = l_hi > 0.f ? 1.f / l_hi : 0.f;
+        if (sinks) {                                        // a weight exp(sink) in the denominator, without key or value
+            i_lo = lb_sink_inverse(m_lo, l_lo, sinks[(flat0 + r_lo) % heads]);
+            i_hi = lb_sink_inverse(m_hi, l_hi, sinks[(flat0 + r_hi) % heads]);
+        }
 #pragma unroll
         for (int p = 0; p < 16; ++p) {
             if (p < 2 * pairs) {
@@ -298,7 +309,8 @@ __global__ void __launch_bounds__(W * 32, 1) latent_attention_bf16_kernel(
 // every thread adds up its columns over the parts.
 #define LB_MERGE_MAX 64
 __global__ void __launch_bounds__(512) latent_attention_merge_kernel(bf16* __restrict__ out, const float* __restrict__ scratch,
-                                                                     long first_pair, int rank, int splits) {
+                                                                     long first_pair, int rank, int splits, int heads,
+                                                                     const float* __restrict__ sinks) {
     __shared__ float wgt[LB_MERGE_MAX];
     __shared__ float inv_l;
     const long i = first_pair + blockIdx.x;
@@ -317,7 +329,7 @@ __global__ void __launch_bounds__(512) latent_attention_merge_kernel(bf16* __res
             l += w * p[(size_t)s * width + 1];
         }
         l = warp_sum(l);
-        if (lane == 0) inv_l = l > 0.f ? 1.f / l : 0.f;
+        if (lane == 0) inv_l = sinks ? lb_sink_inverse(m, l, sinks[i % heads]) : l > 0.f ? 1.f / l : 0.f;
     }
     __syncthreads();
     const float inv = inv_l;
@@ -340,7 +352,8 @@ extern "C" int hb_latent_attention_bf16(void* out, float* scratch, const void* q
                                         const int32_t* block_table, int table_stride, const int32_t* row_slot,
                                         const int32_t* query_start, const int32_t* kv_len, int row0, int row1,
                                         int first_token, int tokens, int heads, int rank, int rot, int pages,
-                                        int page_size, float scale, int window, int splits, hb_stream stream) {
+                                        int page_size, float scale, int window, int splits, const float* sinks,
+                                        hb_stream stream) {
     if (tokens == 0 || row1 <= row0) return 0;
     const int dk = rank + rot;
     if (rank % 16 || rot % 16 || rank < 16 || rank > 512) HB_REFUSE("latent attention on tensor cores: rank %d and rot %d must be multiples of 16, rank 16 to 512", rank, rot);
@@ -358,14 +371,14 @@ extern "C" int hb_latent_attention_bf16(void* out, float* scratch, const void* q
 #define LB_GO(R_, W_) do { \
         if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(latent_attention_bf16_kernel<R_, W_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
         latent_attention_bf16_kernel<R_, W_><<<grid, W_ * 32, smem, s>>>((bf16*)out, scratch, (const bf16*)qa, (const bf16*)cache, \
-            block_table, table_stride, row_slot, query_start, kv_len, row0, row1, heads, rank, dk, pages, page_size, scale, window, splits); \
+            block_table, table_stride, row_slot, query_start, kv_len, row0, row1, heads, rank, dk, pages, page_size, scale, window, splits, sinks); \
     } while (0)
     if (warps == 4) { if (r == 1) LB_GO(1, 4); else if (r == 2) LB_GO(2, 4); else LB_GO(4, 4); }
     else { if (r == 1) LB_GO(1, 8); else if (r == 2) LB_GO(2, 8); else LB_GO(4, 8); }
 #undef LB_GO
     HB_LAUNCH_CHECK("latent_attention_bf16");
     if (splits > 1) {
-        latent_attention_merge_kernel<<<(unsigned)pairs, min(512, (rank + 31) / 32 * 32), 0, s>>>((bf16*)out, scratch, (long)first_token * heads, rank, splits);
+        latent_attention_merge_kernel<<<(unsigned)pairs, min(512, (rank + 31) / 32 * 32), 0, s>>>((bf16*)out, scratch, (long)first_token * heads, rank, splits, heads, sinks);
         HB_LAUNCH_CHECK("latent_attention_merge");
     }
     return 0;

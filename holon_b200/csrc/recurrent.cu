@@ -476,34 +476,35 @@ extern "C" int hb_conv_carry(void* conv_state, const void* first, int dtype, int
 }
 
 // ---------------------------------------------------------------- what the retention mixer's first product becomes
-// A token's row of `first` holds [q (heads dim) | k (heads dim) | v (heads vdim) | ...]. q and k turn by the token's
-// position (the first rot_dims channels of a head, half-split pairs, table [positions, rot_dims]: cosines then sines),
+// A token's row of `first` holds [q (heads dim) | k (heads dim) | v (heads vdim) | ...]. With `silu` every one of these
+// numbers passes silu first. q and k turn by the token's position (the first rot_dims channels of a head, half-split pairs, table [positions, rot_dims]: cosines then sines),
 // k is then scaled. grid (tokens, segments of 256 elements).
 template <typename T>
 __global__ void retention_prepare_kernel(float* __restrict__ qk, float* __restrict__ v, const T* __restrict__ first, int ld,
                                          const int32_t* __restrict__ positions, const float* __restrict__ table,
-                                         int rot_dims, int max_positions, int heads, int dim, int vdim, float k_scale) {
+                                         int rot_dims, int max_positions, int heads, int dim, int vdim, float k_scale, int silu) {
     const size_t t = blockIdx.x;
     const T* row = first + t * ld;
     const int pos = min(max(positions[t], 0), max_positions > 0 ? max_positions - 1 : 0);
     const float* cs = table ? table + (size_t)pos * rot_dims : nullptr;
     const int half = rot_dims >> 1, nq = heads * dim;
+    auto in = [&](int i) -> float { const float x = to_f32(row[i]); return silu ? silu_f(x) : x; };
     int e = blockIdx.y * blockDim.x + threadIdx.x;                       // an element a thread: q and k, then v
     if (e < 2 * nq) {
         const int d = e % dim;
-        float x = to_f32(row[e]);
-        if (d < half) x = x * cs[d] - to_f32(row[e + half]) * cs[half + d];
-        else if (d < rot_dims) x = x * cs[d - half] + to_f32(row[e - half]) * cs[d];
+        float x = in(e);
+        if (d < half) x = x * cs[d] - in(e + half) * cs[half + d];
+        else if (d < rot_dims) x = x * cs[d - half] + in(e - half) * cs[d];
         qk[t * 2 * nq + e] = e >= nq ? x * k_scale : x;
         return;
     }
     e -= 2 * nq;
-    if (e < heads * vdim) v[t * heads * vdim + e] = to_f32(row[2 * nq + e]);
+    if (e < heads * vdim) v[t * heads * vdim + e] = in(2 * nq + e);
 }
 
 extern "C" int hb_retention_prepare(float* qk, float* v, const void* first, int dtype, int ld, const int32_t* positions,
                                     const float* table, int rot_dims, int max_positions, int tokens, int heads, int dim,
-                                    int vdim, float k_scale, hb_stream stream) {
+                                    int vdim, float k_scale, int silu, hb_stream stream) {
     if (tokens == 0) return 0;
     if (rot_dims % 2 || rot_dims < 0 || rot_dims > dim) HB_REFUSE("retention_prepare: %d rotated channels of %d", rot_dims, dim);
     if (rot_dims && !table) HB_REFUSE("retention_prepare: a rotation needs its table");
@@ -511,8 +512,8 @@ extern "C" int hb_retention_prepare(float* qk, float* v, const void* first, int 
     const long segments = (2L * heads * dim + (long)heads * vdim + 255) / 256;
     if (segments > 65535) HB_REFUSE("retention_prepare: %ld segments a token are above 65535", segments);
     const dim3 tokens_by_segments(tokens, (unsigned)segments);
-    if (dtype == HB_F32) retention_prepare_kernel<float><<<tokens_by_segments, 256, 0, s>>>(qk, v, (const float*)first, ld, positions, table, rot_dims, max_positions, heads, dim, vdim, k_scale);
-    else if (dtype == HB_BF16) retention_prepare_kernel<bf16><<<tokens_by_segments, 256, 0, s>>>(qk, v, (const bf16*)first, ld, positions, table, rot_dims, max_positions, heads, dim, vdim, k_scale);
+    if (dtype == HB_F32) retention_prepare_kernel<float><<<tokens_by_segments, 256, 0, s>>>(qk, v, (const float*)first, ld, positions, table, rot_dims, max_positions, heads, dim, vdim, k_scale, silu);
+    else if (dtype == HB_BF16) retention_prepare_kernel<bf16><<<tokens_by_segments, 256, 0, s>>>(qk, v, (const bf16*)first, ld, positions, table, rot_dims, max_positions, heads, dim, vdim, k_scale, silu);
     else HB_REFUSE("retention_prepare: dtype %d", dtype);
     HB_LAUNCH_CHECK("retention_prepare");
     return 0;
@@ -547,6 +548,47 @@ __global__ void head_norm_gate_kernel(T* __restrict__ out, const float* __restri
     }
 }
 
+// The same with a block per row: rows of several hundred numbers (a norm over all heads' channels together), four
+// neighbouring numbers a thread and turn, kept in shared memory between the two passes.
+template <typename T>
+__global__ void head_norm_gate_wide_kernel(T* __restrict__ out, const float* __restrict__ o, const float* __restrict__ weight,
+                                           const float* __restrict__ gate_mul, const T* __restrict__ gate_pre, long ld,
+                                           float eps, int heads, int vdim, int weight_heads, int gate_sigmoid) {
+    extern __shared__ __align__(16) float hn_row[];
+    __shared__ float scratch[33];
+    const long item = blockIdx.x, t = item / heads;
+    const int h = (int)(item - t * heads);
+    const float* x = o + item * vdim;
+    float ss = 0.f;
+    for (int d = threadIdx.x * 4; d < vdim; d += blockDim.x * 4) {
+        const float4 v = *(const float4*)(x + d);
+        *(float4*)(hn_row + d) = v;
+        ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
+    }
+    const float f = rsqrtf(block_sum(ss, scratch) / vdim + eps);
+    for (int d = threadIdx.x * 4; d < vdim; d += blockDim.x * 4) {
+        float y[4], w[4];
+        Vec4<float>::load(hn_row + d, y);
+#pragma unroll
+        for (int e = 0; e < 4; ++e) y[e] *= f;
+        if (weight) {
+            Vec4<float>::load(weight + (weight_heads ? (long)h * vdim : 0) + d, w);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) y[e] *= w[e];
+        }
+        if (gate_mul) {
+            Vec4<float>::load(gate_mul + item * vdim + d, w);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) y[e] *= w[e];
+        } else if (gate_pre) {
+            Vec4<T>::load(gate_pre + t * ld + (long)h * vdim + d, w);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) y[e] *= gate_sigmoid ? sigmoid_f(w[e]) : silu_f(w[e]);
+        }
+        Vec4<T>::store(out + item * vdim + d, y);
+    }
+}
+
 extern "C" int hb_head_norm_gate(void* out, const float* o, int dtype, const float* weight, const float* gate_mul,
                                  const void* gate_pre, long ld, float eps, int tokens, int heads, int vdim,
                                  int weight_heads, int gate_sigmoid, hb_stream stream) {
@@ -554,6 +596,16 @@ extern "C" int hb_head_norm_gate(void* out, const float* o, int dtype, const flo
     if (items == 0) return 0;
     const unsigned blocks = (unsigned)((items + 3) / 4);
     cudaStream_t s = (cudaStream_t)stream;
+    if (vdim >= 512 && vdim <= 12288 && vdim % 4 == 0 && ld % 4 == 0 && items <= 0x7fffffffL &&
+        (((uintptr_t)out | (uintptr_t)o | (uintptr_t)weight | (uintptr_t)gate_mul | (uintptr_t)gate_pre) & 15) == 0) {
+        const int threads = vdim >= 1024 ? 256 : 128;
+        const size_t smem = (size_t)vdim * sizeof(float);
+        if (dtype == HB_F32) head_norm_gate_wide_kernel<float><<<(unsigned)items, threads, smem, s>>>((float*)out, o, weight, gate_mul, (const float*)gate_pre, ld, eps, heads, vdim, weight_heads, gate_sigmoid);
+        else if (dtype == HB_BF16) head_norm_gate_wide_kernel<bf16><<<(unsigned)items, threads, smem, s>>>((bf16*)out, o, weight, gate_mul, (const bf16*)gate_pre, ld, eps, heads, vdim, weight_heads, gate_sigmoid);
+        else HB_REFUSE("head_norm_gate: dtype %d", dtype);
+        HB_LAUNCH_CHECK("head_norm_gate");
+        return 0;
+    }
     if (dtype == HB_F32) head_norm_gate_kernel<float><<<blocks, 128, 0, s>>>((float*)out, o, weight, gate_mul, (const float*)gate_pre, ld, eps, items, heads, vdim, weight_heads, gate_sigmoid);
     else if (dtype == HB_BF16) head_norm_gate_kernel<bf16><<<blocks, 128, 0, s>>>((bf16*)out, o, weight, gate_mul, (const bf16*)gate_pre, ld, eps, items, heads, vdim, weight_heads, gate_sigmoid);
     else HB_REFUSE("head_norm_gate: dtype %d", dtype);

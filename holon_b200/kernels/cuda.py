@@ -325,6 +325,32 @@ class CudaKernels:
                    _code(weight), ctypes.c_float(eps), ctypes.c_float(offset), self._i32(index, "index"), rows,
                    h.shape[1])
 
+    def add_layernorm(self, out, h, delta, scale, weight, eps, index, place=None) -> None:
+        """out = LayerNorm(v) · weight for v = h + scale · delta (delta None: v = h), which goes back to h unless `index`
+        gathers rows. `place` (int32 [tokens · top]): what is added to token t is scale · Σ_k delta[place[t · top + k]]."""
+        self._check(out, h, delta, weight, index, place)
+        tokens, dim = h.shape
+        rows = index.shape[0] if index is not None else tokens
+        if out.shape != (rows, dim) or weight.shape != (dim,) or (delta is not None and (h.dtype != torch.float32 or delta.dtype != out.dtype)):
+            raise KernelError("add_layernorm: h [tokens, dim] (float32 with a delta of out's dtype), out [rows, dim], weight [dim]")
+        top = 0
+        if place is None:
+            if delta is not None and delta.shape != h.shape:
+                raise KernelError("add_layernorm: delta must have h's shape")
+        else:
+            top = place.shape[0] // max(1, tokens)
+            if delta is None or delta.dim() != 2 or delta.shape[1] != dim or place.shape != (tokens * top,) or (tokens and top < 1):
+                raise KernelError("add_layernorm: place int32 [tokens * top] names rows of delta [*, dim]")
+        self._call("hb_add_layernorm", self._p(out), _code(out), self._p(h), _code(h), self._p(delta), ctypes.c_float(scale),
+                   self._i32(place, "place"), top, self._p(weight), _code(weight), ctypes.c_float(eps), self._i32(index, "index"),
+                   rows, dim)
+
+    def softcap(self, x, cap) -> None:
+        """x = cap · tanh(x / cap) in place (float32)."""
+        self._check(x)
+        self._f32("softcap", x)
+        self._call("hb_softcap", self._p(x), ctypes.c_long(x.numel()), ctypes.c_float(cap))
+
     def silu_mul(self, out, gate_up) -> None:
         self._check(out, gate_up)
         if gate_up.shape != (out.shape[0], 2 * out.shape[1]) or out.dtype != gate_up.dtype:
@@ -808,18 +834,25 @@ class CudaKernels:
                    self._i32(index, "index"), rows, dim, streams)
 
     def latent_prepare(self, qa, first, heads, dim, rot, rank, dkv_at, positions, table, rot_dims, norm_weight, eps,
-                       cache, write_index) -> None:
-        self._check(qa, first, positions, table, norm_weight, cache, write_index)
+                       cache, write_index, interleaved=False, cq=None, cq_at=0, cq_weight=None) -> None:
+        """csrc/api.h: hb_latent_prepare. `qa` None: no queries in these rows; `cq` [tokens, q_rank]: the RMS norm of
+        columns cq_at .. of `first` with `cq_weight`, the latent that queries are made from; `interleaved`: neighbours turn."""
+        self._check(qa, first, positions, table, norm_weight, cache, write_index, cq, cq_weight)
         t, ld = first.shape
-        if qa.shape != (t, heads, rank + rot) or qa.dtype != first.dtype or ld < heads * (dim + rot):
+        if cq is not None and (cq.shape[0] != t or cq.dtype != first.dtype or cq_weight is None or cq_weight.shape != (cq.shape[1],)
+                               or cq_at + cq.shape[1] > ld or (norm_weight is not None and norm_weight.dtype != cq_weight.dtype)):
+            raise KernelError("latent_prepare: cq [tokens, q_rank] of first's dtype, cq_weight [q_rank] of norm_weight's")
+        if qa is not None and (qa.shape != (t, heads, rank + rot) or qa.dtype != first.dtype or ld < heads * (dim + rot)):
             raise KernelError("latent_prepare: first [tokens, >= heads (dim + rot)], qa [tokens, heads, rank + rot], one dtype")
         if table is not None and (table.dtype != torch.float32 or table.shape[1] != rot_dims):
             raise KernelError("latent_prepare: the rotation table must be float32 [positions, rot_dims]")
         if cache is not None and (cache.dtype != first.dtype or cache.dim() != 3 or cache.shape[2] != rank + rot):
             raise KernelError("latent_prepare: cache must be [pages, page_size, rank + rot] of first's dtype")
         self._call("hb_latent_prepare", self._p(qa), self._p(first), _code(first), ld, t, heads, dim, rot, rank, int(dkv_at),
+                   self._p(cq), int(cq_at), cq.shape[1] if cq is not None else 0, self._p(cq_weight),
                    self._i32(positions, "positions"), self._p(table), int(rot_dims), table.shape[0] if table is not None else 0,
-                   self._p(norm_weight), _code(norm_weight) if norm_weight is not None else 0, ctypes.c_float(eps),
+                   int(bool(interleaved)), self._p(norm_weight),
+                   _code(norm_weight) if norm_weight is not None else _code(cq_weight) if cq_weight is not None else 0, ctypes.c_float(eps),
                    self._p(cache), self._i32(write_index, "write_index"), cache.shape[0] if cache is not None else 0,
                    cache.shape[1] if cache is not None else 1)
 
@@ -844,8 +877,12 @@ class CudaKernels:
                 self.flush()
             torch.bmm(x.transpose(0, 1), w.transpose(1, 2), out=out.transpose(0, 1))
 
-    def latent_attention(self, out, qa, cache, block_table, rows, scale, rank, window) -> None:
-        self._check(out, qa, cache, block_table, rows.row_slot, rows.query_start, rows.kv_len)
+    def latent_attention(self, out, qa, cache, block_table, rows, scale, rank, window, sinks=None) -> None:
+        """`sinks` (float32 [heads], or None): exp(sinks[h]) stands in each head's softmax denominator besides."""
+        self._check(out, qa, cache, block_table, rows.row_slot, rows.query_start, rows.kv_len, sinks)
+        self._f32("latent_attention", sinks)
+        if sinks is not None and sinks.shape != (qa.shape[1],):
+            raise KernelError("latent_attention: sinks must be float32 [heads]")
         t, heads, dk = qa.shape
         if out.shape != (t, heads, rank) or cache.dim() != 3 or cache.shape[2] != dk or not (out.dtype == qa.dtype == cache.dtype):
             raise KernelError("latent_attention: qa [tokens, heads, rank + rot], out [tokens, heads, rank], cache [pages, "
@@ -858,18 +895,18 @@ class CudaKernels:
         if not fast:                                  # float32, and sizes the tensor-core kernel does not take
             return self._call("hb_latent_attention_generic", self._p(out), self._p(qa), self._p(cache), _code(qa), *common,
                               rows.n_rows, t, heads, rank, rot, cache.shape[0], cache.shape[1], ctypes.c_float(scale),
-                              int(window))
+                              int(window), self._p(sinks))
         sizes = (heads, rank, rot, cache.shape[0], cache.shape[1], ctypes.c_float(scale), int(window))
         ones = rows.n_decode
         if ones:                                      # rows of one token: their keys cut into parts that fill the GPU
-            splits = self.latent_splits(ones, heads, rank, rows.max_kv)
+            splits = self.latent_splits(ones, heads, rank, min(rows.max_kv, window + 63) if window else rows.max_kv)
             scratch = torch.empty(ones * heads * splits * (rank + 2), dtype=torch.float32, device=self.device) \
                 if splits > 1 else None
             self._call("hb_latent_attention_bf16", self._p(out), self._p(scratch), self._p(qa), self._p(cache), *common,
-                       0, ones, 0, ones, *sizes, splits)
+                       0, ones, 0, ones, *sizes, splits, self._p(sinks))
         if rows.n_rows > ones:
             self._call("hb_latent_attention_bf16", self._p(out), None, self._p(qa), self._p(cache), *common, ones,
-                       rows.n_rows, ones, t - ones, *sizes, 1)
+                       rows.n_rows, ones, t - ones, *sizes, 1, self._p(sinks))
 
     def latent_splits(self, rows: int, heads: int, rank: int, max_kv: int) -> int:
         """Parts the keys of one-token rows are cut into for the latent attention kernel: enough that two CTAs an SM
@@ -896,12 +933,15 @@ class CudaKernels:
             raise KernelError("activation: xielu takes two numbers")
         self._call("hb_activation", self._p(x), _code(x), ctypes.c_long(x.numel()), int(act), self._p(numbers))
 
+    SCORES = {"softmax": 0, "sigmoid": 1}     # how a router's logits become scores
+
     def route_top(self, chosen, weight, counts, z, experts, scale, renormalize, bias=None, correction=None, groups=1,
-                  keep=1, tiny=0.0) -> None:
+                  keep=1, tiny=0.0, scores="softmax") -> None:
         """`bias` (float32 [experts] or None) is added to the logits before anything else. `correction` (float32 [experts]
         or None) is added to the softmax scores for the choice alone; `groups` > 1: experts in that many equal groups of
         neighbours, of which the `keep` best (by their best choice score) stay in the running; `tiny` is added to the
-        chosen scores' sum before `renormalize` divides."""
+        chosen scores' sum before `renormalize` divides. `scores` "sigmoid": each logit's own sigmoid in place of its share
+        of the softmax."""
         self._check(chosen, weight, counts, z, bias, correction)
         self._f32("route_top", bias, correction)
         t, top = chosen.shape
@@ -911,14 +951,17 @@ class CudaKernels:
                               "counts int32 [2 experts + 1]")
         self._call("hb_route_top", self._i32(chosen, "chosen"), self._p(weight), self._i32(counts, "counts"), self._p(z),
                    self._p(bias), z.shape[1], t, int(experts), top, ctypes.c_float(scale), int(bool(renormalize)),
-                   self._p(correction), int(groups), int(keep), ctypes.c_float(tiny))
+                   self._p(correction), int(groups), int(keep), ctypes.c_float(tiny), self.SCORES[scores])
 
     def route_rows(self, chosen, weight, counts, place, token_of, z, experts, scale, renormalize, bias=None,
-                   correction=None, groups=1, keep=1, tiny=0.0) -> None:
+                   correction=None, groups=1, keep=1, tiny=0.0, scores="softmax", row_weight=None) -> None:
         """`route_top` and `expert_rows` as one call (one launch for a few tokens). counts int32 [2 experts + 3] need not
-        be zeroed; afterwards counts[2 experts + 1:] = (0, tokens)."""
-        self._check(chosen, weight, counts, place, token_of, z, bias, correction)
-        self._f32("route_rows", bias, correction)
+        be zeroed; afterwards counts[2 experts + 1:] = (0, tokens). `row_weight` (float32 [tokens * top] or None): the weight
+        of each row's pair."""
+        self._check(chosen, weight, counts, place, token_of, z, bias, correction, row_weight)
+        self._f32("route_rows", bias, correction, row_weight)
+        if row_weight is not None and row_weight.numel() != chosen.numel():
+            raise KernelError("route_rows: row_weight must be float32 [tokens * top]")
         if correction is not None and correction.shape != (experts,):
             raise KernelError("route_rows: correction must be float32 [experts]")
         t, top = chosen.shape
@@ -929,7 +972,8 @@ class CudaKernels:
                               "counts int32 [2 experts + 3], place and token_of int32 [tokens * top]")
         self._call("hb_route_rows", self._i32(chosen, "chosen"), self._p(weight), self._i32(counts, "counts"),
                    self._i32(place, "place"), self._i32(token_of, "token_of"), self._p(z), self._p(bias), z.shape[1], t, int(experts), top,
-                   ctypes.c_float(scale), int(bool(renormalize)), self._p(correction), int(groups), int(keep), ctypes.c_float(tiny))
+                   ctypes.c_float(scale), int(bool(renormalize)), self._p(correction), int(groups), int(keep), ctypes.c_float(tiny),
+                   self.SCORES[scores], self._p(row_weight))
 
     def expert_rows(self, place, token_of, counts, chosen, experts) -> None:
         self._check(place, token_of, counts, chosen)
@@ -937,7 +981,7 @@ class CudaKernels:
         if place.shape[0] != t * top or token_of.shape[0] != t * top or counts.shape[0] < 2 * experts + 1:
             raise KernelError("expert_rows: place and token_of int32 [tokens * top], counts int32 [2 experts + 1]")
         self._call("hb_expert_rows", self._i32(place, "place"), self._i32(token_of, "token_of"), self._i32(counts, "counts"),
-                   self._i32(chosen, "chosen"), t, top, int(experts))
+                   self._i32(chosen, "chosen"), t, top, int(experts), self._p(None), self._p(None))
 
     EXPERT_TCGEN05_ROWS = 96                  # rows an expert on average from which its products run on tcgen05
 
@@ -965,11 +1009,11 @@ class CudaKernels:
                    self._i32(starts, "starts"), rows, e, n, k, int(act))
 
     def expert_combine(self, out, y, place, weight, shared, z, experts, x=None, identity_from=None) -> None:
-        """`z` None with `shared`: the shared rows are added without a gate. `x` [tokens, hidden] and `identity_from`
+        """`weight` None: the rows are added as they are. `z` None with `shared`: the shared rows are added without a gate. `x` [tokens, hidden] and `identity_from`
         (int32 [1] on the device): pairs whose row is identity_from[0] or later read x[token] in place of y."""
         self._check(out, y, place, weight, shared, z, x, identity_from)
         t, hidden = out.shape
-        top = weight.shape[1]
+        top = weight.shape[1] if weight is not None else place.shape[0] // max(1, t)
         if y.shape != (t * top, hidden) or y.dtype != out.dtype or place.shape[0] != t * top \
                 or (shared is not None and (shared.shape != out.shape or shared.dtype != out.dtype))\
                 or (z is not None and (z.dtype != torch.float32 or z.shape[1] <= experts)) \
@@ -1020,12 +1064,24 @@ class CudaKernels:
                    self._p(bias), _code(out), self._p(out), self._p(weight), _code(weight), ctypes.c_float(eps),
                    ctypes.c_float(offset), h.shape[0], h.shape[1])
 
-    def glu_clamped(self, out, gate_up, bias, limit, alpha) -> None:
-        self._check(out, gate_up, bias)
+    def expert_glu(self, out, x, token_of, w, starts, limit, alpha, row_scale) -> None:
+        """A clamped gated unit's first half for rows laid out expert by expert: out [rows, inter] from x (gathered by
+        token_of) through w [experts, 2 inter, k] (an expert's gate rows, then its up rows), each row of the product times
+        row_scale (float32 [rows] or None) before the limits: glu_clamped behind expert_linear."""
+        both = torch.empty(out.shape[0], w.shape[1], dtype=out.dtype, device=self.device)
+        self.expert_linear(both, x, token_of, w, starts, 0)
+        self.glu_clamped(out, both, None, limit, alpha, row_scale=row_scale)
+
+    def glu_clamped(self, out, gate_up, bias, limit, alpha, row_scale=None) -> None:
+        """`row_scale` (float32 [tokens] or None): a factor on each row of gate_up, before the bias."""
+        self._check(out, gate_up, bias, row_scale)
+        self._f32("glu_clamped", row_scale)
+        if row_scale is not None and row_scale.shape != (out.shape[0],):
+            raise KernelError("glu_clamped: row_scale must be float32 [tokens]")
         if gate_up.shape != (out.shape[0], 2 * out.shape[1]) or out.dtype != gate_up.dtype \
                 or (bias is not None and (bias.shape != (gate_up.shape[1],) or bias.dtype != out.dtype)):
             raise KernelError("glu_clamped: gate_up [tokens, 2 inter] and bias [2 inter] of out's dtype")
-        self._call("hb_glu_clamped", self._p(out), self._p(gate_up), self._p(bias), _code(out), ctypes.c_float(limit),
+        self._call("hb_glu_clamped", self._p(out), self._p(gate_up), self._p(bias), self._p(row_scale), _code(out), ctypes.c_float(limit),
                    ctypes.c_float(alpha), out.shape[0], out.shape[1])
 
     @staticmethod
@@ -1082,7 +1138,8 @@ class CudaKernels:
         self._call("hb_conv_carry", self._p(conv_state), self._p(first), _code(first), first.shape[1], channels, taps,
                    self._i32(rows.query_start, "query_start"), self._i32(rows.row_slot, "row_slot"), rows.n_rows)
 
-    def retention_prepare(self, qk, v, first, positions, table, rot_dims, k_scale) -> None:
+    def retention_prepare(self, qk, v, first, positions, table, rot_dims, k_scale, silu=False) -> None:
+        """`silu`: q, k and v pass silu before anything else (csrc/api.h: hb_retention_prepare)."""
         self._check(qk, v, first, positions, table)
         self._f32("retention_prepare", qk, v, table)
         t, heads, vdim = v.shape
@@ -1092,7 +1149,7 @@ class CudaKernels:
             raise KernelError("retention_prepare: qk [tokens, 2, heads, dim], v [tokens, heads, vdim], first [tokens, q | k | v | ...]")
         self._call("hb_retention_prepare", self._p(qk), self._p(v), self._p(first), _code(first), first.shape[1],
                    self._i32(positions, "positions"), self._p(table), int(rot_dims),
-                   table.shape[0] if table is not None else 0, t, heads, dim, vdim, ctypes.c_float(k_scale))
+                   table.shape[0] if table is not None else 0, t, heads, dim, vdim, ctypes.c_float(k_scale), int(bool(silu)))
 
     def gdelta_prepare(self, qk, v, decay, rate, first, pre, decay_bias, rate_bias, decay_scale, unit_eps) -> None:
         """From the generalized delta rule's first product [tokens, r | k | v | g | a] and its low-rank decay projection's

@@ -7,10 +7,10 @@ from .experts import Experts
 from .feedforward import MLP, ClampedGLU, SwiGLU
 from .hyper import Hyper
 from .latent import LatentAttention
-from .norm import DynamicTanh, RMSNorm
+from .norm import DynamicTanh, LayerNorm, RMSNorm
 from .parallel import ParallelBlock, SideBySide
 from .position import Rope
-from .recurrent import MLSTM, GatedDelta, GeneralDelta, Retention
+from .recurrent import MLSTM, GatedDelta, GeneralDelta, Lightning, Retention
 
 register_part("norm", "rmsnorm", RMSNorm, replace=True)
 register_part("position", "rope", Rope, replace=True)
@@ -35,3 +35,5 @@ register_part("block", "outnorm", OutNorm, replace=True)
 register_part("norm", "dyt", DynamicTanh, replace=True)
 register_part("block", "sandwich", Sandwich, replace=True)
 register_part("mixer", "general_delta", GeneralDelta, replace=True)
+register_part("norm", "layernorm", LayerNorm, replace=True)
+register_part("mixer", "lightning", Lightning, replace=True)

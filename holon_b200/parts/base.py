@@ -178,16 +178,44 @@ class Residual:
     added its output itself and left the next norm's rows behind (`normed`, made with the weight of `normed_by`):
     then that norm has nothing left to launch."""
 
-    __slots__ = ("h", "delta", "delta_by", "normed", "normed_by")
+    __slots__ = ("h", "delta", "delta_scale", "delta_by", "normed", "normed_by")
 
-    def __init__(self, h: torch.Tensor, delta: torch.Tensor | None = None) -> None:
+    def __init__(self, h: torch.Tensor, delta: "torch.Tensor | PairRows | None" = None) -> None:
         self.h, self.delta = h, delta
+        self.delta_scale = 1.0               # a factor on `delta` (a block's residual multiplier)
         self.delta_by = None                 # a norm that `delta` passes before it is added (None: added as it is)
         self.normed, self.normed_by = None, None
 
     def final_rows(self, norm, index: torch.Tensor) -> torch.Tensor:
         """The rows `index` of what the last block left, under the model's last norm (what the head reads)."""
-        return norm.gather(self, index)
+        return norm.gather(self.settled(norm), index)
+
+    def settled(self, norm) -> "Residual":
+        """This stream as `norm` can read it: a pending output that is still rows of (token, choice) pairs is added up
+        per token, and a pending factor is applied, unless the norm does either itself (`takes_pairs`)."""
+        if self.delta is not None and not getattr(norm, "takes_pairs", False):
+            if isinstance(self.delta, PairRows):
+                self.delta = self.delta.combined()
+            if self.delta_scale != 1.0:
+                norm.ctx.kernels.sum_into(self.h, [(self.delta, self.delta_scale)])
+                self.delta = None
+        self.delta_scale = self.delta_scale if self.delta is not None else 1.0
+        return self
+
+
+class PairRows:
+    """A feed-forward's output before the sum per token: token t's output is the sum of the rows `y[place[t · top + k]]`,
+    k < top. A norm that says `takes_pairs` adds the rows while it reads them."""
+
+    __slots__ = ("y", "place", "tokens", "ctx")
+
+    def __init__(self, ctx: BuildContext, y: torch.Tensor, place: torch.Tensor, tokens: int) -> None:
+        self.ctx, self.y, self.place, self.tokens = ctx, y, place, tokens
+
+    def combined(self) -> torch.Tensor:
+        out = self.ctx.empty(self.tokens, self.y.shape[1])
+        self.ctx.kernels.expert_combine(out, self.y, self.place, None, None, None, 0)
+        return out
 
 
 class Scaled:

@@ -1,7 +1,8 @@
 """Pre-norm residual block: h += mixer(input_norm(h)); h += ffn(post_norm(h))
 (std/holon_std/blocks/units.py:8-25). The sums are folded into the next norm's kernel: the block leaves the
 feed-forward's output pending on the stream. For the few rows of a decode step sum and norm move one kernel further
-up, into the product that ends the mixer or the feed-forward (base.Link, base.Scaled).
+up, into the product that ends the mixer or the feed-forward (base.Link, base.Scaled). `residual_mult` m: h += m ·
+mixer(...), h += m · ffn(...); the factor waits on the stream beside the output it belongs to.
 
 OutNorm: the norm stands on a sublayer's OUTPUT, and the sublayers read the stream itself: x ← x + N(mixer(x)), then
 x ← x + N(ffn(x)). With `average` = n the block ends with an average over depth: with X_0 the embedding's rows and X_j
@@ -24,9 +25,9 @@ from .base import BuildContext, Link, Part, Residual, SlotState
 
 class PreNorm(Part):
     def __init__(self, ctx: BuildContext, *, layer: int, hidden: int, mixer: PartRef, ffn: PartRef | None,
-                 norm: PartRef) -> None:
+                 norm: PartRef, residual_mult: float = 1.0) -> None:
         super().__init__()
-        self.ctx = ctx
+        self.ctx, self.mult = ctx, float(residual_mult)
         self.input_norm = self.add_child("input_norm", ctx.part(norm, dim=hidden))
         self.mixer = self.add_child("mixer", ctx.part(mixer, layer=layer, hidden=hidden))
         self.post_norm = self.ffn = None                             # (a layer may have a mixer only)
@@ -41,20 +42,26 @@ class PreNorm(Part):
         take them unscaled."""
         x = self.input_norm.add(stream)
         if self.ffn is None:
-            stream.delta = self.mixer.forward(x, step, cache)
+            stream.delta, stream.delta_scale = self.mixer.forward(x, step, cache), self.mult
             return stream
         step.link = self._offer(stream, step, self.post_norm, self.ffn)
-        stream.delta = self.mixer.forward(x, step, cache)
+        stream.delta, stream.delta_scale = self.mixer.forward(x, step, cache), self.mult
         step.link = None                                             # (an offer nobody took lapses)
         x = self.post_norm.add(stream)
-        step.link = self._offer(stream, step, getattr(after, "input_norm", None), getattr(after, "mixer", None))
-        stream.delta = self.ffn.forward(x, step)
+        nxt = getattr(after, "input_norm", None)
+        step.link = self._offer(stream, step, nxt, getattr(after, "mixer", None))
+        if getattr(self.ffn, "leaves_pairs", False) and (after is None or getattr(nxt, "takes_pairs", False)):
+            stream.delta = self.ffn.forward(x, step, pairs=True)     # (the next norm adds up each token's rows itself)
+        else:
+            stream.delta = self.ffn.forward(x, step)
+        stream.delta_scale = self.mult
         step.link = None
         return stream
 
     def _offer(self, stream, step, norm, reader):
         can = getattr(self.ctx.kernels, "can_link", None)
-        if can is None or not getattr(reader, "takes_scaled", False) or not hasattr(norm, "weight"):
+        if can is None or not getattr(reader, "takes_scaled", False) or not hasattr(norm, "weight") \
+                or not getattr(norm, "links", True) or self.mult != 1.0:
             return None
         return Link(stream, norm) if can(step.rows.n_tokens, stream.h.shape[1], norm) else None
 
@@ -87,8 +94,8 @@ class OutNorm(Part):
         k, ctx = self.ctx.kernels, self.ctx
         t, hidden = stream.h.shape
         if stream.delta is not None:                                     # (what a block of another kind left pending)
-            k.sum_into(stream.h, [(stream.delta, 1.0)])
-            stream.delta = None
+            k.sum_into(stream.h, [(stream.delta, stream.delta_scale)])
+            stream.delta, stream.delta_scale = None, 1.0
         stream.normed = stream.normed_by = None
         state = step.shared.get(self.KEY)
         if state is None:                                                # the first block of the step

@@ -1,5 +1,5 @@
 """Token embedding (a row gather, no scaling) and the output head (logits in 32-bit; a tied head reads the
-embedding's table) (std/holon_std/ops/units.py:280-348)."""
+embedding's table; with `softcap` c the logits become c · tanh(logits / c)) (std/holon_std/ops/units.py:280-348)."""
 from __future__ import annotations
 
 import torch
@@ -46,9 +46,12 @@ class PairEmbedding(Embedding):
 
 
 class Head(Part):
-    def __init__(self, ctx: BuildContext, *, vocab: int, hidden: int, tied: bool, embed: Embedding | None) -> None:
+    def __init__(self, ctx: BuildContext, *, vocab: int, hidden: int, tied: bool, embed: Embedding | None,
+                 softcap: float | None = None) -> None:
         super().__init__()
-        self.ctx, self.vocab = ctx, vocab
+        if softcap is not None and not softcap > 0:
+            raise ValueError(f"head: softcap {softcap} must be positive")
+        self.ctx, self.vocab, self.cap = ctx, vocab, softcap
         if tied and embed is None:
             raise ValueError("a tied head needs the embedding")
         self._embed = embed if tied else None
@@ -58,4 +61,6 @@ class Head(Part):
         w = self._embed.weight.tensor if self._embed is not None else self.weight.tensor
         logits = self.ctx.empty(x.shape[0], self.vocab, dtype=torch.float32)
         self.ctx.kernels.linear(logits, x, w)
+        if self.cap is not None:
+            self.ctx.kernels.softcap(logits, self.cap)
         return logits

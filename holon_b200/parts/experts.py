@@ -14,6 +14,13 @@ a last kernel adds each token's `top` rows in the order of its choices, so the s
 the batch. For few tokens the shared expert's first product runs in the experts' kernel too, as one expert that
 takes every token, with its activation in the epilogue.
 
+`scores` "sigmoid": s_e = sigmoid(z_e), each expert's own, in place of the softmax. `weight_on` "input": the weight multiplies
+what the expert reads, y = Σ_chosen expert_e(weight_e · x), and the outputs are added as they are; since an expert's first
+product is linear, the weight is applied to that product's rows in 32-bit, ahead of the limits. `activation` "clamped" (gated,
+without biases; the form of parts/feedforward.py: ClampedGLU): g = min(W_gate x, limit), u = clamp(W_up x, −limit, limit),
+W_down (g · sigmoid(alpha · g) · (u + 1)). Where outputs are added as they are, with no shared or identity experts beside them, the sum
+per token can be left to the norm that reads it (`leaves_pairs`, base.PairRows).
+
 `identity` more experts stand behind the real ones in the router's rows: they have no tensors, their output is their
 input. With `groups` G > 1 the experts (identity ones included) form G equal groups of neighbours; a group's score is its
 largest choice score, and only experts of the `keep_groups` best groups can be chosen. With `correction` a stored vector
@@ -28,7 +35,7 @@ from __future__ import annotations
 
 import torch
 
-from .base import BuildContext, Part
+from .base import BuildContext, PairRows, Part
 from .linear import Linear
 
 ACTIVATIONS = {"relu2": 1, "silu": 2, "gelu_tanh": 3, "xielu": 4, "tanh": 5}
@@ -39,22 +46,33 @@ class Experts(Part):
     def __init__(self, ctx: BuildContext, *, experts: int, top: int, scale: float, inter: int, hidden: int,
                  shared_inter: int | None = None, activation: str = "relu2", renormalize: bool = False,
                  gated: bool = False, router_bias: bool = False, identity: int = 0, groups: int = 1, keep_groups: int = 1,
-                 correction: bool = False, shared_gated: bool = False, tiny: float = 0.0, layer: int = 0) -> None:
+                 correction: bool = False, shared_gated: bool = False, tiny: float = 0.0, scores: str = "softmax",
+                 weight_on: str = "output", limit: float | None = None, alpha: float = 1.702, layer: int = 0) -> None:
         super().__init__()
-        if activation not in EXPERT_ACTIVATIONS:
-            raise ValueError(f"experts: activation {activation!r}; known: {sorted(EXPERT_ACTIVATIONS)}")
+        if activation not in (*EXPERT_ACTIVATIONS, "clamped"):
+            raise ValueError(f"experts: activation {activation!r}; known: {sorted((*EXPERT_ACTIVATIONS, 'clamped'))}")
+        if scores not in ("softmax", "sigmoid") or weight_on not in ("output", "input"):
+            raise ValueError(f"experts: scores {scores!r} (softmax, sigmoid), weight_on {weight_on!r} (output, input)")
+        self.clamped = activation == "clamped"
+        if self.clamped and (not gated or limit is None or shared_inter):
+            raise ValueError("experts: clamped experts are gated, have a limit and no shared expert beside them")
+        if weight_on == "input" and (not self.clamped or identity):
+            raise ValueError("experts: a weight on the input is built for clamped gated experts, without identity experts")
+        self.scores, self.weight_in = scores, weight_on == "input"
+        self.limit, self.alpha = float(limit) if limit is not None else 0.0, float(alpha)
+        self.leaves_pairs = self.weight_in
         if identity < 0 or not 1 <= top <= experts + identity:
             raise ValueError(f"experts: top {top} of {experts} experts and {identity} identity experts")
         if groups < 1 or (experts + identity) % groups or not 1 <= keep_groups <= groups \
                 or keep_groups * ((experts + identity) // groups) < top:
             raise ValueError(f"experts: {groups} groups of which {keep_groups} are kept, for top {top} of {experts + identity}")
         self.ctx, self.experts, self.top, self.scale, self.inter, self.hidden = ctx, experts, top, float(scale), inter, hidden
-        self.act, self.renormalize, self.shared_inter = ACTIVATIONS[activation], bool(renormalize), shared_inter
+        self.act, self.renormalize, self.shared_inter = ACTIVATIONS.get(activation, 0), bool(renormalize), shared_inter
         self.gated, self.shared_gated = bool(gated), bool(shared_gated)
         self.identity, self.routed = int(identity), experts + int(identity)        # routed: the router's rows
         self.groups, self.keep_groups, self.tiny = int(groups), int(keep_groups), float(tiny)
-        if self.gated and (activation != "silu" or (shared_inter and not shared_gated)):
-            raise ValueError("experts: gated experts have silu gates, and a shared expert beside them is gated too")
+        if self.gated and (activation not in ("silu", "clamped") or (shared_inter and not shared_gated)):
+            raise ValueError("experts: gated experts have silu or clamped gates, and a shared expert beside them is gated too")
         if self.shared_gated and not self.gated:
             raise ValueError("experts: a gated shared expert goes with gated experts")
         pieces = {"router": self.routed}
@@ -90,7 +108,8 @@ class Experts(Part):
 
     FEW = 8                  # rows up to which the shared expert's first product runs in the experts' kernel
 
-    def forward(self, x: torch.Tensor, step) -> torch.Tensor:
+    def forward(self, x: torch.Tensor, step, pairs: bool = False) -> torch.Tensor | PairRows:
+        """`pairs` (only where `leaves_pairs`): the sum per token is left to whoever reads the result (base.PairRows)."""
         t, k, ctx, e, top = x.shape[0], self.ctx.kernels, self.ctx, self.experts, self.top
         r = self.routed                                                  # the router's rows: real experts, then identity ones
         z = self.router.forward(x, out_dtype=torch.float32)             # [t, routed (+ 1)]: router logits, gate
@@ -100,17 +119,24 @@ class Experts(Part):
         place = ctx.empty(t * top, dtype=torch.int32)                    # the row of each (token, choice)
         token_of = ctx.empty(t * top, dtype=torch.int32)                 # the token of each row
         bias = self.route_bias.tensor if self.route_bias is not None else None
-        if self.correction is not None or self.groups > 1 or self.tiny:
+        row_weight = ctx.empty(t * top, dtype=torch.float32) if self.weight_in else None
+        extra = {} if self.scores == "softmax" else {"scores": self.scores}
+        if row_weight is not None:
+            extra["row_weight"] = row_weight
+        if self.correction is not None or self.groups > 1 or self.tiny or extra:
             k.route_rows(chosen, weight, counts, place, token_of, z, r, self.scale, self.renormalize, bias,
                          correction=self.correction.tensor if self.correction is not None else None, groups=self.groups,
-                         keep=self.keep_groups, tiny=self.tiny)
+                         keep=self.keep_groups, tiny=self.tiny, **extra)
         elif bias is not None:
             k.route_rows(chosen, weight, counts, place, token_of, z, r, self.scale, self.renormalize, bias)
         else:
             k.route_rows(chosen, weight, counts, place, token_of, z, r, self.scale, self.renormalize)
         starts = counts[r:r + e + 1]                                     # rows are laid out expert by expert: the real ones first
         act = ctx.empty(t * top, self.inter)
-        if self.gated:
+        if self.clamped:
+            k.expert_glu(act, x, token_of, self.up.tensor.view(e, 2 * self.inter, self.hidden), starts, self.limit, self.alpha,
+                         row_weight)
+        elif self.gated:
             both = ctx.empty(t * top, 2 * self.inter)
             k.expert_linear(both, x, token_of, self.up.tensor.view(e, 2 * self.inter, self.hidden), starts, 0)
             k.silu_mul(act, both)
@@ -118,6 +144,9 @@ class Experts(Part):
             k.expert_linear(act, x, token_of, self.up.tensor.view(e, self.inter, self.hidden), starts, self.act)
         y = ctx.empty(t * top, self.hidden)
         k.expert_linear(y, act, None, self.down.tensor.view(e, self.hidden, self.inter), starts, 0)
+        if self.weight_in:                                               # the outputs are added as they are
+            rows = PairRows(ctx, y, place, t)
+            return rows if pairs else rows.combined()
         shared = None
         if self.shared_up is not None and self.shared_gated:
             hs = ctx.empty(t, self.shared_inter)

@@ -16,6 +16,11 @@ A layer without a down-projection of its own (`own_latent=False`) reads the cach
 run order says which) with its own W_uk, W_uv, queries, gate and output product.
 
 The first products (q, gate, down-projection) are one merged product; the rotation table is the position part's.
+
+Options that other designs use: `q_rank` (queries come from a latent of their own: q = W_uq RMSnorm(W_dq x), stored as dq,
+dq.norm, uq; W_dq takes q's place in the merged product), `gate=False` (no output gate, no g), `sink` (one learned number per
+head, stored as `sink`: exp(sink) stands in the softmax's denominator, without key or value and without the score scale),
+`window` W > 0 (a query at position p sees only keys with p − j < W).
 """
 from __future__ import annotations
 
@@ -29,14 +34,23 @@ from .linear import Linear
 class LatentAttention(Part):
     def __init__(self, ctx: BuildContext, *, heads: int, dim: int, rot_dim: int, vdim: int, rank: int, scale: float,
                  hidden: int, norm: PartRef, position: PartRef | None, own_latent: bool = True, window: int = 0,
-                 layer: int = 0) -> None:
+                 q_rank: int | None = None, gate: bool = True, sink: bool = False, layer: int = 0) -> None:
         super().__init__()
         self.ctx, self.heads, self.dim, self.rot_dim, self.vdim, self.rank = ctx, heads, dim, rot_dim, vdim, rank
         self.scale, self.own_latent, self.window = float(scale), bool(own_latent), int(window)
-        pieces = {"q": heads * (dim + rot_dim), "g": heads * vdim}
+        self.q_rank, self.gate = q_rank, bool(gate)
+        self.n_q = heads * (dim + rot_dim) if q_rank is None else q_rank          # columns of the first product ahead of the gate's
+        pieces = {"q": self.n_q} if q_rank is None else {"dq": q_rank}
+        if gate:
+            pieces["g"] = heads * vdim
         if own_latent:
             pieces["dkv"] = rank + rot_dim
         self.first = self.add_child("first", Linear(ctx, "weight", hidden, pieces))
+        self.q_norm = self.uq = None
+        if q_rank is not None:
+            self.q_norm = self.add_child("q_norm", ctx.part(norm, dim=q_rank))
+            self.uq = self.add_child("up_q", Linear(ctx, "weight", q_rank, {"uq": heads * (dim + rot_dim)}))
+        self.sink = self.add_param("sink", (heads,), "coef") if sink else None
         self.uk = self.add_param("uk", (heads * dim, rank), "matrix")
         self.uv = self.add_param("uv", (heads * vdim, rank), "matrix")
         self.out = self.add_child("out", Linear(ctx, "weight", heads * vdim, {"o": hidden}))
@@ -45,10 +59,10 @@ class LatentAttention(Part):
         self.uk_t = None                    # [heads, rank, dim]: W_uk per head, transposed (made in finalize)
 
     def loadables(self, prefix: str = ""):
-        """Stored names: q, g, dkv, dkv.norm, uk, uv, o."""
-        rename = {prefix + "latent_norm.weight": prefix + "dkv.norm"}
+        """Stored names: q (or dq, dq.norm, uq), g, dkv, dkv.norm, uk, uv, sink, o."""
+        rename = {prefix + "latent_norm.weight": prefix + "dkv.norm", prefix + "q_norm.weight": prefix + "dq.norm"}
         for name, p, rows in super().loadables(prefix):
-            for child in ("first.", "out."):
+            for child in ("first.", "up_q.", "out."):
                 if name.startswith(prefix + child):
                     name = prefix + name[len(prefix + child):]
             yield rename.get(name, name), p, rows
@@ -76,20 +90,32 @@ class LatentAttention(Part):
         t, k, ctx = x.shape[0], self.ctx.kernels, self.ctx
         heads, dim, rot, rank, vdim = self.heads, self.dim, self.rot_dim, self.rank, self.vdim
         fills = cache.fills and self.own_latent
-        first = self.first.forward(x)                                   # [t, q | g | dkv]
-        n_q, n_g = heads * (dim + rot), heads * vdim
+        first = self.first.forward(x)                                   # [t, q or dq | g | dkv]
+        n_q, n_g = self.n_q, heads * vdim if self.gate else 0
         pos = self.position
         qa = ctx.empty(t, heads, rank + rot)                             # the folded queries [a_h | q_h^r]
-        k.latent_prepare(qa, first, heads, dim, rot, rank, n_q + n_g if fills else -1, step.positions,
-                         pos.table if pos else None, pos.rotary_dim if pos else 0,
-                         self.latent_norm.weight.tensor if fills else None, self.latent_norm.eps if fills else 0.0,
-                         cache.kv if fills else None, cache.group.write_index if fills else None)
-        q_u = first[:, :n_q].view(t, heads, dim + rot)[:, :, :dim]
+        turn = (step.positions, pos.table if pos else None, pos.rotary_dim if pos else 0)
+        neighbours = {"interleaved": True} if pos is not None and pos.interleaved else {}
+        row = (self.latent_norm.weight.tensor, self.latent_norm.eps, cache.kv, cache.group.write_index) if fills \
+            else (None, self.q_norm.eps if self.q_norm else 0.0, None, None)
+        at = n_q + n_g if fills else -1
+        if self.uq is None:
+            q = first
+            k.latent_prepare(qa, first, heads, dim, rot, rank, at, *turn, *row, **neighbours)
+        else:                                                            # cache row and query latent, then the queries' rotation
+            cq = ctx.empty(t, self.q_rank)
+            k.latent_prepare(None, first, heads, dim, rot, rank, at, *turn, *row, cq=cq, cq_at=0,
+                             cq_weight=self.q_norm.weight.tensor, **neighbours)
+            q = self.uq.forward(cq)
+            k.latent_prepare(qa, q, heads, dim, rot, rank, -1, *turn, None, 0.0, None, None, **neighbours)
+        q_u = q[:, :heads * (dim + rot)].view(t, heads, dim + rot)[:, :, :dim]
         k.linear_heads(qa[:, :, :rank], q_u, self.uk_t)                   # a_h = W_uk,hᵀ q_h^u
         mix = ctx.empty(t, heads, rank)
-        k.latent_attention(mix, qa, cache.kv, cache.group.block_table, step.rows, self.scale, rank, self.window)
+        sinks = {"sinks": self.sink.tensor} if self.sink is not None else {}
+        k.latent_attention(mix, qa, cache.kv, cache.group.block_table, step.rows, self.scale, rank, self.window, **sinks)
         o = ctx.empty(t, heads, vdim)
         k.linear_heads(o, mix, self.uv.tensor.view(heads, vdim, rank))    # W_uv,h on the weighted sum of latents
-        o = o.view(t, n_g)
-        k.sigmoid_gate(o, first[:, n_q:n_q + n_g])
+        o = o.view(t, heads * vdim)
+        if self.gate:
+            k.sigmoid_gate(o, first[:, n_q:n_q + n_g])
         return self.out.forward(o)

@@ -1,12 +1,14 @@
 """RMSNorm: x · rsqrt(mean(x²) + eps) · (weight + offset), all in 32-bit, one rounding at the end
 (std/holon_std/ops/units.py:16-35; formula std/holon_std/ops/reference.py:7-18).
 
+LayerNorm: (x − mean) / sqrt(variance + eps) · weight without a bias, the variance the mean of the squared deviations.
+
 DynamicTanh: tanh(alpha · x) · weight + bias, no statistics of the row at all."""
 from __future__ import annotations
 
 import torch
 
-from .base import BuildContext, Part, Residual
+from .base import BuildContext, PairRows, Part, Residual
 
 
 class RMSNorm(Part):
@@ -26,6 +28,7 @@ class RMSNorm(Part):
         has done both, the rows it left (base.Scaled)."""
         if getattr(stream, "delta_by", None) is not None:
             raise RuntimeError("rmsnorm: the pending output must pass a norm of its own first; this norm adds it as it is")
+        stream.settled(self)
         if stream.normed is not None:
             rows, by, stream.normed, stream.normed_by = stream.normed, stream.normed_by, None, None
             if by is self:
@@ -40,6 +43,45 @@ class RMSNorm(Part):
         out = self.ctx.empty(index.shape[0], self.dim)
         self.ctx.kernels.add_rmsnorm(out, stream.h, stream.delta, self.weight.tensor, self.eps, self.offset, index)
         return out
+
+
+class LayerNorm(Part):
+    """`takes_pairs`: a pending output may still be rows of (token, choice) pairs (base.PairRows) and may carry a factor
+    (`Residual.delta_scale`); the kernel that norms the sum does both."""
+
+    takes_pairs = True
+    links = False                            # its statistics need the whole row: no product leaves its rows behind (base.Link)
+
+    def __init__(self, ctx: BuildContext, *, eps: float, dim: int) -> None:
+        super().__init__()
+        self.ctx, self.eps, self.dim = ctx, float(eps), dim
+        self.weight = self.add_param("weight", (dim,), "gain")
+
+    def apply(self, x: torch.Tensor) -> torch.Tensor:
+        """The norm of the rows of `x` [rows, dim] (engine dtype or 32-bit), as a new tensor of the engine's dtype."""
+        out = self.ctx.empty(*x.shape)
+        self.ctx.kernels.add_layernorm(out, x, None, 1.0, self.weight.tensor, self.eps, None)
+        return out
+
+    def _run(self, stream: Residual, index) -> torch.Tensor:
+        if getattr(stream, "delta_by", None) is not None:
+            raise RuntimeError("layernorm: the pending output must pass a norm of its own first; this norm adds it as it is")
+        delta = stream.delta
+        y, place = (delta.y, delta.place) if isinstance(delta, PairRows) else (delta, None)
+        out = self.ctx.empty(index.shape[0] if index is not None else stream.h.shape[0], self.dim)
+        self.ctx.kernels.add_layernorm(out, stream.h, y, stream.delta_scale, self.weight.tensor, self.eps, index, place=place)
+        return out
+
+    def add(self, stream: Residual) -> torch.Tensor:
+        """Adds the stream's pending output into it and returns the norm of the sum."""
+        stream.normed = stream.normed_by = None
+        out = self._run(stream, None)
+        stream.delta, stream.delta_scale = None, 1.0
+        return out
+
+    def gather(self, stream: Residual, index: torch.Tensor) -> torch.Tensor:
+        """The norm of rows `index` of the stream (pending output included); the stream is left as it is."""
+        return self._run(stream, index)
 
 
 class DynamicTanh(Part):

@@ -32,6 +32,10 @@ times one number c per head and token, the removal term is k_i Â· a_i cÂ² Â· (ká
 channel beside k itself (`recurrent_scan(rate=)`). Each head's o is divided by its root mean square, times a weight over
 all heads' channels, times sigmoid(W_g x), then W_o.
 
+`Lightning`: linear attention with one fixed decay per head and nothing else in the recurrence: q, k, v = silu of their
+projections, no rotation, no scale, o = Sáµ€ q; all heads' o together under one RMS norm with a weight over all their channels,
+times sigmoid(W_g x), then W_o.
+
 Everything that enters the recurrence is 32-bit (the scan's inputs are made in 32-bit from the first product's rows);
 the products themselves are the engine's. All first projections of a mixer are one merged product.
 """
@@ -99,6 +103,42 @@ class Retention(_MatrixState):
         at = 2 * heads * dim + heads * vdim
         k.head_norm_gate(y, o, None, None, first[:, at:at + heads * vdim], self.eps)
         return self.out.forward(y.view(t, heads * vdim))
+
+
+class Lightning(_MatrixState):
+    def __init__(self, ctx: BuildContext, *, heads: int, dim: int, vdim: int, decay: tuple[float, ...], eps: float,
+                 hidden: int, layer: int = 0) -> None:
+        super().__init__()
+        if len(decay) != heads:
+            raise ValueError(f"lightning: {len(decay)} decays for {heads} heads")
+        self.ctx, self.heads, self.dim, self.vdim, self.eps = ctx, heads, dim, vdim, float(eps)
+        self.decay = tuple(float(d) for d in decay)
+        self.first = self.add_child("first", Linear(ctx, "weight", hidden, {
+            "q": heads * dim, "k": heads * dim, "v": heads * vdim, "g": heads * vdim}))
+        self.gain = self.add_param("norm", (heads * vdim,), "coef")
+        self.out = self.add_child("out", Linear(ctx, "weight", heads * vdim, {"o": hidden}))
+        self._decay = None
+
+    def finalize(self) -> None:
+        super().finalize()
+        if self.first.weight.tensor is not None:
+            self._decay = torch.tensor(self.decay, dtype=torch.float32, device=self.first.weight.tensor.device)
+
+    def slot_states(self):
+        return (SlotState("state", (self.heads, self.vdim, self.dim)),)
+
+    def forward(self, x: torch.Tensor, step, cache) -> torch.Tensor:
+        t, k, ctx, heads, dim, vdim = x.shape[0], self.ctx.kernels, self.ctx, self.heads, self.dim, self.vdim
+        first = self.first.forward(x)                                    # [t, q | k | v | g]
+        qk = ctx.empty(t, 2, heads, dim, dtype=torch.float32)
+        v = ctx.empty(t, heads, vdim, dtype=torch.float32)
+        k.retention_prepare(qk, v, first, step.positions, None, 0, 1.0, silu=True)
+        o = ctx.empty(t, heads, vdim, dtype=torch.float32)
+        k.recurrent_scan(o, qk, v, None, self._decay, None, cache.slots["state"], step.rows)
+        n, at = heads * vdim, 2 * heads * dim + heads * vdim
+        y = ctx.empty(t, 1, n)                                           # (one norm over all heads: a single head of their width)
+        k.head_norm_gate(y, o.view(t, 1, n), self.gain.tensor, None, first[:, at:at + n], self.eps, gate="sigmoid")
+        return self.out.forward(y.view(t, n))
 
 
 class GatedDelta(_MatrixState):

@@ -39,6 +39,21 @@ class RefKernels:
             h.copy_(v)
         self.rmsnorm(out, v, weight, eps, offset)
 
+    def add_layernorm(self, out, h, delta, scale, weight, eps, index, place=None):
+        v = h.float()
+        if delta is not None:
+            d = delta.float() if place is None else delta.float()[place.long()].view(h.shape[0], -1, h.shape[1]).sum(1)
+            v = v + scale * d
+            if index is None:
+                h.copy_(v)
+        if index is not None:
+            v = v[index.long()]
+        d = v - v.mean(-1, keepdim=True)
+        out.copy_((d * torch.rsqrt((d * d).mean(-1, keepdim=True) + eps) * weight.float()).to(out.dtype))
+
+    def softcap(self, x, cap):
+        x.copy_(cap * torch.tanh(x / cap))
+
     def qk_norm_rope_kv_write(self, q_out, qkv, positions, table, rotary_dim, q_weight, k_weight, eps, offset, kv,
                               write_index, heads, kv_heads, head_dim, bias=None):
         t, dt = qkv.shape[0], qkv.dtype
@@ -130,8 +145,14 @@ class RefKernels:
         self.sum_into(h, terms, bias)
         self.rmsnorm(out, h, weight, eps, offset)
 
-    def glu_clamped(self, out, gate_up, bias, limit, alpha):
-        z = gate_up.float() + (bias.float() if bias is not None else 0.0)
+    def expert_glu(self, out, x, token_of, w, starts, limit, alpha, row_scale):
+        both = torch.empty(out.shape[0], w.shape[1], dtype=out.dtype)
+        self.expert_linear(both, x, token_of, w, starts, 0)
+        self.glu_clamped(out, both, None, limit, alpha, row_scale=row_scale)
+
+    def glu_clamped(self, out, gate_up, bias, limit, alpha, row_scale=None):
+        z = gate_up.float() * (row_scale[:, None] if row_scale is not None else 1.0)
+        z = z + (bias.float() if bias is not None else 0.0)
         g, u = z.chunk(2, dim=-1)
         g, u = g.clamp(max=limit), u.clamp(-limit, limit)
         out.copy_((g * torch.sigmoid(alpha * g) * (u + 1)).to(out.dtype))
@@ -189,10 +210,12 @@ class RefKernels:
             seq = torch.cat((conv_state[slots[b]], first[qs[b]:qs[b + 1], :channels]), 0)
             conv_state[slots[b]] = seq[-(taps - 1):]
 
-    def retention_prepare(self, qk, v, first, positions, table, rot_dims, k_scale):
+    def retention_prepare(self, qk, v, first, positions, table, rot_dims, k_scale, silu=False):
         t, heads, vdim = v.shape
         dim = qk.shape[3]
         x = first.float()
+        if silu:
+            x = x * torch.sigmoid(x)
         for which in (0, 1):
             z = x[:, which * heads * dim:(which + 1) * heads * dim].view(t, heads, dim)
             if rot_dims:
@@ -277,27 +300,36 @@ class RefKernels:
         self.rmsnorm(out, u, weight, eps, offset)
 
     @staticmethod
-    def _turn(x, cs, dims):
+    def _turn(x, cs, dims, interleaved=False):
         half = dims // 2
         cos, sin = cs[..., :half], cs[..., half:]
+        if interleaved:
+            x = x.clone()
+            a, b = x[..., 0:dims:2].clone(), x[..., 1:dims:2].clone()
+            x[..., 0:dims:2], x[..., 1:dims:2] = a * cos - b * sin, b * cos + a * sin
+            return x
         a, b, rest = x[..., :half], x[..., half:dims], x[..., dims:]
         return torch.cat((a * cos - b * sin, b * cos + a * sin, rest), dim=-1)
 
     def latent_prepare(self, qa, first, heads, dim, rot, rank, dkv_at, positions, table, rot_dims, norm_weight, eps,
-                       cache, write_index):
+                       cache, write_index, interleaved=False, cq=None, cq_at=0, cq_weight=None):
         t, dt = first.shape[0], first.dtype
         cs = table[positions.long()] if rot_dims else None
-        q_r = first[:, :heads * (dim + rot)].view(t, heads, dim + rot)[:, :, dim:].float()
-        if rot_dims:
-            q_r = self._turn(q_r, cs[:, None, :], rot_dims)
-        qa[:, :, rank:] = q_r.to(dt)
+        if qa is not None:
+            q_r = first[:, :heads * (dim + rot)].view(t, heads, dim + rot)[:, :, dim:].float()
+            if rot_dims:
+                q_r = self._turn(q_r, cs[:, None, :], rot_dims, interleaved)
+            qa[:, :, rank:] = q_r.to(dt)
+        if cq is not None:
+            z = first[:, cq_at:cq_at + cq.shape[1]].float()
+            cq.copy_((z * torch.rsqrt((z * z).mean(-1, keepdim=True) + eps) * cq_weight.float()).to(dt))
         if dkv_at >= 0:
             d = first[:, dkv_at:dkv_at + rank + rot].float()
             c = d[:, :rank]
             c = c * torch.rsqrt((c * c).mean(-1, keepdim=True) + eps) * norm_weight.float()
             k_r = d[:, rank:]
             if rot_dims:
-                k_r = self._turn(k_r, cs, rot_dims)
+                k_r = self._turn(k_r, cs, rot_dims, interleaved)
             w = write_index.long()
             ok = w >= 0
             cache.view(-1, rank + rot)[w[ok]] = torch.cat((c, k_r), dim=-1).to(dt)[ok]
@@ -305,7 +337,7 @@ class RefKernels:
     def linear_heads(self, out, x, w):
         out.copy_(torch.einsum("tbk,bnk->tbn", x.float(), w.float()).to(out.dtype))
 
-    def latent_attention(self, out, qa, cache, block_table, rows, scale, rank, window):
+    def latent_attention(self, out, qa, cache, block_table, rows, scale, rank, window, sinks=None):
         page_size = cache.shape[1]
         out.zero_()
         qs, slots, lens = rows.query_start.tolist(), rows.row_slot.tolist(), rows.kv_len.tolist()
@@ -321,16 +353,19 @@ class RefKernels:
             hidden = key > pos
             if window > 0:
                 hidden = hidden | (pos - key >= window)
-            probs = scores.masked_fill(hidden, float("-inf")).softmax(-1)
+            scores = scores.masked_fill(hidden, float("-inf"))
+            if sinks is not None:
+                scores = torch.cat((scores, sinks.float()[:, None, None].expand(-1, e - s, 1)), -1)
+            probs = scores.softmax(-1)[..., :n]
             out[s:e] = torch.einsum("hqk,kd->qhd", probs, kc[:, :rank]).to(out.dtype)
 
     def sigmoid_gate(self, o, g):
         o.copy_((o.float() * torch.sigmoid(g.float())).to(o.dtype))
 
     def route_top(self, chosen, weight, counts, z, experts, scale, renormalize, bias=None, correction=None, groups=1,
-                  keep=1, tiny=0.0):
+                  keep=1, tiny=0.0, scores="softmax"):
         z = z[:, :experts].float() + (bias.float() if bias is not None else 0.0)
-        s = torch.softmax(z, dim=-1)
+        s = torch.softmax(z, dim=-1) if scores == "softmax" else torch.sigmoid(z)
         top = chosen.shape[1]
         choice = s + correction.float() if correction is not None else s.clone()
         if groups > 1:                                         # only experts of the best groups stay in the running
@@ -347,10 +382,12 @@ class RefKernels:
         counts[:experts] += torch.bincount(order.reshape(-1), minlength=experts).to(torch.int32)
 
     def route_rows(self, chosen, weight, counts, place, token_of, z, experts, scale, renormalize, bias=None,
-                   correction=None, groups=1, keep=1, tiny=0.0):
+                   correction=None, groups=1, keep=1, tiny=0.0, scores="softmax", row_weight=None):
         counts.zero_()
-        self.route_top(chosen, weight, counts, z, experts, scale, renormalize, bias, correction, groups, keep, tiny)
+        self.route_top(chosen, weight, counts, z, experts, scale, renormalize, bias, correction, groups, keep, tiny, scores)
         self.expert_rows(place, token_of, counts, chosen, experts)
+        if row_weight is not None:
+            row_weight[place.long()] = weight.reshape(-1)
         counts[2 * experts + 1], counts[2 * experts + 2] = 0, chosen.shape[0]
 
     def expert_rows(self, place, token_of, counts, chosen, experts):
@@ -391,14 +428,15 @@ class RefKernels:
         x.copy_(self._act(x.float(), act, numbers).to(x.dtype))
 
     def expert_combine(self, out, y, place, weight, shared, z, experts, x=None, identity_from=None):
-        t, top = weight.shape
+        t = out.shape[0]
+        top = place.shape[0] // t
         acc = torch.zeros(out.shape, dtype=torch.float32)
         for k in range(top):
             rows = place.view(t, top)[:, k].long()
             term = y[rows].float()
             if x is not None:                                  # rows of identity experts: the token's input itself
                 term = torch.where((rows >= int(identity_from[0]))[:, None], x.float(), term)
-            acc += weight[:, k:k + 1] * term
+            acc += (weight[:, k:k + 1] if weight is not None else 1.0) * term
         if shared is not None:
             acc += (torch.sigmoid(z[:, experts:experts + 1].float()) if z is not None else 1.0) * shared.float()
         out.copy_(acc.to(out.dtype))
