@@ -208,6 +208,15 @@ int hb_expert_linear_tcgen05_tiles(int rows, int experts);
 int hb_expert_linear_tcgen05(void* out, const void* x, const int32_t* token_of, void* gathered, const void* w,
                              const int32_t* starts, int32_t* table, int rows, int experts, int n, int k, int act,
                              hb_stream stream);
+// The clamped gated unit in the products' epilogues: out [rows, inter] = g sigmoid(alpha g) (u + 1) with g = min(f gate, limit),
+// u = clamp(f up, -limit, limit), f = row_scale[row] (null: 1), gate and up the row's products with an expert's first and last
+// inter rows of w [experts, 2 inter, k]; bfloat16. _few: on CUDA cores for a row or two an expert (k a multiple of 8);
+// _tcgen05: for prompts, inter a multiple of 8, scratch as hb_expert_linear_tcgen05.
+int hb_expert_glu_few(void* out, const void* x, const int32_t* token_of, const void* w, const int32_t* starts,
+                      const float* row_scale, float limit, float alpha, int rows, int experts, int inter, int k, hb_stream stream);
+int hb_expert_glu_tcgen05(void* out, const void* x, const int32_t* token_of, void* gathered, const void* w,
+                          const int32_t* starts, int32_t* table, const float* row_scale, float limit, float alpha, int rows,
+                          int experts, int inter, int k, hb_stream stream);
 int hb_experts_tcgen05_status(unsigned int* status);
 // x = act(x) in place (act as above, 3 the tanh form of gelu, 4 xielu with the two numbers `numbers`, 5 tanh);
 // o [tokens, n] *= sigmoid(g[t * ld + i]).
@@ -399,14 +408,15 @@ int hb_gdelta_prepare(float* qk, float* v, float* decay, float* rate, const void
 // unit vectors per head (eps unit_eps), q times q_scale; beta = sigmoid(b); decay = exp(-exp(rate_log[h])
 // softplus(low2[:, :heads dim] + dt_bias)) [tokens, heads, dim]; gate = sigmoid(low2[:, heads dim:]) [tokens, heads vdim].
 int hb_delta_prepare(float* qk, float* v, float* beta, float* decay, float* gate, const void* first, int dtype, int ld,
-                     const void* conv, int taps, const void* conv_state, const float* low2, const float* dt_bias,
+                     const void* conv, int taps, void* conv_state, const float* low2, const float* dt_bias,
                      const float* rate_log, const int32_t* query_start, const int32_t* row_slot, int rows, int tokens,
-                     int heads, int kv_heads, int dim, int vdim, float q_scale, float unit_eps, hb_stream stream);
-// conv_state <- the last taps - 1 inputs of each row (what was carried, then the step's tokens). After hb_delta_prepare.
+                     int heads, int kv_heads, int dim, int vdim, float q_scale, float unit_eps, int carry, hb_stream stream);
+// conv_state <- the last taps - 1 inputs of each row (what was carried, then the step's tokens), of rows of at least `least`
+// tokens. After hb_delta_prepare, which with `carry` has done it for rows of one token itself.
 int hb_conv_carry(void* conv_state, const void* first, int dtype, int ld, int channels, int taps,
-                  const int32_t* query_start, const int32_t* row_slot, int rows, hb_stream stream);
+                  const int32_t* query_start, const int32_t* row_slot, int rows, int least, hb_stream stream);
 // A retention mixer's first product, rows [q (heads dim) | k (heads dim) | v (heads vdim) | ...]: q and k turned by the
-// position (as hb_qk_norm_rope_kv_write turns them), k times k_scale, all to 32-bit.
+// position (as hb_qk_norm_rope_kv_write turns them), k times k_scale, all to 32-bit; with `silu` every number passes silu first.
 int hb_retention_prepare(float* qk, float* v, const void* first, int dtype, int ld, const int32_t* positions,
                          const float* table, int rot_dims, int max_positions, int tokens, int heads, int dim, int vdim,
                          float k_scale, int silu, hb_stream stream);

@@ -761,14 +761,19 @@ __global__ void __launch_bounds__(BM == 128 ? 256 : 128) expert_linear_bf16_kern
 // are on their way: a CTA of eight warps keeps the tile's rows of x in shared memory and takes 32 weight rows, four a
 // warp; a lane reads 16 bytes of each of them per step of 256 columns (two steps in flight) and multiplies on the CUDA
 // cores in 32-bit; the lanes' sums meet by shuffles. No tensor cores: with one or two rows they would idle anyway.
+// GLU: w [experts, 2 n, k] holds an expert's n gate rows, then its n up rows; a warp takes two gate rows and the two up rows
+// beside them, and the epilogue is the clamped unit: with f = row_scale[row] (null: 1), g = min(f gate, limit),
+// u = clamp(f up, -limit, limit), out [rows, n] = g sigmoid(alpha g) (u + 1).
 #define XF_ROWS 8
 #define XF_WROWS 4
 
+template <bool GLU>
 __global__ void __launch_bounds__(256) expert_linear_few_kernel(bf16* __restrict__ out, const bf16* __restrict__ x,
                                                                 const int32_t* __restrict__ token_of,
                                                                 const bf16* __restrict__ w,
                                                                 const int32_t* __restrict__ starts, int experts, int n,
-                                                                int k, int act) {
+                                                                int k, int act, const float* __restrict__ row_scale,
+                                                                float limit, float alpha) {
     extern __shared__ __align__(16) unsigned char xf_smem[];
     bf16* xs = (bf16*)xf_smem;                              // [XF_ROWS][k]
     __shared__ int tile_info[3];
@@ -784,9 +789,10 @@ __global__ void __launch_bounds__(256) expert_linear_few_kernel(bf16* __restrict
         *(uint4*)(xs + (size_t)r * k + col) = __ldg((const uint4*)(x + (size_t)src * k + col));
     }
     __syncthreads();
-    const int nr = blockIdx.x * 32 + warp * XF_WROWS;       // this warp's first weight row
+    constexpr int COLS = GLU ? XF_WROWS / 2 : XF_WROWS;     // output columns a warp
+    const int nr = (blockIdx.x * 8 + warp) * COLS;          // this warp's first output column: weight row nr (and, GLU, n + nr)
     if (nr >= n) return;
-    const bf16* we = w + (size_t)e * n * k;
+    const bf16* we = w + (size_t)e * (GLU ? 2 : 1) * n * k;
     float acc[XF_WROWS][XF_ROWS];
 #pragma unroll
     for (int j = 0; j < XF_WROWS; ++j)
@@ -797,7 +803,7 @@ __global__ void __launch_bounds__(256) expert_linear_few_kernel(bf16* __restrict
         uint4 wv[XF_WROWS];
 #pragma unroll
         for (int j = 0; j < XF_WROWS; ++j)
-            wv[j] = nr + j < n ? __ldg((const uint4*)(we + (size_t)(nr + j) * k + kc)) : make_uint4(0u, 0u, 0u, 0u);
+            wv[j] = nr + j % COLS < n ? __ldg((const uint4*)(we + (size_t)(nr + j % COLS + (j / COLS) * n) * k + kc)) : make_uint4(0u, 0u, 0u, 0u);
         float wf[XF_WROWS][8];
 #pragma unroll
         for (int j = 0; j < XF_WROWS; ++j) {
@@ -823,6 +829,15 @@ __global__ void __launch_bounds__(256) expert_linear_few_kernel(bf16* __restrict
 #pragma unroll
     for (int r = 0; r < XF_ROWS; ++r) {
         if (r < nrows) {
+            if constexpr (GLU) {
+                const float f = row_scale ? row_scale[m0 + r] : 1.f;
+#pragma unroll
+                for (int j = 0; j < COLS; ++j) {
+                    const float g = fminf(f * warp_sum(acc[j][r]), limit), u = fminf(fmaxf(f * warp_sum(acc[j + COLS][r]), -limit), limit);
+                    if (lane == 0 && nr + j < n) out[(size_t)(m0 + r) * n + nr + j] = __float2bfloat16_rn(g / (1.f + expf(-alpha * g)) * (u + 1.f));
+                }
+                continue;
+            }
 #pragma unroll
             for (int j = 0; j < XF_WROWS; ++j) {
                 const float v = warp_sum(acc[j][r]);
@@ -849,9 +864,9 @@ extern "C" int hb_expert_linear_bf16(void* out, const void* x, const int32_t* to
     cudaStream_t s = (cudaStream_t)stream;
     if (bm == 8) {
         const size_t smem = (size_t)XF_ROWS * k * sizeof(bf16);
-        if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(expert_linear_few_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(expert_linear_few_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         dim3 few((n + 31) / 32, (unsigned)tiles);
-        expert_linear_few_kernel<<<few, 256, smem, s>>>((bf16*)out, (const bf16*)x, token_of, (const bf16*)w, starts, experts, n, k, act);
+        expert_linear_few_kernel<false><<<few, 256, smem, s>>>((bf16*)out, (const bf16*)x, token_of, (const bf16*)w, starts, experts, n, k, act, nullptr, 0.f, 0.f);
         HB_LAUNCH_CHECK("expert_linear_few");
         return 0;
     }
@@ -863,5 +878,22 @@ extern "C" int hb_expert_linear_bf16(void* out, const void* x, const int32_t* to
     if (bm == 16) XB_GO(16, 128); else if (bm == 64) XB_GO(64, 128); else XB_GO(128, 256);
 #undef XB_GO
     HB_LAUNCH_CHECK("expert_linear_bf16");
+    return 0;
+}
+
+// The clamped gated unit's first half for a row or two an expert: out [rows, inter] from w [experts, 2 inter, k] in one kernel.
+extern "C" int hb_expert_glu_few(void* out, const void* x, const int32_t* token_of, const void* w, const int32_t* starts,
+                                 const float* row_scale, float limit, float alpha, int rows, int experts, int inter, int k,
+                                 hb_stream stream) {
+    if (rows == 0 || inter == 0) return 0;
+    const size_t smem = (size_t)XF_ROWS * k * sizeof(bf16);
+    if (k <= 0 || k % 8 || experts < 1 || smem > 200 * 1024) HB_REFUSE("expert_glu_few: k = %d must be a multiple of 8 of at most 12800", k);
+    if (((uintptr_t)x | (uintptr_t)w) % 16) HB_REFUSE("expert_glu_few: pointers must be 16-byte aligned");
+    const long tiles = (rows + XF_ROWS - 1) / XF_ROWS + (experts < rows ? experts : rows);
+    if (tiles > 65535) HB_REFUSE("expert_glu_few: %d rows over %d experts are above the kernel's limit", rows, experts);
+    if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(expert_linear_few_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    expert_linear_few_kernel<true><<<dim3((inter + 15) / 16, (unsigned)tiles), 256, smem, (cudaStream_t)stream>>>(
+        (bf16*)out, (const bf16*)x, token_of, (const bf16*)w, starts, experts, inter, k, 0, row_scale, limit, alpha);
+    HB_LAUNCH_CHECK("expert_glu_few");
     return 0;
 }

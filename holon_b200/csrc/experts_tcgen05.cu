@@ -7,6 +7,8 @@
 // end, where TMA fills zeros): those rows and columns are computed and not stored. Which tiles there are is only known
 // on the device: a small kernel lists them (expert, first row, the expert's end), the product launches persistent
 // CTAs over the most tiles any split of the rows can have, and every role stops at the first tile the list leaves empty.
+// GLU (hb_expert_glu_tcgen05): an expert's weight is its gate rows, then its up rows; a tile's two weight boxes are 128 gate
+// rows and the 128 up rows beside them, so the accumulator's halves meet in the epilogue, which is the clamped gated unit.
 // Every wait is bounded as in the other tcgen05 kernels (status word: hb_experts_tcgen05_status).
 #include "tcgen05.cuh"
 
@@ -53,10 +55,18 @@ __device__ __forceinline__ float xt_act(float v, int act) {
     return v;
 }
 
+// What the epilogue of the gated form needs: a factor per row (null: 1), then g = min(f gate, limit), u = clamp(f up, +-limit),
+// g sigmoid(alpha g) (u + 1).
+struct XtGlu {
+    const float* row_scale;
+    float limit, alpha;
+};
+
+template <bool GLU>
 __global__ void __launch_bounds__(192, 1) expert_linear_tcgen05_kernel(const __grid_constant__ CUtensorMap map_x,
                                                                        const __grid_constant__ CUtensorMap map_w,
                                                                        bf16* __restrict__ out, const int32_t* __restrict__ table,
-                                                                       int n, int k, int act, int tiles_m, int tiles_n) {
+                                                                       int n, int k, int act, int tiles_m, int tiles_n, XtGlu glu) {
     extern __shared__ unsigned char smem_raw[];
     const uint32_t base = (smem_addr(smem_raw) + 1023u) & ~1023u;
     const uint32_t bars = base + XT_STAGES * XT_STAGE_BYTES;
@@ -91,7 +101,7 @@ __global__ void __launch_bounds__(192, 1) expert_linear_tcgen05_kernel(const __g
                 const int e = table[3 * mt];
                 if (e < 0) break;                                     // (the list's tiles are its first entries)
                 const int m0 = table[3 * mt + 1];
-                const int w0 = e * n + nt * XT_BN, w1 = w0 + 128;
+                const int w0 = GLU ? 2 * e * n + nt * 128 : e * n + nt * XT_BN, w1 = w0 + (GLU ? n : 128);   // (GLU: n is the unit's size)
                 bool ok = true;
                 for (int kb = 0; kb < kblocks && ok; ++kb, ++kb_all) {
                     const int s = kb_all % XT_STAGES;
@@ -141,17 +151,30 @@ __global__ void __launch_bounds__(192, 1) expert_linear_tcgen05_kernel(const __g
             if (table[3 * mt] < 0) break;
             const int acc = local & 1, use = local >> 1;
             const int row = table[3 * mt + 1] + q * 32 + lane, row_end = table[3 * mt + 2];
-            const int col0 = nt * XT_BN;
+            const int col0 = nt * (GLU ? 128 : XT_BN);
             if (!mbar_wait(acc_full0 + 8 * acc, use & 1, 3)) break;
             tc_fence_after();
             const uint32_t d = tmem + acc * XT_BN + ((uint32_t)(q * 32) << 16);
-            for (int c = 0; c < 8; ++c) {
+            const float f = GLU && glu.row_scale && row < row_end ? glu.row_scale[row] : 1.f;
+            constexpr int CHUNKS = GLU ? 4 : 8;
+            for (int c = 0; c < CHUNKS; ++c) {
                 uint32_t r[32];
                 tc_ld32(d + c * 32, r);
                 float v[32];
+                if constexpr (GLU) {
+                    uint32_t r2[32];
+                    tc_ld32(d + 128 + c * 32, r2);
 #pragma unroll
-                for (int i = 0; i < 32; ++i) v[i] = xt_act(__uint_as_float(r[i]), act);
-                if (c == 7) {                                         // everything is in registers: hand the accumulator back
+                    for (int i = 0; i < 32; ++i) {
+                        const float g = fminf(f * __uint_as_float(r[i]), glu.limit);
+                        const float u = fminf(fmaxf(f * __uint_as_float(r2[i]), -glu.limit), glu.limit);
+                        v[i] = g / (1.f + __expf(-glu.alpha * g)) * (u + 1.f);
+                    }
+                } else {
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) v[i] = xt_act(__uint_as_float(r[i]), act);
+                }
+                if (c == CHUNKS - 1) {                                         // everything is in registers: hand the accumulator back
                     tc_fence_before();
                     __syncwarp();
                     if (lane == 0) mbar_arrive(acc_empty0 + 8 * acc);
@@ -208,12 +231,11 @@ extern "C" int hb_expert_linear_tcgen05_tiles(int rows, int experts) {
     return (rows + XT_BM - 1) / XT_BM + (experts < rows ? experts : rows);
 }
 
-// out [rows, n] = act(x' · w[e]ᵀ) for the rows of expert e (starts [experts + 1]); x' = x gathered by token_of into
-// `gathered` [rows, k] (token_of null: x itself, its rows already expert by expert). table: 3 * hb_expert_linear_tcgen05_tiles
-// (rows, experts) int32 of scratch. bfloat16; k and n multiples of 8; pointers 16-byte aligned.
-extern "C" int hb_expert_linear_tcgen05(void* out, const void* x, const int32_t* token_of, void* gathered, const void* w,
-                                        const int32_t* starts, int32_t* table, int rows, int experts, int n, int k, int act,
-                                        hb_stream stream) {
+// The shared host half: tiles, gathered rows, tensor maps, launch. n: output columns (GLU: the unit's size, an expert's weight
+// having 2 n rows).
+template <bool GLU>
+static int xt_launch(void* out, const void* x, const int32_t* token_of, void* gathered, const void* w, const int32_t* starts,
+                     int32_t* table, int rows, int experts, int n, int k, int act, XtGlu glu, hb_stream stream) {
     if (rows == 0 || n == 0) return 0;
     if (k < 8 || k % 8 || n % 8) HB_REFUSE("expert_linear_tcgen05: k = %d and n = %d must be multiples of 8", k, n);
     if (token_of && !gathered) HB_REFUSE("expert_linear_tcgen05: rows that are gathered need room for the gathered copy");
@@ -221,7 +243,7 @@ extern "C" int hb_expert_linear_tcgen05(void* out, const void* x, const int32_t*
     if ((((uintptr_t)xs | (uintptr_t)x | (uintptr_t)w | (uintptr_t)out) % 16) != 0) HB_REFUSE("expert_linear_tcgen05: pointers must be 16-byte aligned");
     cudaStream_t s = (cudaStream_t)stream;
     const int tiles_m = hb_expert_linear_tcgen05_tiles(rows, experts);
-    const int tiles_n = (n + XT_BN - 1) / XT_BN;
+    const int per = GLU ? 128 : XT_BN, tiles_n = (n + per - 1) / per;
     expert_tiles_kernel<<<1, 32, 0, s>>>(table, starts, experts, tiles_m);
     HB_LAUNCH_CHECK("expert_tiles");
     if (token_of) {
@@ -231,9 +253,9 @@ extern "C" int hb_expert_linear_tcgen05(void* out, const void* x, const int32_t*
     CUtensorMap map_x, map_w;
     int rc = xt_encode_map(&map_x, xs, rows, k);
     if (rc) return rc;
-    rc = xt_encode_map(&map_w, w, (long)experts * n, k);
+    rc = xt_encode_map(&map_w, w, (long)experts * n * (GLU ? 2 : 1), k);
     if (rc) return rc;
-    HB_CUDA(cudaFuncSetAttribute(expert_linear_tcgen05_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, XT_SMEM));
+    HB_CUDA(cudaFuncSetAttribute(expert_linear_tcgen05_kernel<GLU>, cudaFuncAttributeMaxDynamicSharedMemorySize, XT_SMEM));
     static int sms = 0;
     if (sms == 0) {
         int device = 0;
@@ -242,7 +264,23 @@ extern "C" int hb_expert_linear_tcgen05(void* out, const void* x, const int32_t*
     }
     const long tiles = (long)tiles_m * tiles_n;
     const int grid = (int)(tiles < sms ? tiles : sms);
-    expert_linear_tcgen05_kernel<<<grid, 192, XT_SMEM, s>>>(map_x, map_w, (bf16*)out, table, n, k, act, tiles_m, tiles_n);
+    expert_linear_tcgen05_kernel<GLU><<<grid, 192, XT_SMEM, s>>>(map_x, map_w, (bf16*)out, table, n, k, act, tiles_m, tiles_n, glu);
     HB_LAUNCH_CHECK("expert_linear_tcgen05");
     return 0;
+}
+
+// out [rows, n] = act(x' · w[e]ᵀ) for the rows of expert e (starts [experts + 1]); x' = x gathered by token_of into
+// `gathered` [rows, k] (token_of null: x itself, its rows already expert by expert). table: 3 * hb_expert_linear_tcgen05_tiles
+// (rows, experts) int32 of scratch. bfloat16; k and n multiples of 8; pointers 16-byte aligned.
+extern "C" int hb_expert_linear_tcgen05(void* out, const void* x, const int32_t* token_of, void* gathered, const void* w,
+                                        const int32_t* starts, int32_t* table, int rows, int experts, int n, int k, int act,
+                                        hb_stream stream) {
+    return xt_launch<false>(out, x, token_of, gathered, w, starts, table, rows, experts, n, k, act, XtGlu{nullptr, 0.f, 0.f}, stream);
+}
+
+// out [rows, inter]: the clamped gated unit over w [experts, 2 inter, k] (an expert's gate rows, then its up rows).
+extern "C" int hb_expert_glu_tcgen05(void* out, const void* x, const int32_t* token_of, void* gathered, const void* w,
+                                     const int32_t* starts, int32_t* table, const float* row_scale, float limit, float alpha,
+                                     int rows, int experts, int inter, int k, hb_stream stream) {
+    return xt_launch<true>(out, x, token_of, gathered, w, starts, table, rows, experts, inter, k, 0, XtGlu{row_scale, limit, alpha}, stream);
 }

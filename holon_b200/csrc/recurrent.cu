@@ -378,20 +378,23 @@ extern "C" int hb_recurrent_scan(float* out, const float* qk, const float* v, co
 // decay[h, d] = exp(-exp(rate_log[h]) softplus(a[h dim + d] + dt_bias[h dim + d])), gate = sigmoid(g).
 // grid (tokens, segments): the first segments take the q and k heads, a warp a head (the convolution twice: once for the
 // sum of squares, once for the values); the others an element a thread of v, beta, the decays and the gate. No thread
-// waits for another, so a step of a few tokens still spreads over many blocks.
+// waits for another, so a step of a few tokens still spreads over many blocks. `carry`: the carried inputs of a row of ONE
+// token move on here (the thread that owns a channel is the only one that reads them, and it has read them by then); rows of
+// several tokens, whose first tokens' blocks all read them, are left to hb_conv_carry.
 template <typename T>
 __global__ void delta_prepare_kernel(float* __restrict__ qk, float* __restrict__ v, float* __restrict__ beta,
                                      float* __restrict__ decay, float* __restrict__ gate, const T* __restrict__ first,
-                                     int ld, const T* __restrict__ conv, int taps, const T* __restrict__ conv_state,
+                                     int ld, const T* __restrict__ conv, int taps, T* conv_state,
                                      const float* __restrict__ low2, const float* __restrict__ dt_bias,
                                      const float* __restrict__ rate_log, const int32_t* __restrict__ query_start,
                                      const int32_t* __restrict__ row_slot, int rows, int heads, int kv_heads, int dim,
-                                     int vdim, float q_scale, float unit_eps) {
+                                     int vdim, float q_scale, float unit_eps, int carry) {
     const int t = blockIdx.x, seg = blockIdx.y;
     const int b = row_of_token(query_start, rows, t);
     const int t0 = query_start[b];
     const int nq = kv_heads * dim, nv = heads * vdim, C = 2 * nq + nv;
-    const T* st = conv_state ? conv_state + (size_t)row_slot[b] * (taps - 1) * C : nullptr;
+    T* st = conv_state ? conv_state + (size_t)row_slot[b] * (taps - 1) * C : nullptr;
+    const bool moves = carry && st && taps > 1 && query_start[b + 1] - t0 == 1;
     auto channel = [&](int c) -> float {                               // convolution over time and silu of channel c
         float acc = 0.f;
         for (int j = 0; j < taps; ++j) {
@@ -401,6 +404,11 @@ __global__ void delta_prepare_kernel(float* __restrict__ qk, float* __restrict__
         }
         return silu_f(acc);
     };
+    auto move_on = [&](int c) {                                          // channel c's carried inputs: the oldest leaves, the token's enters
+        if (!moves) return;
+        for (int i = 0; i + 1 < taps - 1; ++i) st[(size_t)i * C + c] = st[(size_t)(i + 1) * C + c];
+        st[(size_t)(taps - 2) * C + c] = first[(size_t)t * ld + c];
+    };
     const int head_segments = (2 * kv_heads + 7) / 8;
     if (seg < head_segments) {                                          // unit vectors: q heads, then k heads
         const int g = seg * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
@@ -408,11 +416,14 @@ __global__ void delta_prepare_kernel(float* __restrict__ qk, float* __restrict__
         float ss = 0.f;
         for (int d = lane; d < dim; d += 32) { const float x = channel(g * dim + d); ss = fmaf(x, x, ss); }
         const float f = rsqrtf(warp_sum(ss) + unit_eps) * (g < kv_heads ? q_scale : 1.f);
-        for (int d = lane; d < dim; d += 32) qk[((size_t)t * 2 * kv_heads + g) * dim + d] = channel(g * dim + d) * f;
+        for (int d = lane; d < dim; d += 32) {
+            qk[((size_t)t * 2 * kv_heads + g) * dim + d] = channel(g * dim + d) * f;
+            move_on(g * dim + d);
+        }
         return;
     }
     int e = (seg - head_segments) * blockDim.x + threadIdx.x;
-    if (e < nv) { v[(size_t)t * nv + e] = channel(2 * nq + e); return; }
+    if (e < nv) { v[(size_t)t * nv + e] = channel(2 * nq + e); move_on(2 * nq + e); return; }
     e -= nv;
     if (e < heads) { beta[(size_t)t * heads + e] = sigmoid_f(to_f32(first[(size_t)t * ld + C + e])); return; }
     e -= heads;
@@ -426,10 +437,10 @@ __global__ void delta_prepare_kernel(float* __restrict__ qk, float* __restrict__
 }
 
 extern "C" int hb_delta_prepare(float* qk, float* v, float* beta, float* decay, float* gate, const void* first, int dtype,
-                                int ld, const void* conv, int taps, const void* conv_state, const float* low2,
+                                int ld, const void* conv, int taps, void* conv_state, const float* low2,
                                 const float* dt_bias, const float* rate_log, const int32_t* query_start,
                                 const int32_t* row_slot, int rows, int tokens, int heads, int kv_heads, int dim, int vdim,
-                                float q_scale, float unit_eps, hb_stream stream) {
+                                float q_scale, float unit_eps, int carry, hb_stream stream) {
     if (tokens == 0) return 0;
     if (taps < 1 || (taps > 1 && !conv_state)) HB_REFUSE("delta_prepare: %d taps need the carried inputs", taps);
     const long elements = 2L * heads * vdim + heads + (long)heads * dim;
@@ -437,8 +448,8 @@ extern "C" int hb_delta_prepare(float* qk, float* v, float* beta, float* decay, 
     if (segments > 65535) HB_REFUSE("delta_prepare: %ld segments a token are above 65535", segments);
     dim3 grid(tokens, (unsigned)segments);
     cudaStream_t s = (cudaStream_t)stream;
-#define HB_ARGS(T) (const T*)first, ld, (const T*)conv, taps, (const T*)conv_state, low2, dt_bias, rate_log, \
-    query_start, row_slot, rows, heads, kv_heads, dim, vdim, q_scale, unit_eps
+#define HB_ARGS(T) (const T*)first, ld, (const T*)conv, taps, (T*)conv_state, low2, dt_bias, rate_log, \
+    query_start, row_slot, rows, heads, kv_heads, dim, vdim, q_scale, unit_eps, carry
     if (dtype == HB_F32) delta_prepare_kernel<float><<<grid, 256, 0, s>>>(qk, v, beta, decay, gate, HB_ARGS(float));
     else if (dtype == HB_BF16) delta_prepare_kernel<bf16><<<grid, 256, 0, s>>>(qk, v, beta, decay, gate, HB_ARGS(bf16));
     else HB_REFUSE("delta_prepare: dtype %d", dtype);
@@ -448,13 +459,15 @@ extern "C" int hb_delta_prepare(float* qk, float* v, float* beta, float* decay, 
 }
 
 // The carried inputs of the convolution after a step: the last taps - 1 inputs of (what was carried, the row's tokens).
-// A thread per (row, channel); entry i takes what lies n places further on, so ascending i reads nothing written.
+// A thread per (row, channel); entry i takes what lies n places further on, so ascending i reads nothing written. `least`:
+// rows of fewer tokens are passed over.
 template <typename T>
 __global__ void conv_carry_kernel(T* __restrict__ conv_state, const T* __restrict__ first, int ld, int C, int keep,
-                                  const int32_t* __restrict__ query_start, const int32_t* __restrict__ row_slot) {
+                                  const int32_t* __restrict__ query_start, const int32_t* __restrict__ row_slot, int least) {
     const int b = blockIdx.y, c = blockIdx.x * blockDim.x + threadIdx.x;
     if (c >= C) return;
     const int t0 = query_start[b], n = query_start[b + 1] - t0;
+    if (n < least) return;
     T* st = conv_state + (size_t)row_slot[b] * keep * C;
     for (int i = 0; i < keep; ++i) {
         const int src = n - keep + i;                                // among the row's tokens; negative: carried before
@@ -463,13 +476,13 @@ __global__ void conv_carry_kernel(T* __restrict__ conv_state, const T* __restric
 }
 
 extern "C" int hb_conv_carry(void* conv_state, const void* first, int dtype, int ld, int channels, int taps,
-                             const int32_t* query_start, const int32_t* row_slot, int rows, hb_stream stream) {
+                             const int32_t* query_start, const int32_t* row_slot, int rows, int least, hb_stream stream) {
     if (rows == 0 || taps <= 1) return 0;
     if (rows > 65535) HB_REFUSE("conv_carry: %d rows are above 65535", rows);
     dim3 grid((channels + 127) / 128, rows);
     cudaStream_t s = (cudaStream_t)stream;
-    if (dtype == HB_F32) conv_carry_kernel<float><<<grid, 128, 0, s>>>((float*)conv_state, (const float*)first, ld, channels, taps - 1, query_start, row_slot);
-    else if (dtype == HB_BF16) conv_carry_kernel<bf16><<<grid, 128, 0, s>>>((bf16*)conv_state, (const bf16*)first, ld, channels, taps - 1, query_start, row_slot);
+    if (dtype == HB_F32) conv_carry_kernel<float><<<grid, 128, 0, s>>>((float*)conv_state, (const float*)first, ld, channels, taps - 1, query_start, row_slot, least);
+    else if (dtype == HB_BF16) conv_carry_kernel<bf16><<<grid, 128, 0, s>>>((bf16*)conv_state, (const bf16*)first, ld, channels, taps - 1, query_start, row_slot, least);
     else HB_REFUSE("conv_carry: dtype %d", dtype);
     HB_LAUNCH_CHECK("conv_carry");
     return 0;

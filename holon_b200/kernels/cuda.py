@@ -1067,7 +1067,29 @@ class CudaKernels:
     def expert_glu(self, out, x, token_of, w, starts, limit, alpha, row_scale) -> None:
         """A clamped gated unit's first half for rows laid out expert by expert: out [rows, inter] from x (gathered by
         token_of) through w [experts, 2 inter, k] (an expert's gate rows, then its up rows), each row of the product times
-        row_scale (float32 [rows] or None) before the limits: glu_clamped behind expert_linear."""
+        row_scale (float32 [rows] or None) before the limits. In bfloat16 the unit sits in the product's epilogue where the
+        product runs on the 8-row kernel or on tcgen05; else it is glu_clamped behind expert_linear."""
+        self._check(out, x, token_of, w, starts, row_scale)
+        self._f32("expert_glu", row_scale)
+        e, n2, k = w.shape
+        rows, inter = out.shape
+        if n2 != 2 * inter or x.shape[1] != k or not (out.dtype == x.dtype == w.dtype) or starts.shape[0] != e + 1 \
+                or (token_of is not None and token_of.shape[0] != rows) or (token_of is None and x.shape[0] != rows) \
+                or (row_scale is not None and row_scale.shape != (rows,)):
+            raise KernelError("expert_glu: x [*, k], w [experts, 2 inter, k], out [rows, inter], starts int32 [experts + 1], row_scale [rows]")
+        common = (self._p(out), self._p(x), self._i32(token_of, "token_of"))
+        unit = (self._p(row_scale), ctypes.c_float(limit), ctypes.c_float(alpha), rows, e, inter, k)
+        aligned = k % 8 == 0 and inter % 8 == 0 and (x.data_ptr() | w.data_ptr() | out.data_ptr()) % 16 == 0
+        if x.dtype == torch.bfloat16 and aligned and (self.expert_products == "tcgen05" or (
+                self.expert_products == "fast" and self.expert_tile_rows == 0 and rows >= self.EXPERT_TCGEN05_ROWS * e)):
+            tiles = -(-rows // 128) + min(e, rows)
+            table = torch.empty(3 * tiles, dtype=torch.int32, device=self.device)
+            gathered = torch.empty((rows, k), dtype=x.dtype, device=self.device) if token_of is not None else None
+            return self._call("hb_expert_glu_tcgen05", *common, self._p(gathered), self._p(w), self._i32(starts, "starts"),
+                              self._i32(table, "table"), *unit)
+        if x.dtype == torch.bfloat16 and aligned and self.expert_products in ("fast", "mma") and self.expert_tile_rows in (0, 8) \
+                and (rows <= 8 * e or self.expert_tile_rows == 8) and k <= 12800:
+            return self._call("hb_expert_glu_few", *common, self._p(w), self._i32(starts, "starts"), *unit)
         both = torch.empty(out.shape[0], w.shape[1], dtype=out.dtype, device=self.device)
         self.expert_linear(both, x, token_of, w, starts, 0)
         self.glu_clamped(out, both, None, limit, alpha, row_scale=row_scale)
@@ -1111,9 +1133,9 @@ class CudaKernels:
                    int(getattr(rows, "max_q", 0) or 0))
 
     def delta_prepare(self, qk, v, beta, decay, gate, first, conv, conv_state, low2, dt_bias, rate_log, rows, q_scale,
-                      unit_eps) -> None:
+                      unit_eps, carry=False) -> None:
         """From a delta-rule mixer's first product and its low-rank projections' outputs to the scan's inputs
-        (csrc/api.h: hb_delta_prepare)."""
+        (csrc/api.h: hb_delta_prepare). `carry`: the convolution's carried inputs of rows of one token move on too."""
         self._check(qk, v, beta, decay, gate, first, conv, conv_state, low2, dt_bias, rate_log, rows.query_start, rows.row_slot)
         self._f32("delta_prepare", qk, v, beta, decay, gate, low2, dt_bias, rate_log)
         t, heads, vdim = v.shape
@@ -1129,14 +1151,15 @@ class CudaKernels:
                    self._p(first), _code(first), first.shape[1], self._p(conv), taps, self._p(conv_state), self._p(low2),
                    self._p(dt_bias), self._p(rate_log), self._i32(rows.query_start, "query_start"),
                    self._i32(rows.row_slot, "row_slot"), rows.n_rows, t, heads, kv_heads, dim, vdim,
-                   ctypes.c_float(q_scale), ctypes.c_float(unit_eps))
+                   ctypes.c_float(q_scale), ctypes.c_float(unit_eps), int(bool(carry)))
 
-    def conv_carry(self, conv_state, first, channels, taps, rows) -> None:
+    def conv_carry(self, conv_state, first, channels, taps, rows, least=0) -> None:
+        """`least`: rows of fewer tokens are passed over."""
         if taps <= 1:
             return
         self._check(conv_state, first, rows.query_start, rows.row_slot)
         self._call("hb_conv_carry", self._p(conv_state), self._p(first), _code(first), first.shape[1], channels, taps,
-                   self._i32(rows.query_start, "query_start"), self._i32(rows.row_slot, "row_slot"), rows.n_rows)
+                   self._i32(rows.query_start, "query_start"), self._i32(rows.row_slot, "row_slot"), rows.n_rows, int(least))
 
     def retention_prepare(self, qk, v, first, positions, table, rot_dims, k_scale, silu=False) -> None:
         """`silu`: q, k and v pass silu before anything else (csrc/api.h: hb_retention_prepare)."""

@@ -194,8 +194,9 @@ class GatedDelta(_MatrixState):
         gate = ctx.empty(t, heads * vdim, dtype=f32)
         carried = cache.slots.get("conv")
         k.delta_prepare(qk, v, beta, decay, gate, first, self.conv.tensor, carried, low2, self.dt_bias.tensor,
-                        self.rate_log.tensor, step.rows, dim ** -0.5, self.UNIT_EPS)
-        k.conv_carry(carried, first, self.channels, self.taps, step.rows)
+                        self.rate_log.tensor, step.rows, dim ** -0.5, self.UNIT_EPS, carry=True)
+        if step.rows.n_rows > step.rows.n_decode:                        # (rows of one token: moved on by the kernel above)
+            k.conv_carry(carried, first, self.channels, self.taps, step.rows, least=2)
         o = ctx.empty(t, heads, vdim, dtype=f32)
         k.recurrent_scan(o, qk, v, decay, None, beta, cache.slots["state"], step.rows)
         y = ctx.empty(t, heads, vdim)

@@ -1,6 +1,6 @@
 """Trace replay: feeds given token ids through the model step by step and writes logits. It samples nothing.
 
-    bin/trace_run --model DIR --dtype bfloat16|float32 --out DIR --max-tokens N [--page-size P]
+    bin/trace_run --model DIR --dtype bfloat16|float32 --out DIR --max-tokens N [--page-size P] [--max-live R]
 
 Standard input brings one JSON object a line:
 
@@ -11,8 +11,8 @@ ones generation uses; this file has no forward pass of its own). A request is ad
 and continues where it stopped; ids listed under `end` give back what they hold after the step. For a step that
 wants logits, `DIR/<step>.f32` receives them as little-endian float32 [wanted, vocab], in the order of the entries
 and of each entry's `want`. After every step a line `done <step>` is printed and flushed. The cache pool holds
-`--max-tokens` tokens, each live request's count rounded up to whole pages of `--page-size` tokens (64 unless given),
-so pages are used again.
+`--max-tokens` tokens, each live request's count rounded up to whole pages of `--page-size` tokens (64 unless given), and
+there are state slots for `--max-live` requests (4 unless given), so pages and slots are used again.
 
 The reference has no such program; the nearest are its teacher-forced scoring and its per-step snapshot trace
 (judge/holon_judge/engine.py:49-80, judge/holon_judge/snapshot.py:59-99).
@@ -25,19 +25,20 @@ import pathlib
 import sys
 
 PAGE_SIZE = 64
-MAX_LIVE = 16
+MAX_LIVE = 4
 
 
 class Replayer:
     def __init__(self, model: str, dtype: str, max_tokens: int, device="cuda:0", kernels=None,
-                 page_size: int = PAGE_SIZE) -> None:
+                 page_size: int = PAGE_SIZE, max_live: int = MAX_LIVE) -> None:
         from .engine import build
         from .weights import SafetensorsSource
         pages = max(1, -(-max_tokens // page_size))
         self.built = build(SafetensorsSource(model), dtype=dtype, device=device, kernels=kernels, page_size=page_size,
-                           max_seqs=MAX_LIVE, max_model_len=pages * page_size, max_step_tokens=pages * page_size,
+                           max_seqs=max_live, max_model_len=pages * page_size, max_step_tokens=pages * page_size,
                            pages=pages)
         self.slots: dict[str, int] = {}
+        self.max_live = max_live
 
     def step(self, record: dict):
         """Runs one step; returns the logits tensor [wanted, vocab] (32-bit) or None."""
@@ -48,7 +49,7 @@ class Replayer:
             if rid not in self.slots:
                 slot = cache.admit()
                 if slot is None:
-                    raise RuntimeError(f"step {record.get('step')}: more than {MAX_LIVE} live requests")
+                    raise RuntimeError(f"step {record.get('step')}: more than {self.max_live} live requests")
                 self.slots[rid] = slot
             slot = self.slots[rid]
             start = int(cache.computed[slot])
@@ -73,15 +74,17 @@ def main(argv=None) -> int:
     ap.add_argument("--max-tokens", required=True, type=int,
                     help="the most tokens live requests hold at any time (each rounded up to a multiple of 64)")
     ap.add_argument("--page-size", type=int, default=PAGE_SIZE, help="tokens per page of the cache (default: 64)")
+    ap.add_argument("--max-live", type=int, default=MAX_LIVE, help="requests that may be live at once (default: 4)")
     ap.add_argument("--device", default="cuda:0")
     args = ap.parse_args(argv)
-    if args.page_size < 1:
-        ap.error("--page-size must be at least 1")
+    if args.page_size < 1 or args.max_live < 1:
+        ap.error("--page-size and --max-live must be at least 1")
     out = pathlib.Path(args.out)
     out.mkdir(parents=True, exist_ok=True)
     import torch
     with torch.inference_mode():
-        replayer = Replayer(args.model, args.dtype, args.max_tokens, args.device, page_size=args.page_size)
+        replayer = Replayer(args.model, args.dtype, args.max_tokens, args.device, page_size=args.page_size,
+                            max_live=args.max_live)
         for line in sys.stdin:
             line = line.strip()
             if not line:

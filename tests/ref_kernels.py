@@ -178,7 +178,7 @@ class RefKernels:
                 state[slots[b], h] = s.T
 
     def delta_prepare(self, qk, v, beta, decay, gate, first, conv, conv_state, low2, dt_bias, rate_log, rows, q_scale,
-                      unit_eps):
+                      unit_eps, carry=False):
         t, heads, vdim = v.shape
         kv_heads, dim = qk.shape[2], qk.shape[3]
         taps = conv.shape[1]
@@ -193,6 +193,10 @@ class RefKernels:
             seq = torch.cat((carried, x[s:e, :c]), 0)
             y[s:e] = sum(seq[j:j + e - s] * conv.float()[:, j] for j in range(taps))
         y = y * torch.sigmoid(y)
+        if carry and taps > 1:
+            for b in range(rows.n_rows):
+                if qs[b + 1] - qs[b] == 1:
+                    conv_state[slots[b]] = torch.cat((conv_state[slots[b]][1:], first[qs[b]:qs[b] + 1, :c]), 0)
         unit = lambda z: z / torch.sqrt((z * z).sum(-1, keepdim=True) + unit_eps)      # noqa: E731
         qk[:, 0] = unit(y[:, :nq].view(t, kv_heads, dim)) * q_scale
         qk[:, 1] = unit(y[:, nq:2 * nq].view(t, kv_heads, dim))
@@ -202,11 +206,13 @@ class RefKernels:
         decay.copy_(torch.exp(-torch.exp(rate_log)[None, :, None] * torch.nn.functional.softplus(a).view(t, heads, dim)))
         gate.copy_(torch.sigmoid(low2[:, heads * dim:]).view(gate.shape))
 
-    def conv_carry(self, conv_state, first, channels, taps, rows):
+    def conv_carry(self, conv_state, first, channels, taps, rows, least=0):
         if taps <= 1:
             return
         qs, slots = rows.query_start.tolist(), rows.row_slot.tolist()
         for b in range(rows.n_rows):
+            if qs[b + 1] - qs[b] < least:
+                continue
             seq = torch.cat((conv_state[slots[b]], first[qs[b]:qs[b + 1], :channels]), 0)
             conv_state[slots[b]] = seq[-(taps - 1):]
 

@@ -221,9 +221,9 @@ class _Faulty(RefKernels):
             window -= 1
         super().paged_attention(out, q, kv, block_table, rows, scale, window, sinks)
 
-    def conv_carry(self, conv_state, first, channels, taps, rows):
+    def conv_carry(self, conv_state, first, channels, taps, rows, least=0):
         if self.fault != "inputs_not_carried":
-            super().conv_carry(conv_state, first, channels, taps, rows)
+            super().conv_carry(conv_state, first, channels, taps, rows, least)
 
     def embed_pair(self, out, table, scale, pair, ids, positions, rows, prev, mul_prev, mul_cur, buckets):
         keep = prev.clone()
