@@ -167,6 +167,40 @@ VOBOSUN_SIZES = {
 }
 
 
+def gegunex_config(width: int, heads: int, dim: int, rot: int, vdim: int, q_rank: int, rank: int, window: int, delta_heads: int,
+                   delta_kv_heads: int, delta_dim: int, low_rank: int, experts: int, top: int, expert_ff: int, layers: int,
+                   taps: int = 4, vocab: int = 32768) -> dict:
+    """A Gegunex model for `--only gegunex`: channel-delta, latent-attention and lightning layers in turn, every layer with
+    routed clamped experts."""
+    latent = {"heads": heads, "dim": dim, "rot_dim": rot, "vdim": vdim, "q_rank": q_rank, "kv_rank": rank, "mask": {"size": window},
+              "scale": (dim + rot) ** -0.5,
+              "rot": {"base": 1000000.0, "dims": rot, "scaling": {"factor": 16.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    delta = {"heads": delta_heads, "kv_heads": delta_kv_heads, "dim": delta_dim, "vdim": delta_dim, "conv": taps,
+             "decay_rank": low_rank, "gate_rank": low_rank}
+    lightning = {"heads": delta_heads, "dim": delta_dim, "vdim": delta_dim, "decay": [1 - 2.0 ** (-5 - h % 6) for h in range(delta_heads)]}
+    moe = {"kind": "moe", "router": {"experts": experts, "top": top}, "expert": {"ff": expert_ff, "limit": 7.0}}
+    turns = [("channel_delta", delta), ("latent_attention", latent), ("lightning", lightning)]
+    return {"architecture": "Gegunex", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "residual_mult": 0.5, "logit_softcap": 30.0,
+            "layers": [{"type": turns[i % 3][0], "mixer": turns[i % 3][1], "mlp": moe} for i in range(layers)]}
+
+
+# Layers of the sizes of published decoders of 1.5 and 8 billion parameters (as Kasovik's), matrix-state heads of 128 x 128,
+# latents of 512 with a rotated part of 64 (Rulorax's "lite") and queries through a latent of three eighths of the width, windows of 1,024 and
+# 2,048 tokens, 32 experts of which the 4 chosen ones together have the dense feed-forward's size. Beside each the two designs
+# whose parts it is closest to, Kasovik (delta rule, fixed decays) of `KASOVIK_SIZES` and Rulorax (latent attention, experts) of
+# the same width, heads, latents and experts, and the Qwen3 decoder of the same width, heads and layers.
+GEGUNEX_SIZES = {
+    "base": (dict(width=2048, heads=16, dim=128, rot=64, vdim=128, q_rank=768, rank=512, window=1024, delta_heads=16, delta_kv_heads=4,
+                  delta_dim=128, low_rank=64, experts=32, top=4, expert_ff=1536, layers=6), "base",
+             dict(width=2048, heads=16, rank=512, rot=64, dim=128, vdim=128, dense_ff=6144, experts=32, top=4, expert_ff=1536,
+                  shared_ff=1536, layers=6)),
+    "wide": (dict(width=4096, heads=32, dim=128, rot=64, vdim=128, q_rank=1536, rank=512, window=2048, delta_heads=32, delta_kv_heads=8,
+                  delta_dim=128, low_rank=128, experts=32, top=4, expert_ff=3072, layers=6), "wide",
+             dict(width=4096, heads=32, rank=512, rot=64, dim=128, vdim=128, dense_ff=12288, experts=32, top=4, expert_ff=3072,
+                  shared_ff=3072, layers=6)),
+}
+
+
 def _find_number(data, key: str):
     """The first number stored under `key` anywhere in a nested JSON value (a dict under the key: its "value")."""
     if isinstance(data, dict):
@@ -638,6 +672,13 @@ def vobosun_run(args) -> dict:
     return beside_qwen3(args, "vobosun", table, vobosun_config, args.vobosun_sizes)
 
 
+def gegunex_run(args) -> dict:
+    """The same for Gegunex beside the Kasovik and Rulorax models and the Qwen3 decoder of the same width, heads and layers."""
+    table = {name: (ours, KASOVIK_SIZES[like][1], {"kasovik": kasovik_config(**KASOVIK_SIZES[like][0]), "rulorax": rulorax_config(**latent)})
+             for name, (ours, like, latent) in GEGUNEX_SIZES.items()}
+    return beside_qwen3(args, "gegunex", table, gegunex_config, args.gegunex_sizes)
+
+
 def beside_qwen3(args, design: str, table: dict, make_config, chosen: str, context: int = 2048) -> dict:
     import gc
     import torch
@@ -788,6 +829,8 @@ def run_ours(args) -> dict:
         return tilarax_run(args)
     if args.only == "vobosun":
         return vobosun_run(args)
+    if args.only == "gegunex":
+        return gegunex_run(args)
     cfg = dict(QWEN3_8B, num_hidden_layers=args.layers)
     context, batch = args.context, args.batch
     engine = Engine(EngineConfig(model="random weights, seed 2", device="cuda:0", dtype="bfloat16", page_size=64,
@@ -910,7 +953,7 @@ def main() -> int:
                          "several passes should hold a few GB only (e.g. 0.03 with --layers 4 --batch 8)")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=8192)
-    ap.add_argument("--only", default="all", choices=("all", "decode", "prefill", "long_prompt", "sizes", "shared_prompt", "rulorax", "kasovik", "tilarax", "vobosun"),
+    ap.add_argument("--only", default="all", choices=("all", "decode", "prefill", "long_prompt", "sizes", "shared_prompt", "rulorax", "kasovik", "tilarax", "vobosun", "gegunex"),
                     help="run one part only (for profiling a small case); the JSON line then lacks the other parts. "
                          "long_prompt: time to first token of a 30,000-token prompt behind three decoding requests; "
                          "sizes: the workloads of the Qwen3-32B and Qwen3-0.6B configurations (--sizes); "
@@ -921,6 +964,7 @@ def main() -> int:
     ap.add_argument("--kasovik-sizes", default="", help="with --only kasovik: which sizes (base, wide; default both)")
     ap.add_argument("--tilarax-sizes", default="", help="with --only tilarax: which sizes (base, wide; default both)")
     ap.add_argument("--vobosun-sizes", default="", help="with --only vobosun: which sizes (base, wide; default both)")
+    ap.add_argument("--gegunex-sizes", default="", help="with --only gegunex: which sizes (base, wide; default both)")
     ap.add_argument("--no-points", action="store_true", help="leave out the points at other batch sizes and contexts")
     ap.add_argument("--no-kernels", action="store_true", help="leave out the per-kernel table")
     args = ap.parse_args()

@@ -759,7 +759,7 @@ __global__ void __launch_bounds__(BM == 128 ? 256 : 128) expert_linear_bf16_kern
 // ---------------------------------------------------------------- a row or two an expert (decode steps)
 // Tiles of 8 rows; the product is bound by reading each chosen expert's weight once, and what counts is how many bytes
 // are on their way: a CTA of eight warps keeps the tile's rows of x in shared memory and takes 32 weight rows, four a
-// warp; a lane reads 16 bytes of each of them per step of 256 columns (two steps in flight) and multiplies on the CUDA
+// warp; a lane reads 16 bytes of each of them per step of 256 columns (two steps in flight, requested ahead) and multiplies on the CUDA
 // cores in 32-bit; the lanes' sums meet by shuffles. No tensor cores: with one or two rows they would idle anyway.
 // GLU: w [experts, 2 n, k] holds an expert's n gate rows, then its n up rows; a warp takes two gate rows and the two up rows
 // beside them, and the epilogue is the clamped unit: with f = row_scale[row] (null: 1), g = min(f gate, limit),
@@ -783,46 +783,59 @@ __global__ void __launch_bounds__(256) expert_linear_few_kernel(bf16* __restrict
     if (e < 0) return;
     const int nrows = min(XF_ROWS, tile_info[2] - m0);
     const int chunks = k >> 3;
+    constexpr int COLS = GLU ? XF_WROWS / 2 : XF_WROWS;     // output columns a warp
+    const int nr = (blockIdx.x * 8 + warp) * COLS;          // this warp's first output column: weight row nr (and, GLU, n + nr)
+    const bf16* we = w + (size_t)e * (GLU ? 2 : 1) * n * k;
+    const bf16* wr[XF_WROWS];                               // this warp's weight rows (past the last: the last once more, never stored)
+#pragma unroll
+    for (int j = 0; j < XF_WROWS; ++j) wr[j] = we + (size_t)(min(nr + j % COLS, n - 1) + (j / COLS) * n) * k;
+    // weights are requested two steps of 256 columns ahead, the first two before x is staged: a CTA's first bytes are on
+    // their way while it still waits for its rows
+    uint4 ahead[2][XF_WROWS];
+    auto request = [&](int kc, uint4 (&v)[XF_WROWS]) {
+#pragma unroll
+        for (int j = 0; j < XF_WROWS; ++j) v[j] = kc < k ? __ldcs((const uint4*)(wr[j] + kc)) : make_uint4(0u, 0u, 0u, 0u);
+    };
+    request(lane * 8, ahead[0]);
+    request(lane * 8 + 256, ahead[1]);
     for (int c = tid; c < nrows * chunks; c += 256) {
         const int r = c / chunks, col = (c % chunks) * 8;
         const int src = token_of ? token_of[m0 + r] : m0 + r;
         *(uint4*)(xs + (size_t)r * k + col) = __ldg((const uint4*)(x + (size_t)src * k + col));
     }
     __syncthreads();
-    constexpr int COLS = GLU ? XF_WROWS / 2 : XF_WROWS;     // output columns a warp
-    const int nr = (blockIdx.x * 8 + warp) * COLS;          // this warp's first output column: weight row nr (and, GLU, n + nr)
     if (nr >= n) return;
-    const bf16* we = w + (size_t)e * (GLU ? 2 : 1) * n * k;
     float acc[XF_WROWS][XF_ROWS];
 #pragma unroll
     for (int j = 0; j < XF_WROWS; ++j)
 #pragma unroll
         for (int r = 0; r < XF_ROWS; ++r) acc[j][r] = 0.f;
-#pragma unroll 2
-    for (int kc = lane * 8; kc < k; kc += 256) {
-        uint4 wv[XF_WROWS];
+    for (int k0 = lane * 8; k0 < k; k0 += 512) {
 #pragma unroll
-        for (int j = 0; j < XF_WROWS; ++j)
-            wv[j] = nr + j % COLS < n ? __ldg((const uint4*)(we + (size_t)(nr + j % COLS + (j / COLS) * n) * k + kc)) : make_uint4(0u, 0u, 0u, 0u);
-        float wf[XF_WROWS][8];
+        for (int step = 0; step < 2; ++step) {
+            const int kc = k0 + step * 256;
+            if (kc >= k) break;
+            float wf[XF_WROWS][8];
 #pragma unroll
-        for (int j = 0; j < XF_WROWS; ++j) {
-            const __nv_bfloat162* h = (const __nv_bfloat162*)&wv[j];
+            for (int j = 0; j < XF_WROWS; ++j) {
+                const __nv_bfloat162* h = (const __nv_bfloat162*)&ahead[step][j];
 #pragma unroll
-            for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(h[i]); wf[j][2 * i] = f.x; wf[j][2 * i + 1] = f.y; }
-        }
+                for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(h[i]); wf[j][2 * i] = f.x; wf[j][2 * i + 1] = f.y; }
+            }
+            request(kc + 512, ahead[step]);
 #pragma unroll
-        for (int r = 0; r < XF_ROWS; ++r) {
-            if (r < nrows) {
-                const uint4 xv = *(const uint4*)(xs + (size_t)r * k + kc);
-                const __nv_bfloat162* h = (const __nv_bfloat162*)&xv;
-                float xf[8];
+            for (int r = 0; r < XF_ROWS; ++r) {
+                if (r < nrows) {
+                    const uint4 xv = *(const uint4*)(xs + (size_t)r * k + kc);
+                    const __nv_bfloat162* h = (const __nv_bfloat162*)&xv;
+                    float xf[8];
 #pragma unroll
-                for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(h[i]); xf[2 * i] = f.x; xf[2 * i + 1] = f.y; }
+                    for (int i = 0; i < 4; ++i) { const float2 f = __bfloat1622float2(h[i]); xf[2 * i] = f.x; xf[2 * i + 1] = f.y; }
 #pragma unroll
-                for (int j = 0; j < XF_WROWS; ++j)
+                    for (int j = 0; j < XF_WROWS; ++j)
 #pragma unroll
-                    for (int i = 0; i < 8; ++i) acc[j][r] = fmaf(wf[j][i], xf[i], acc[j][r]);
+                        for (int i = 0; i < 8; ++i) acc[j][r] = fmaf(wf[j][i], xf[i], acc[j][r]);
+                }
             }
         }
     }

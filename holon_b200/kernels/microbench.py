@@ -413,13 +413,64 @@ def scan(k, args) -> None:
                   f"{kind}: {us:8.1f} us  ({us / counts[0]:6.3f} us a token, {moved / 1e6:6.1f} MB moved)")
 
 
+def layernorm(k, args) -> None:
+    """The residual sum with its layer norm (`add_layernorm`) over rows of `--hidden`: a sublayer's row added, four rows a token
+    out of the experts' pile, and beside them `add_rmsnorm`. Two sets of buffers alternate; many rows are larger than the L2."""
+    dev, dim = k.device, args.hidden
+    for t in args.rows:
+        sets = []
+        for _ in range(2):
+            h, y = torch.randn(t, dim, device=dev), torch.randn(t, dim, device=dev).bfloat16()
+            pile = torch.randn(4 * t, dim, device=dev).bfloat16()
+            place = torch.randperm(4 * t, device=dev).to(torch.int32)
+            sets.append((h, y, pile, place, torch.empty(t, dim, device=dev, dtype=torch.bfloat16)))
+        w = torch.ones(dim, device=dev, dtype=torch.bfloat16)
+        base = t * dim * (4 + 4 + 2)                                     # the stream in and out, the normed rows
+        cases = (("one row a token", base + 2 * t * dim, lambda h, y, pile, place, out: k.add_layernorm(out, h, y, 0.5, w, 1e-5, None)),
+                 ("four rows a token", base + 8 * t * dim, lambda h, y, pile, place, out: k.add_layernorm(out, h, pile, 0.5, w, 1e-5, None, place=place)),
+                 ("add_rmsnorm", base + 2 * t * dim, lambda h, y, pile, place, out: k.add_rmsnorm(out, h, y, w, 1e-5, 0.0, None)))
+        for name, moved, fn in cases:
+            us = in_graph([lambda s=s, fn=fn: fn(*s) for s in sets])
+            print(f"layernorm {t:6d} rows of {dim}, {name:18s}: {us:7.1f} us  ({moved / us / 1e3:7.0f} GB/s)")
+
+
+def expert_glu(k, args) -> None:
+    """The clamped unit of routed experts (`expert_glu`: 32 experts, 4 a token, experts of three eighths of twice the width)
+    beside the product with the unit in a kernel of its own."""
+    dev, hidden, experts, top = k.device, args.hidden, 32, 4
+    inter = hidden * 3 // 4
+    w = torch.randn(experts, 2 * inter, hidden, device=dev).mul_(0.02).bfloat16()
+    for t in args.rows:
+        x = torch.randn(t, hidden, device=dev).bfloat16()
+        z = torch.randn(t, experts, device=dev)
+        chosen, weight = torch.empty(t, top, dtype=torch.int32, device=dev), torch.empty(t, top, device=dev)
+        counts = torch.empty(2 * experts + 3, dtype=torch.int32, device=dev)
+        place, token_of = (torch.empty(t * top, dtype=torch.int32, device=dev) for _ in range(2))
+        scale = torch.empty(t * top, device=dev)
+        k.route_rows(chosen, weight, counts, place, token_of, z, experts, 1.0, False, scores="sigmoid", row_weight=scale)
+        starts = counts[experts:2 * experts + 1]
+        used = int((counts[:experts] > 0).sum())
+        out = torch.empty(t * top, inter, device=dev, dtype=torch.bfloat16)
+        both = torch.empty(t * top, 2 * inter, device=dev, dtype=torch.bfloat16)
+
+        def apart():
+            k.expert_linear(both, x, token_of, w, starts, 0)
+            k.glu_clamped(out, both, None, 7.0, 1.702, row_scale=scale)
+        for name, fn in (("in the epilogue", lambda: k.expert_glu(out, x, token_of, w, starts, 7.0, 1.702, scale)), ("apart", apart)):
+            us = in_graph([fn])
+            flops, moved = 4.0 * t * top * hidden * inter, 4.0 * used * inter * hidden + 2.0 * t * hidden + 2.0 * t * top * inter
+            print(f"expert_glu {t:5d} tokens, {used} of {experts} experts of {inter} over {hidden}, {name:16s}: {us:7.1f} us  "
+                  f"({flops / us / 1e6:6.1f} TFLOP/s, {moved / us / 1e3:6.0f} GB/s)")
+
+
 def main() -> None:
     ap = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
-    ap.add_argument("what", choices=("decode_attention", "gemm", "prefill_attention", "chain", "layer", "scan"))
+    ap.add_argument("what", choices=("decode_attention", "gemm", "prefill_attention", "chain", "layer", "scan", "layernorm", "expert_glu"))
     ap.add_argument("--heads", type=int, default=16, help="scan: value heads")
     ap.add_argument("--kv-heads", type=int, default=4, help="scan: query/key heads of the delta rule")
     ap.add_argument("--dim", type=int, default=128, help="scan: key size")
     ap.add_argument("--vdim", type=int, default=128, help="scan: value size")
+    ap.add_argument("--hidden", type=int, default=2048, help="layernorm, expert_glu: the width")
     ap.add_argument("--rows", type=int, nargs="*", default=None)
     ap.add_argument("--context", type=int, default=8192)
     ap.add_argument("--splits", type=int, nargs="*", default=None)
@@ -441,6 +492,12 @@ def main() -> None:
         elif args.what == "prefill_attention":
             args.rows = args.rows or [2048]
             prefill_attention(k, args)
+        elif args.what == "layernorm":
+            args.rows = args.rows or [8, 2048, 8192]
+            layernorm(k, args)
+        elif args.what == "expert_glu":
+            args.rows = args.rows or [1, 8, 2048]
+            expert_glu(k, args)
         elif args.what == "scan":
             args.rows = args.rows or [2048, 256, 1]
             scan(k, args)

