@@ -116,7 +116,7 @@ static int launch_add_layernorm(void* out, void* h, const void* delta, float sca
     size_t smem = (size_t)dim * sizeof(float);
     if (vec && quads <= 2048) {
         // few rows (latency counts): a group a thread where a block has that many threads; many rows: blocks of up to 512
-        const int wide = rows <= 256 ? 1024 : 512;
+        const int wide = rows <= 256 ? 1024 : quads > 512 ? 512 : 256;
         nv = quads <= wide ? 1 : quads <= 2 * wide ? 2 : quads <= 4 * wide ? 4 : 8;
         threads = ((quads + nv - 1) / nv + 31) / 32 * 32;
         smem = 0;
