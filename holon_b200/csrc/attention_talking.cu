@@ -552,7 +552,7 @@ static int launch_talking(void* out, const void* q, const void* kv, const int32_
 #define HB_TALK(E) do { \
         auto kernel = splits > 1 ? (vec && E >= 4 ? attention_talking_kernel<T, E, true, (E >= 4)> : attention_talking_kernel<T, E, true, false>) \
                                  : (vec && E >= 4 ? attention_talking_kernel<T, E, false, (E >= 4)> : attention_talking_kernel<T, E, false, false>); \
-        if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+        if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
         kernel<<<dim3(tokens, splits > 1 ? splits : 1), warps * 32, smem, s>>>((T*)out, (const T*)q, (const T*)kv, block_table, \
             table_stride, row_slot, query_start, kv_len, rows, heads, kv_heads, kd, vd, pages, page_size, scale, head_scale, \
             chunk, window, talk, partial); \
@@ -600,10 +600,10 @@ extern "C" int hb_talking_mix(void* out, const void* wide, int dtype, int token0
     if (smem > 200 * 1024) HB_REFUSE("talking_mix: %zu bytes of shared memory a token", smem);
     cudaStream_t s = (cudaStream_t)stream;
     if (dtype == HB_BF16) {
-        if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(talking_mix_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(talking_mix_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         talking_mix_kernel<bf16><<<count, 256, smem, s>>>((bf16*)out, (const bf16*)wide, token0, heads, kv_heads, value_dim, talk);
     } else if (dtype == HB_F32) {
-        if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(talking_mix_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(talking_mix_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         talking_mix_kernel<float><<<count, 256, smem, s>>>((float*)out, (const float*)wide, token0, heads, kv_heads, value_dim, talk);
     } else HB_REFUSE("talking_mix: dtype %d", dtype);
     HB_LAUNCH_CHECK("talking_mix");

@@ -156,7 +156,7 @@ static int launch_add_rmsnorm(void* out, void* h, const void* delta, const void*
     if (smem > 200 * 1024) HB_REFUSE("rmsnorm: a row of %d values does not fit shared memory (limit 51200)", dim);
     const bool vec = dim % 4 == 0 && (((uintptr_t)out | (uintptr_t)h | (uintptr_t)delta | (uintptr_t)weight) % 16 == 0);
     auto kernel = vec ? add_rmsnorm_kernel<TH, TD, TW, true> : add_rmsnorm_kernel<TH, TD, TW, false>;
-    if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     const int per = vec ? 4 : 1;
     int threads = dim >= 4096 * per ? 1024 : (dim >= 1024 * per ? 512 : (dim >= 256 * per ? 256 : 128));
     if (vec && dim <= 4096 && rows <= 256) threads = (dim / 4 + 31) / 32 * 32;   // few rows (latency counts): a row in one pass, four values a thread in registers
@@ -501,7 +501,7 @@ extern "C" int hb_sum_norm(float* h, const void* x0, const void* x1, const void*
         && aligned16(bias) && aligned16(out) && aligned16(weight);
 #define HB_RUN(T, TW) do { \
         auto kernel = vec ? sum_norm_kernel<T, TW, true> : sum_norm_kernel<T, TW, false>; \
-        if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+        if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
         kernel<<<tokens, threads, smem, s>>>(h, (const T*)x0, (const T*)x1, (const T*)x2, (const T*)x3, s0, s1, s2, s3, \
                                             (const T*)bias, (T*)out, (const TW*)weight, eps, offset, hidden); } while (0)
     if (dtype == HB_F32 && weight_dtype == HB_F32) HB_RUN(float, float);
@@ -584,11 +584,11 @@ extern "C" int hb_out_norm_add(float* dst, const float* src, const void* y, int 
     const int threads = dim >= 1024 ? 256 : 128;
     cudaStream_t s = (cudaStream_t)stream;
     if (y_dtype == HB_F32 || !y) {
-        if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(out_norm_add_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(out_norm_add_kernel<float>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         out_norm_add_kernel<float><<<rows, threads, smem, s>>>(dst, src, (const float*)y, bias, bias_dtype == HB_F32, weight,
             weight_dtype == HB_F32, eps, offset, hist, hist_stride, n_hist, coef, avg, cast, cast_dtype, dim);
     } else if (y_dtype == HB_BF16) {
-        if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(out_norm_add_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(out_norm_add_kernel<bf16>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         out_norm_add_kernel<bf16><<<rows, threads, smem, s>>>(dst, src, (const bf16*)y, bias, bias_dtype == HB_F32, weight,
             weight_dtype == HB_F32, eps, offset, hist, hist_stride, n_hist, coef, avg, cast, cast_dtype, dim);
     } else HB_REFUSE("out_norm_add: dtype %d", y_dtype);

@@ -164,7 +164,7 @@ extern "C" int hb_route_top(int32_t* chosen, float* weight, int32_t* counts, con
     if (correction || groups > 1 || tiny != 0.f) {
         const size_t smem = (size_t)24 * experts * sizeof(float);
         if (smem > 200 * 1024) HB_REFUSE("route_top: a choice in groups takes up to 2133 experts, not %d", experts);
-        if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(route_choice_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(route_choice_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         route_choice_kernel<<<(tokens + 7) / 8, 256, smem, (cudaStream_t)stream>>>(chosen, weight, counts, z, ld, tokens, experts, top,
                                                                                   scale, renormalize, bias, correction, groups, keep, tiny, sigmoid);
         HB_LAUNCH_CHECK("route_choice");
@@ -335,7 +335,7 @@ extern "C" int hb_route_rows(int32_t* chosen, float* weight, int32_t* counts, in
     const int grouped = correction || groups > 1 || tiny != 0.f;
     if (tokens <= RS_TOKENS && experts <= RS_EXPERTS) {
         const size_t smem = ((size_t)(grouped ? 24 : 8) * experts + 2 * experts + 1) * sizeof(float);
-        if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(route_rows_small_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(route_rows_small_kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         route_rows_small_kernel<<<1, 256, smem, s>>>(chosen, weight, counts, place, token_of, z, ld, tokens, experts, top, scale,
                                                      renormalize, bias, correction, groups, keep, tiny, grouped, sigmoid, row_weight);
         HB_LAUNCH_CHECK("route_rows_small");
@@ -877,7 +877,7 @@ extern "C" int hb_expert_linear_bf16(void* out, const void* x, const int32_t* to
     cudaStream_t s = (cudaStream_t)stream;
     if (bm == 8) {
         const size_t smem = (size_t)XF_ROWS * k * sizeof(bf16);
-        if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(expert_linear_few_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+        if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(expert_linear_few_kernel<false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
         dim3 few((n + 31) / 32, (unsigned)tiles);
         expert_linear_few_kernel<false><<<few, 256, smem, s>>>((bf16*)out, (const bf16*)x, token_of, (const bf16*)w, starts, experts, n, k, act, nullptr, 0.f, 0.f);
         HB_LAUNCH_CHECK("expert_linear_few");
@@ -885,7 +885,7 @@ extern "C" int hb_expert_linear_bf16(void* out, const void* x, const int32_t* to
     }
     const size_t smem = sizeof(bf16) * XB_STAGES * (size_t)(bm + XB_BN) * XB_LD;
 #define XB_GO(BM_, T_) do { \
-        if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(expert_linear_bf16_kernel<BM_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+        if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(expert_linear_bf16_kernel<BM_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
         expert_linear_bf16_kernel<BM_><<<grid, T_, smem, s>>>((bf16*)out, (const bf16*)x, token_of, (const bf16*)w, starts, experts, n, k, act); \
     } while (0)
     if (bm == 16) XB_GO(16, 128); else if (bm == 64) XB_GO(64, 128); else XB_GO(128, 256);
@@ -904,7 +904,7 @@ extern "C" int hb_expert_glu_few(void* out, const void* x, const int32_t* token_
     if (((uintptr_t)x | (uintptr_t)w) % 16) HB_REFUSE("expert_glu_few: pointers must be 16-byte aligned");
     const long tiles = (rows + XF_ROWS - 1) / XF_ROWS + (experts < rows ? experts : rows);
     if (tiles > 65535) HB_REFUSE("expert_glu_few: %d rows over %d experts are above the kernel's limit", rows, experts);
-    if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(expert_linear_few_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(expert_linear_few_kernel<true>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     expert_linear_few_kernel<true><<<dim3((inter + 15) / 16, (unsigned)tiles), 256, smem, (cudaStream_t)stream>>>(
         (bf16*)out, (const bf16*)x, token_of, (const bf16*)w, starts, experts, inter, k, 0, row_scale, limit, alpha);
     HB_LAUNCH_CHECK("expert_glu_few");

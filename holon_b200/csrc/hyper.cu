@@ -147,7 +147,7 @@ static int hyper_launch(void* out, float* xs, const float* src, const void* y, c
 #define HC_GO(S_) hyper_mix_norm_kernel<TD, TW, S_><<<rows, threads, smem, s>>>((TD*)out, xs, src, (const TD*)y, mix, outc, \
         inc, (const TW*)weight, eps, offset, index, dim, streams)
 #define HC_CASE(S_) case S_: \
-        if (smem > 48 * 1024 && cudaFuncSetAttribute(hyper_mix_norm_kernel<TD, TW, S_ % HC_MAX_STREAMS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) \
+        if (smem > 46 * 1024 && cudaFuncSetAttribute(hyper_mix_norm_kernel<TD, TW, S_ % HC_MAX_STREAMS>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem) != cudaSuccess) \
             HB_REFUSE("hyper_mix_norm: %d columns do not fit in shared memory", dim); \
         HC_GO(S_ % HC_MAX_STREAMS); break
     switch (streams <= 4 || streams == 8 ? streams : HC_MAX_STREAMS) {      // (16 stands for the kernel of any number)

@@ -369,7 +369,7 @@ extern "C" int hb_latent_attention_bf16(void* out, float* scratch, const void* q
     const size_t smem = (size_t)(mt + 2 * LB_BN) * (dk + 8) * sizeof(bf16) + (r > 1 ? (size_t)(warps / r) * 16 * LB_SLD * sizeof(float) : 0);
     dim3 grid((unsigned)tiles, (unsigned)splits);
 #define LB_GO(R_, W_) do { \
-        if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(latent_attention_bf16_kernel<R_, W_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+        if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(latent_attention_bf16_kernel<R_, W_>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
         latent_attention_bf16_kernel<R_, W_><<<grid, W_ * 32, smem, s>>>((bf16*)out, scratch, (const bf16*)qa, (const bf16*)cache, \
             block_table, table_stride, row_slot, query_start, kv_len, row0, row1, heads, rank, dk, pages, page_size, scale, window, splits, sinks); \
     } while (0)

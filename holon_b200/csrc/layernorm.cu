@@ -124,7 +124,7 @@ static int launch_add_layernorm(void* out, void* h, const void* delta, float sca
     if (smem > 200 * 1024) HB_REFUSE("add_layernorm: a row of %d values does not fit shared memory (limit 51200)", dim);
 #define LN_GO(NV_, P_) do { \
         auto kernel = add_layernorm_kernel<TH, TD, TW, NV_, P_>; \
-        if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
+        if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem)); \
         kernel<<<rows, threads, smem, s>>>((TD*)out, (TH*)h, (const TD*)delta, scale, place, top, (const TW*)weight, eps, index, dim); \
     } while (0)
 #define LN_NV(P_) do { if (nv == 0) LN_GO(0, P_); else if (nv == 1) LN_GO(1, P_); else if (nv == 2) LN_GO(2, P_); \

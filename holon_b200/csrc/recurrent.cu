@@ -333,7 +333,7 @@ static int launch_scan(float* out, const float* qk, const float* v, const float*
                         : (beta ? recurrent_scan_kernel<DPT, P, false, true> : recurrent_scan_kernel<DPT, P, false, false>);
     if (token_decay) { kernel = recurrent_scan_kernel<DPT, P, false, false, true>; head_decay = token_decay; }
     if (rate) kernel = recurrent_scan_kernel<DPT, P, true, false, false, true>;
-    if (smem > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
+    if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     kernel<<<dim3(rows, heads, tiles), threads, smem, s>>>(out, qk, v, decay, head_decay, beta, rate, state, query_start, row_slot,
                                                           heads, kv_heads, dim, vdim, VT, tb);
     HB_LAUNCH_CHECK("recurrent_scan");
@@ -609,7 +609,7 @@ extern "C" int hb_head_norm_gate(void* out, const float* o, int dtype, const flo
     if (items == 0) return 0;
     const unsigned blocks = (unsigned)((items + 3) / 4);
     cudaStream_t s = (cudaStream_t)stream;
-    if (vdim >= 512 && vdim <= 12288 && vdim % 4 == 0 && ld % 4 == 0 && items <= 0x7fffffffL &&
+    if (vdim >= 512 && vdim <= 11264 && vdim % 4 == 0 && ld % 4 == 0 && items <= 0x7fffffffL &&
         (((uintptr_t)out | (uintptr_t)o | (uintptr_t)weight | (uintptr_t)gate_mul | (uintptr_t)gate_pre) & 15) == 0) {
         const int threads = vdim >= 1024 ? 256 : 128;
         const size_t smem = (size_t)vdim * sizeof(float);
