@@ -510,7 +510,7 @@ static int launch_talking_merge(void* out, const float* partial, int splits, int
                                 const float* talk, cudaStream_t s) {
     const int slices = vd >= TM_THREADS ? 1 : TM_THREADS / vd;
     const size_t merge_bytes = ((size_t)2 * heads * splits + (size_t)slices * vd) * sizeof(float);
-    if (merge_bytes > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(talking_merge_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)merge_bytes));
+    if (merge_bytes > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(talking_merge_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)merge_bytes));
     talking_merge_kernel<T><<<dim3(tokens, heads), TM_THREADS, merge_bytes, s>>>((T*)out, partial, splits, heads, kv_heads, vd, talk);
     HB_LAUNCH_CHECK("talking_merge");
     return 0;
@@ -538,7 +538,7 @@ static int launch_talking(void* out, const void* q, const void* kv, const int32_
                 && (hpt == 1 || hpt == 2 || hpt == 4 || hpt == 8 || hpt == 16)) {
 #define HB_ROWS1(H) do { \
                 auto kernel = talking_rows1_kernel<T, H>; \
-                if (bytes > 48 * 1024) HB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes)); \
+                if (bytes > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)bytes)); \
                 kernel<<<dim3(tokens, splits), R1_THREADS, bytes, s>>>((const T*)q, (const T*)kv, block_table, table_stride, row_slot, \
                     kv_len, heads, kv_heads, kd, vd, pages, page_size, scale, head_scale, chunk, window, partial); \
             } while (0)
