@@ -7,7 +7,8 @@ page number of a group names the same page in each of its entries, so a request 
 Groups have pools of their own, sized to hold the same number of tokens
 (core/holon/core/memory.py:327-330; core/holon/core/assembly.py:140-189). A page goes back to its pool when its
 request ends, or, in a group with a window, when every position in it lies before the window of the next token
-(core/holon/core/state.py:398-418, 499-517). The last page of each pool's tensor is the null page: never handed
+(core/holon/core/state.py:398-418, 499-517) and is none of the first ones that the group keeps (`keep_first`: a request's
+pages may then have a gap between the kept ones and the window's). The last page of each pool's tensor is the null page: never handed
 out, it stands in every unused block-table cell (memory.py:49-54).
 
 With `prefix_cache` whole pages of prompts are shared between requests through `prefix.PrefixIndex`, in every group
@@ -41,7 +42,9 @@ class CacheGroup:
         self.pool = PagePool(pages)
         self.null_page = pages
         self.table = np.full((max_seqs + 1, self.max_pages), self.null_page, dtype=np.int32)   # the host block table
-        self.first = np.zeros(max_seqs + 1, dtype=np.int64)       # first logical page still held
+        # Pages of a sequence's first positions that a window does not let go of (`keep_first` of the declaration)
+        self.kept = math.ceil(getattr(decl, "keep_first", 0) / page_size) if decl.window > 0 else 0
+        self.first = np.zeros(max_seqs + 1, dtype=np.int64)       # first logical page still held behind the kept ones
         self.count = np.zeros(max_seqs + 1, dtype=np.int64)       # logical pages reserved so far
         self.dirty: set[int] = set()
         self.kv = torch.zeros((len(entries), pages + 1, *decl.page_shape(page_size)), dtype=dtype, device=device)
@@ -50,6 +53,11 @@ class CacheGroup:
     @staticmethod
     def page_bytes(decl: PagedKV, entries: int, page_size: int, itemsize: int) -> int:
         return entries * math.prod(decl.page_shape(page_size)) * itemsize
+
+    def held(self, slot: int) -> list[int]:
+        """The pages a slot holds, in the order of their positions: the kept first ones, then from `first` on."""
+        first, count = int(self.first[slot]), int(self.count[slot])
+        return self.table[slot, :min(self.kept, first)].tolist() + self.table[slot, first:count].tolist()
 
     def need(self, slot: int, tokens: int) -> int:
         return max(0, math.ceil(tokens / self.page_size) - int(self.count[slot]))
@@ -78,22 +86,22 @@ class CacheGroup:
 
     def passed(self, slot: int, computed: int) -> None:
         """With a window W the next token (position `computed`) reads keys after computed − W only: pages that end
-        at or before computed − W + 1 go back."""
+        at or before computed − W + 1 go back, except the kept first ones."""
         w = self.decl.window
         if w <= 0:
             return
         keep_from = max(0, computed - w + 1) // self.page_size
         first = int(self.first[slot])
-        if keep_from > first:
-            keep_from = min(keep_from, int(self.count[slot]))
+        if keep_from > max(first, self.kept):
+            keep_from, first = min(keep_from, int(self.count[slot])), max(first, self.kept)
             self.pool.give(self.table[slot, first:keep_from].tolist(), slot)
             self.table[slot, first:keep_from] = self.null_page
             self.first[slot] = keep_from
             self.dirty.add(slot)
 
     def release(self, slot: int) -> None:
-        first, count = int(self.first[slot]), int(self.count[slot])
-        self.pool.give(self.table[slot, first:count].tolist()[::-1], slot)     # the last block first: kept leaves go first
+        count = int(self.count[slot])
+        self.pool.give(self.held(slot)[::-1], slot)                            # the last block first: kept leaves go first
         self.table[slot, :count] = self.null_page
         self.first[slot] = self.count[slot] = 0
         self.dirty.add(slot)
@@ -155,7 +163,8 @@ class CacheManager:
                                                                   dtype=getattr(torch, s.dtype), device=device)
         self.prefix: PrefixIndex | None = None
         if prefix_cache and self.groups and not self.slot_states:
-            self.prefix = PrefixIndex(page_size, [max(0, g.decl.window) for g in self.groups])
+            # (a group that keeps first positions beside its window is asked for every page, as one without a window)
+            self.prefix = PrefixIndex(page_size, [0 if g.kept else max(0, g.decl.window) for g in self.groups])
             for g in self.groups:
                 g.pool.on_evict = functools.partial(self.prefix.evicted, g.index)
         self._chain_node = np.full(max_seqs + 1, ROOT, dtype=np.int64)    # per slot: the index node of its last known block
@@ -197,7 +206,7 @@ class CacheManager:
         known = min(len(tokens), int(self.computed[slot]))
         i, node = int(self._chain_blocks[slot]), int(self._chain_node[slot])
         while (i + 1) * p <= known and node != DEAD:
-            pages = [int(g.table[slot, i]) if i >= int(g.first[slot]) else None for g in self.groups]   # None: passed by the window
+            pages = [int(g.table[slot, i]) if i >= int(g.first[slot]) or i < g.kept else None for g in self.groups]   # None: passed by the window
             node, entered = self.prefix.extend(node, tokens[i * p:(i + 1) * p], pages)
             for g, page, new in zip(self.groups, pages, entered):
                 if new:
@@ -241,7 +250,7 @@ class CacheManager:
         """Whether `reserve(slot, tokens)` would succeed once the slots in `releasing` were released."""
         gone = set(releasing)
         for g in self.groups:
-            freed = {page for s in gone for page in g.table[s, int(g.first[s]):int(g.count[s])].tolist()
+            freed = {page for s in gone for page in g.held(s)
                      if g.pool.holders(page) <= gone}             # (a page shared with a request that stays is not freed)
             have = g.pool.available + len(freed)
             need = math.ceil(tokens / g.page_size) - (int(g.count[slot]) if slot is not None else 0)
@@ -265,8 +274,8 @@ class CacheManager:
                 if slot not in self.live:
                     assert count == 0 and (row == g.null_page).all(), f"slot {slot} is free but holds pages"
                     continue
-                assert (row[:first] == g.null_page).all() and (row[count:] == g.null_page).all()
-                pages = row[first:count].tolist()
+                assert (row[min(g.kept, first):first] == g.null_page).all() and (row[count:] == g.null_page).all()
+                pages = g.held(slot)
                 assert len(set(pages)) == len(pages), f"slot {slot} holds a page twice"
                 for page in pages:
                     assert 0 <= page < g.pool.pages, f"slot {slot} holds page {page}"

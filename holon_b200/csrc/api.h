@@ -391,10 +391,11 @@ int hb_softcap(float* x, long count, float cap, hb_stream stream);
 // (S column by column), all 32-bit; head h reads key head h / (heads / kv_heads). Per token: S <- g S with g = decay[t, h, :] (per key channel)
 // or head_decay[h] or token_decay[t, h] (give exactly one of the three; no beta with the last); u = beta[t, h] (v - S^T k) (beta null: u = v); S <- S + k u^T;
 // out[t, h, :] = S^T q. The state is read at the start of a row and written back at its end. `most`: no row brings more
-// tokens than this (0: unknown); it bounds the stage of tokens a block keeps in shared memory.
+// tokens than this (0: unknown); it bounds the stage of tokens a block keeps in shared memory. `take` [tokens, heads] and `skip`
+// [heads] (both or neither, with token_decay): u = take[t, h] v, and out[t, h, :] = S^T q + skip[h] v.
 int hb_recurrent_scan(float* out, const float* qk, const float* v, const float* decay, const float* head_decay,
-                      const float* token_decay, const float* beta, const float* rate, float* state, const int32_t* query_start,
-                      const int32_t* row_slot, int rows, int heads, int kv_heads, int dim, int vdim, int most, hb_stream stream);
+                      const float* token_decay, const float* beta, const float* rate, const float* take, const float* skip,
+                      float* state, const int32_t* query_start, const int32_t* row_slot, int rows, int heads, int kv_heads, int dim, int vdim, int most, hb_stream stream);
 // The generalized delta rule's inputs from its first product, rows [r | k | v | g | a] of `dtype` (each heads dim wide,
 // `ld` apart) and the low-rank decay projection's output `pre` [tokens, heads dim] in 32-bit: qk = (r, k), v,
 // decay = exp(-decay_scale sigmoid(pre + decay_bias)), rate = sigmoid(a + rate_bias) / (sum_head k^2 + unit_eps); with
@@ -422,10 +423,18 @@ int hb_retention_prepare(float* qk, float* v, const void* first, int dtype, int 
                          float k_scale, int silu, hb_stream stream);
 // out [tokens, heads, vdim] (`dtype`) = o / sqrt(mean(o^2) + eps) * weight (float [vdim], with `weight_heads` [heads
 // vdim], or null) * gate, the gate a 32-bit multiplier gate_mul [tokens, heads vdim], or silu (`gate_sigmoid`: sigmoid)
-// of gate_pre (rows `ld` apart, `dtype`), or none.
+// of gate_pre (rows `ld` apart, `dtype`), or none. `gate_first`: the gate (gate_pre) multiplies o ahead of the norm.
 int hb_head_norm_gate(void* out, const float* o, int dtype, const float* weight, const float* gate_mul,
                       const void* gate_pre, long ld, float eps, int tokens, int heads, int vdim, int weight_heads,
-                      int gate_sigmoid, hb_stream stream);
+                      int gate_sigmoid, int gate_first, hb_stream stream);
+// A state-space mixer's first product, rows `ld` apart with [x (heads vdim) | B (groups n) | C (groups n) | dt (heads)] from column
+// `at` on: x, B, C through a causal convolution over time with a bias (conv [channels, taps], conv_bias [channels], carried inputs
+// conv_state [slots, taps - 1, channels], which move on here for rows of one token) and silu -> v [tokens, heads, vdim], cb
+// [tokens, 2, groups, n] = (C, B); dt = softplus(. + dt_bias) and decay = exp(-exp(rate_log) dt) [tokens, heads].
+int hb_state_space_prepare(float* cb, float* v, float* dt, float* decay, const void* first, int dtype, long ld, int at,
+                           const void* conv, const void* conv_bias, int taps, void* conv_state, const float* dt_bias,
+                           const float* rate_log, const int32_t* query_start, const int32_t* row_slot, int rows, int tokens,
+                           int heads, int vdim, int groups, int n, hb_stream stream);
 
 // ---- the matrix memory with exponential gates (csrc/mlstm.cu): the kernels around hb_recurrent_scan with token_decay.
 // pre [tokens, ld] 32-bit: the input gate's pre-activations of the heads, then the forget gate's; bias [2 heads] likewise.
@@ -449,6 +458,36 @@ int hb_mlstm_read_out(void* out, const float* o1, const float* floor_, int dtype
 int hb_out_norm_add(float* dst, const float* src, const void* y, int y_dtype, const void* bias, int bias_dtype,
                     const void* weight, int weight_dtype, float eps, float offset, const float* hist, long hist_stride,
                     int n_hist, const float* coef, float* avg, void* cast, int cast_dtype, int rows, int dim, hb_stream stream);
+// The same without bias and average, `cast` of y's type (csrc/out_norm.cu), and for a pair of outputs put together first: with R(y) = y
+// rsqrt(mean(y^2) + pair_eps), dst = src + N(scale (R(a) a_weight + R(b) b_weight)).
+int hb_out_norm_rows(float* dst, const float* src, const void* y, int dtype, const void* weight, int weight_dtype, float eps,
+                     float offset, void* cast, int rows, int dim, hb_stream stream);
+int hb_out_norm_pair_add(float* dst, const float* src, const void* a, const void* b, int dtype, const void* a_weight,
+                         const void* b_weight, int pair_weight_dtype, float pair_eps, float scale, const void* weight,
+                         int weight_dtype, float eps, float offset, void* cast, int rows, int dim, hb_stream stream);
+
+// ---- attention with one or two maps a head (csrc/attention_maps.cu, csrc/attention_maps_tcgen05.cu)
+// cache [pages, kv_heads, page_size, maps dim + vdim]: a row [key of map 1 | key of map 2 | value]. first: rows `ld` apart, [q (heads
+// maps dim) | k (kv_heads maps dim) | v (kv_heads vdim) | ...]; norm 0: none; 1: RMSNorm per head and map with q_weight / k_weight
+// [dim], then the rotation; 2: the rotation, then an RMSNorm without weight. The first rot_dims channels turn in half-split pairs
+// (table [table_rows, rot_dims] cosines then sines). q_out [tokens, heads, maps, dim].
+int hb_qkv_maps_prepare(void* q_out, void* kv, const void* first, int dtype, long ld, const float* q_weight, const float* k_weight,
+                        float eps, int norm, const int32_t* positions, const float* table, int rot_dims, int table_rows,
+                        const int32_t* write_index, int pages, int page_size, int tokens, int heads, int kv_heads, int maps,
+                        int dim, int vdim, hb_stream stream);
+// out [tokens, heads, vdim] = o sigmoid(gate) (gate rows gate_ld apart, or null: o). A map's result is the softmax over the keys j <=
+// i with i - j < window (0: all) or j < keep of q . k scale (cap > 0: cap tanh(. / cap)), weighing the values; o is that for one map,
+// (a1 - lam a2) rsqrt(mean(.^2) + eps) factor for two.
+int hb_attention_maps(void* out, const void* q, const void* kv, int dtype, const int32_t* block_table, int table_stride,
+                      const int32_t* row_slot, const int32_t* query_start, const int32_t* kv_len, int rows, int tokens, int heads,
+                      int kv_heads, int maps, int dim, int vdim, int pages, int page_size, float scale, float cap, int window,
+                      int keep, float lam, float factor, float eps, const void* gate, long gate_ld, hb_stream stream);
+// bfloat16, rows 0 .. rows - 1 bring one token each: dim and vdim multiples of 8, maps dim and vdim up to 256; a row's keys in
+// `splits` parts (1 to 8), a CTA each, which form a thread-block cluster and merge through distributed shared memory.
+int hb_attention_maps_decode(void* out, const void* q, const void* kv, const int32_t* block_table, int table_stride,
+                             const int32_t* row_slot, const int32_t* query_start, const int32_t* kv_len, int rows, int heads,
+                             int kv_heads, int maps, int dim, int vdim, int pages, int page_size, float scale, float cap, int window,
+                             int keep, float lam, float factor, float eps, const void* gate, long gate_ld, int splits, hb_stream stream);
 
 // ---- attention whose heads share their weights after the softmax, keys and values of unequal sizes (csrc/attention_talking.cu)
 // cache [pages, kv_heads, page_size, key_dim + value_dim]. qkv rows [q | k | v] -> bias, RMSNorm of q and k per head with

@@ -243,7 +243,7 @@ __global__ void embed_pair_kernel(float* __restrict__ out, const T* __restrict__
                                   int vocab, long mul_prev, long mul_cur, int buckets) {
     const int t = blockIdx.x;
     __shared__ int s_before;
-    if (threadIdx.x == 0) {
+    if (pair && threadIdx.x == 0) {                  // (without a pair table nobody asks for the token before, and prev is null)
         int lo = 0, hi = rows;
         while (hi - lo > 1) {
             const int mid = (lo + hi) >> 1;
@@ -580,6 +580,8 @@ extern "C" int hb_out_norm_add(float* dst, const float* src, const void* y, int 
     if (y && !weight) HB_REFUSE("out_norm_add: a norm needs its weight");
     if (hist && (n_hist < 1 || !coef || !avg)) HB_REFUSE("out_norm_add: the depth average needs its coefficients and a place for the result");
     if (hist && dst != hist + (size_t)(n_hist - 1) * hist_stride) HB_REFUSE("out_norm_add: the layer's result is the last of the kept ones");
+    if (y && !bias && !hist && (!cast || cast_dtype == y_dtype))
+        return hb_out_norm_rows(dst, src, y, y_dtype, weight, weight_dtype, eps, offset, cast, rows, dim, stream);
     const size_t smem = (size_t)dim * sizeof(float);
     const int threads = dim >= 1024 ? 256 : 128;
     cudaStream_t s = (cudaStream_t)stream;

@@ -5,6 +5,8 @@
 //                                            decay per head)
 //     u  = beta_t (v_t - S^T k_t)           (the delta rule; without beta: u = v_t)
 //     S <- S + k_t u^T,      o_t = S^T q_t  (the read-out sees the token's own write)
+// (with a factor per head and token on what is written, u = take_t v_t, and a skip per head, o_t = S^T q_t + skip v_t: a state
+// space's step size and skip)
 // or, with a removal rate r_t per key channel (the generalized delta rule, both terms on the old S),
 //     S <- diag(g_t) S - (r_t o k_t)(k_t^T S) + k_t v_t^T,      o_t = S^T q_t
 // and the kernels around that scan: what turns a layer's first product into q, k, v, decays and gates (a short causal
@@ -45,10 +47,13 @@ __device__ __forceinline__ void cp_async_f32x4(float* dst, const float* src) {
 // TOKEN: `head_decay` holds one decay per token and head [tokens, heads]; it rides in the stage's beta column (no delta rule then).
 // GENERAL (with PER_CHANNEL, without DELTA): `rate` [tokens, heads, dim] is the removal rate per key channel; a fourth
 // array of the stage holds it, and a token's step is S_i <- g_i S_i + k_i (v - r_i (k . S_old)).
-template <int DPT, int P, bool PER_CHANNEL, bool DELTA, bool TOKEN = false, bool GENERAL = false>
+// TAKE (with TOKEN): `take` [tokens, heads] multiplies what is written, `skip` [heads] times the value joins the read-out; the
+// factors ride in a column of the stage of their own.
+template <int DPT, int P, bool PER_CHANNEL, bool DELTA, bool TOKEN = false, bool GENERAL = false, bool TAKE = false>
 __global__ void recurrent_scan_kernel(float* __restrict__ out, const float* __restrict__ qk, const float* __restrict__ v,
                                       const float* __restrict__ decay, const float* __restrict__ head_decay,
-                                      const float* __restrict__ beta, const float* __restrict__ rate, float* __restrict__ state,
+                                      const float* __restrict__ beta, const float* __restrict__ rate, const float* __restrict__ take,
+                                      const float* __restrict__ skip, float* __restrict__ state,
                                       const int32_t* __restrict__ query_start, const int32_t* __restrict__ row_slot,
                                       int heads, int kv_heads, int dim, int vdim, int VT, int tb) {
     extern __shared__ __align__(16) float sm[];
@@ -67,6 +72,7 @@ __global__ void recurrent_scan_kernel(float* __restrict__ out, const float* __re
         S[i] = col && d < dim ? S_g[d] : 0.f;
     }
     float fixed = head_decay && !TOKEN ? head_decay[h] : 1.f;
+    const float passes = TAKE && p == 0 ? skip[h] : 0.f;              // (one lane of a column adds the skip to its share of the sum)
     const bool vec = (dim & 3) == 0;
     if (n == 1) {                            // a row of one token (a decode step): no stage, no barrier; every thread reads
         const size_t t = (size_t)t0;         // its own channels of k, q and the decays straight from global memory
@@ -123,6 +129,8 @@ __global__ void recurrent_scan_kernel(float* __restrict__ out, const float* __re
                 S[4 * i] *= fixed; S[4 * i + 1] *= fixed; S[4 * i + 2] *= fixed; S[4 * i + 3] *= fixed;
             }
         }
+        const float value = u;
+        if (TAKE) u *= take[t * heads + h];
         if (DELTA) {
             float a = 0.f;
 #pragma unroll
@@ -132,7 +140,7 @@ __global__ void recurrent_scan_kernel(float* __restrict__ out, const float* __re
             for (int o = 1; o < P; o <<= 1) a += __shfl_xor_sync(0xffffffffu, a, o);
             u = beta[t * heads + h] * (u - a);
         }
-        float o = 0.f;
+        float o = TAKE ? passes * value : 0.f;
 #pragma unroll
         for (int i = 0; i < DPT / 4; ++i) {
             S[4 * i] = fmaf(k4[i].x, u, S[4 * i]);
@@ -152,7 +160,7 @@ __global__ void recurrent_scan_kernel(float* __restrict__ out, const float* __re
         return;
     }
     constexpr int ARRAYS = PER_CHANNEL ? (GENERAL ? 4 : 3) : 2;       // q, k, decays, removal rates
-    const int used = tb * (ARRAYS * DP + VT + 1), per_stage = (used + 3) & ~3;   // (stages start on 16-byte boundaries)
+    const int used = tb * (ARRAYS * DP + VT + (TAKE ? 2 : 1)), per_stage = (used + 3) & ~3;   // (stages start on 16-byte boundaries)
     for (int e = threadIdx.x; e < 2 * per_stage; e += blockDim.x) {      // what no copy fills stays neutral: k = q = v = 0,
         const int at = e % per_stage;                                    // decay = beta = 1
         const bool one = (PER_CHANNEL && at >= 2 * tb * DP && at < 3 * tb * DP) || (at >= used - tb && at < used);
@@ -195,6 +203,7 @@ __global__ void recurrent_scan_kernel(float* __restrict__ out, const float* __re
         }
         if ((DELTA || TOKEN) && (int)threadIdx.x < m)
             cp_async_f32(sb + threadIdx.x, (TOKEN ? head_decay : beta) + (size_t)(t0 + j0 + threadIdx.x) * heads + h);
+        if (TAKE && (int)threadIdx.x < m) cp_async_f32(sb + tb + threadIdx.x, take + (size_t)(t0 + j0 + threadIdx.x) * heads + h);
         asm volatile("cp.async.commit_group;\n" ::: "memory");
     };
 
@@ -256,6 +265,7 @@ __global__ void recurrent_scan_kernel(float* __restrict__ out, const float* __re
                 at_before = t0 + j0 + j;
                 continue;
             }
+            float value = 0.f;
             if (PER_CHANNEL) {
                 const float4* gj = (const float4*)(sg + j * DP) + p;
 #pragma unroll
@@ -265,6 +275,7 @@ __global__ void recurrent_scan_kernel(float* __restrict__ out, const float* __re
                 }
             } else {
                 if (TOKEN) fixed = sb[j];
+                if (TAKE) { value = u; u *= sb[tb + j]; }
 #pragma unroll
                 for (int i = 0; i < DPT; ++i) S[i] *= fixed;
             }
@@ -298,7 +309,7 @@ __global__ void recurrent_scan_kernel(float* __restrict__ out, const float* __re
                 o0 = fmaf(S[4 * i], q4.x, o0); o1 = fmaf(S[4 * i + 1], q4.y, o1);
                 o0 = fmaf(S[4 * i + 2], q4.z, o0); o1 = fmaf(S[4 * i + 3], q4.w, o1);
             }
-            o_before = o0 + o1;
+            o_before = TAKE ? fmaf(passes, value, o0 + o1) : o0 + o1;
             at_before = t0 + j0 + j;
         }
         __syncthreads();                                            // this stage is read: the next fetch may fill it
@@ -315,14 +326,14 @@ __global__ void recurrent_scan_kernel(float* __restrict__ out, const float* __re
 
 template <int DPT, int P>
 static int launch_scan(float* out, const float* qk, const float* v, const float* decay, const float* head_decay,
-                       const float* token_decay, const float* beta, const float* rate, float* state, const int32_t* query_start, const int32_t* row_slot, int rows,
+                       const float* token_decay, const float* beta, const float* rate, const float* take, const float* skip, float* state, const int32_t* query_start, const int32_t* row_slot, int rows,
                        int heads, int kv_heads, int dim, int vdim, int most, cudaStream_t s) {
     const int unit = 32 / P > 1 ? 32 / P : 1;                         // columns a warp holds
     int VT = vdim < 256 / P ? vdim : 256 / P;
     if (VT < 1) VT = 1;
     const int threads = ((VT + unit - 1) / unit) * unit * P;
     const int tiles = (vdim + VT - 1) / VT;
-    const int per_token = (decay ? (rate ? 4 : 3) : 2) * P * DPT + VT + 1;
+    const int per_token = (decay ? (rate ? 4 : 3) : 2) * P * DPT + VT + (take ? 2 : 1);
     int tb = 96 * 1024 / 8 / per_token;                               // two stages in at most 96 KB
     if (tb > SC_TB) tb = SC_TB;
     if (tb < 1) HB_REFUSE("recurrent_scan: key size %d needs more shared memory than a block has", dim);
@@ -331,28 +342,32 @@ static int launch_scan(float* out, const float* qk, const float* v, const float*
     const size_t smem = (size_t)2 * ((tb * per_token + 3) & ~3) * sizeof(float);
     auto kernel = decay ? (beta ? recurrent_scan_kernel<DPT, P, true, true> : recurrent_scan_kernel<DPT, P, true, false>)
                         : (beta ? recurrent_scan_kernel<DPT, P, false, true> : recurrent_scan_kernel<DPT, P, false, false>);
-    if (token_decay) { kernel = recurrent_scan_kernel<DPT, P, false, false, true>; head_decay = token_decay; }
+    if (token_decay) {
+        kernel = take ? recurrent_scan_kernel<DPT, P, false, false, true, false, true> : recurrent_scan_kernel<DPT, P, false, false, true>;
+        head_decay = token_decay;
+    }
     if (rate) kernel = recurrent_scan_kernel<DPT, P, true, false, false, true>;
     if (smem > 46 * 1024) HB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
-    kernel<<<dim3(rows, heads, tiles), threads, smem, s>>>(out, qk, v, decay, head_decay, beta, rate, state, query_start, row_slot,
+    kernel<<<dim3(rows, heads, tiles), threads, smem, s>>>(out, qk, v, decay, head_decay, beta, rate, take, skip, state, query_start, row_slot,
                                                           heads, kv_heads, dim, vdim, VT, tb);
     HB_LAUNCH_CHECK("recurrent_scan");
     return 0;
 }
 
 extern "C" int hb_recurrent_scan(float* out, const float* qk, const float* v, const float* decay, const float* head_decay,
-                                 const float* token_decay, const float* beta, const float* rate, float* state, const int32_t* query_start, const int32_t* row_slot,
-                                 int rows, int heads, int kv_heads, int dim, int vdim, int most, hb_stream stream) {
+                                 const float* token_decay, const float* beta, const float* rate, const float* take, const float* skip,
+                                 float* state, const int32_t* query_start, const int32_t* row_slot, int rows, int heads, int kv_heads, int dim, int vdim, int most, hb_stream stream) {
     if (rows == 0) return 0;
     if (kv_heads < 1 || heads % kv_heads) HB_REFUSE("recurrent_scan: %d heads are no multiple of %d key heads", heads, kv_heads);
     if (dim < 1 || dim > 1024 || vdim < 1) HB_REFUSE("recurrent_scan: key size %d (1 to 1024), value size %d", dim, vdim);
     if ((decay != nullptr) + (head_decay != nullptr) + (token_decay != nullptr) != 1) HB_REFUSE("recurrent_scan: give decays per channel and token, per head and token, or one per head");
     if (token_decay && beta) HB_REFUSE("recurrent_scan: the delta rule does not go with a decay per head and token");
+    if ((take || skip) && (!take || !skip || !token_decay)) HB_REFUSE("recurrent_scan: a factor on what is written and a skip go together, with a decay per head and token");
     if (rate && (!decay || beta)) HB_REFUSE("recurrent_scan: removal rates per key channel go with decays per key channel and without beta");
     if (rows > 65535 * 32 || heads > 65535 || (vdim + 7) / 8 > 65535) HB_REFUSE("recurrent_scan: %d rows, %d heads, value size %d", rows, heads, vdim);
     if ((((uintptr_t)qk | (uintptr_t)decay | (uintptr_t)rate) & 15) != 0) HB_REFUSE("recurrent_scan: qk, decay and rate must lie on 16-byte boundaries");
     cudaStream_t s = (cudaStream_t)stream;
-#define HB_SCAN(D, PP) return launch_scan<D, PP>(out, qk, v, decay, head_decay, token_decay, beta, rate, state, query_start, row_slot, rows, heads, \
+#define HB_SCAN(D, PP) return launch_scan<D, PP>(out, qk, v, decay, head_decay, token_decay, beta, rate, take, skip, state, query_start, row_slot, rows, heads, \
                                                  kv_heads, dim, vdim, most, s)
     // Four channels a thread up to a key size of 64, then more channels a thread. (Key size 128, 2,048 tokens of 16 heads,
     // microseconds a token with the delta rule: 16 lanes of 8 channels 0.37, 32 lanes of 4 0.40, 8 lanes of 16 0.40, 4 lanes of
@@ -458,6 +473,82 @@ extern "C" int hb_delta_prepare(float* qk, float* v, float* beta, float* decay, 
     return 0;
 }
 
+// ---------------------------------------------------------------- what the state-space mixer's first product becomes
+// A token's row of `first` holds, from column `at` on, [x (heads vdim) | B (groups n) | C (groups n) | dt (heads)]. x, B and C
+// pass a causal convolution over time with a bias (weights conv [channels, taps], the last tap the token's own; inputs before
+// the step's first token of the row come from conv_state [slots, taps - 1, channels], oldest first) and silu; x goes to v, C and
+// B to cb [token][C, B][groups n]. dt = softplus(. + dt_bias), decay = exp(-exp(rate_log) dt). grid (tokens, segments); a thread
+// owns W neighbouring channels, or one head's dt. The carried inputs of a row of one token move on here, those of longer rows in
+// hb_conv_carry (as above).
+template <typename T, int W>
+__global__ void state_space_prepare_kernel(float* __restrict__ cb, float* __restrict__ v, float* __restrict__ dt,
+                                           float* __restrict__ decay, const T* __restrict__ first, long ld, int at,
+                                           const T* __restrict__ conv, const T* __restrict__ conv_bias, int taps, T* conv_state,
+                                           const float* __restrict__ dt_bias, const float* __restrict__ rate_log,
+                                           const int32_t* __restrict__ query_start, const int32_t* __restrict__ row_slot, int rows,
+                                           int heads, int inner, int gn) {
+    const int t = blockIdx.x, C = inner + 2 * gn, quads = C / W;
+    int e = blockIdx.y * blockDim.x + threadIdx.x;
+    if (e >= quads) {
+        e -= quads;
+        if (e >= heads) return;
+        const float d = softplus_f(to_f32(first[(size_t)t * ld + at + C + e]) + dt_bias[e]);
+        dt[(size_t)t * heads + e] = d;
+        decay[(size_t)t * heads + e] = expf(-expf(rate_log[e]) * d);
+        return;
+    }
+    const int c = e * W, b = row_of_token(query_start, rows, t), t0 = query_start[b];
+    T* st = conv_state ? conv_state + (size_t)row_slot[b] * (taps - 1) * C + c : nullptr;
+    auto load = [&](const T* p, float* x) {
+        if constexpr (W == 4) { float f[4]; Vec4<T>::load(p, f); x[0] = f[0]; x[1] = f[1]; x[2] = f[2]; x[3] = f[3]; }
+        else x[0] = to_f32(p[0]);
+    };
+    float acc[W], x[W];
+    load(conv_bias + c, acc);
+    for (int j = 0; j < taps; ++j) {
+        const int from = t - (taps - 1 - j);                             // the token this tap weighs
+        load(from >= t0 ? first + (size_t)from * ld + at + c : st + (size_t)(taps - 1 + (from - t0)) * C, x);
+#pragma unroll
+        for (int i = 0; i < W; ++i) acc[i] = fmaf(to_f32(conv[(size_t)(c + i) * taps + j]), x[i], acc[i]);
+    }
+    if (st && taps > 1 && query_start[b + 1] - t0 == 1) {                // a row of one token: its carried inputs move on
+        for (int i = 0; i + 1 < taps - 1; ++i)
+#pragma unroll
+            for (int k = 0; k < W; ++k) st[(size_t)i * C + k] = st[(size_t)(i + 1) * C + k];
+#pragma unroll
+        for (int k = 0; k < W; ++k) st[(size_t)(taps - 2) * C + k] = first[(size_t)t * ld + at + c + k];
+    }
+    float* dst = c < inner ? v + (size_t)t * inner + c
+               : c < inner + gn ? cb + (size_t)t * 2 * gn + gn + (c - inner) : cb + (size_t)t * 2 * gn + (c - inner - gn);
+    if constexpr (W == 4) *(float4*)dst = make_float4(silu_f(acc[0]), silu_f(acc[1]), silu_f(acc[2]), silu_f(acc[3]));
+    else dst[0] = silu_f(acc[0]);
+}
+
+extern "C" int hb_state_space_prepare(float* cb, float* v, float* dt, float* decay, const void* first, int dtype, long ld, int at,
+                                      const void* conv, const void* conv_bias, int taps, void* conv_state, const float* dt_bias,
+                                      const float* rate_log, const int32_t* query_start, const int32_t* row_slot, int rows,
+                                      int tokens, int heads, int vdim, int groups, int n, hb_stream stream) {
+    if (tokens == 0) return 0;
+    if (taps < 1 || (taps > 1 && !conv_state)) HB_REFUSE("state_space_prepare: %d taps need the carried inputs", taps);
+    if (heads < 1 || groups < 1 || heads % groups || vdim < 1 || n < 1) HB_REFUSE("state_space_prepare: %d heads of %d, %d groups of %d", heads, vdim, groups, n);
+    const int inner = heads * vdim, gn = groups * n;
+    const size_t four = dtype == HB_F32 ? 16 : 8;
+    const bool vec = inner % 4 == 0 && gn % 4 == 0 && ld % 4 == 0 && at % 4 == 0 && (((uintptr_t)cb | (uintptr_t)v) & 15) == 0 &&
+                     (((uintptr_t)first | (uintptr_t)conv_bias | (uintptr_t)conv_state) % four) == 0;
+    const long elements = (inner + 2L * gn) / (vec ? 4 : 1) + heads, segments = (elements + 127) / 128;
+    if (segments > 65535) HB_REFUSE("state_space_prepare: %ld segments a token are above 65535", segments);
+    const dim3 grid(tokens, (unsigned)segments);
+    cudaStream_t s = (cudaStream_t)stream;
+#define HB_RUN(T, W) state_space_prepare_kernel<T, W><<<grid, 128, 0, s>>>(cb, v, dt, decay, (const T*)first, ld, at, (const T*)conv, \
+    (const T*)conv_bias, taps, (T*)conv_state, dt_bias, rate_log, query_start, row_slot, rows, heads, inner, gn)
+    if (dtype == HB_F32) { if (vec) HB_RUN(float, 4); else HB_RUN(float, 1); }
+    else if (dtype == HB_BF16) { if (vec) HB_RUN(bf16, 4); else HB_RUN(bf16, 1); }
+    else HB_REFUSE("state_space_prepare: dtype %d", dtype);
+#undef HB_RUN
+    HB_LAUNCH_CHECK("state_space_prepare");
+    return 0;
+}
+
 // The carried inputs of the convolution after a step: the last taps - 1 inputs of (what was carried, the row's tokens).
 // A thread per (row, channel); entry i takes what lies n places further on, so ascending i reads nothing written. `least`:
 // rows of fewer tokens are passed over.
@@ -535,28 +626,30 @@ extern "C" int hb_retention_prepare(float* qk, float* v, const void* first, int 
 // ---------------------------------------------------------------- per-head norm and output gate behind the scan
 // out[t, h, :] = o / sqrt(mean(o^2) + eps) * weight * gate. `weight` [vdim], [heads vdim] (`weight_heads`) or null; the
 // gate is either a ready multiplier in 32-bit (gate_mul [tokens, heads vdim]) or silu (`gate_sigmoid`: sigmoid) of a
-// pre-activation in the engine's dtype (gate_pre, rows `ld` apart). One warp per (token, head).
+// pre-activation in the engine's dtype (gate_pre, rows `ld` apart). `gate_first`: the gate multiplies o ahead of the norm. One
+// warp per (token, head).
 template <typename T>
 __global__ void head_norm_gate_kernel(T* __restrict__ out, const float* __restrict__ o, const float* __restrict__ weight,
                                       const float* __restrict__ gate_mul, const T* __restrict__ gate_pre, long ld,
-                                      float eps, long items, int heads, int vdim, int weight_heads, int gate_sigmoid) {
+                                      float eps, long items, int heads, int vdim, int weight_heads, int gate_sigmoid, int gate_first) {
     const long item = (long)blockIdx.x * (blockDim.x >> 5) + (threadIdx.x >> 5);
     if (item >= items) return;
     const int lane = threadIdx.x & 31;
     const long t = item / heads;
     const int h = (int)(item - t * heads);
     const float* x = o + item * vdim;
+    auto pre = [&](int d) -> float {
+        const float g = to_f32(gate_pre[t * ld + (long)h * vdim + d]);
+        return gate_sigmoid ? sigmoid_f(g) : silu_f(g);
+    };
     float ss = 0.f;
-    for (int d = lane; d < vdim; d += 32) ss += x[d] * x[d];
+    for (int d = lane; d < vdim; d += 32) { const float y = gate_first ? x[d] * pre(d) : x[d]; ss += y * y; }
     const float f = rsqrtf(warp_sum(ss) / vdim + eps);
     for (int d = lane; d < vdim; d += 32) {
-        float y = x[d] * f;
+        float y = (gate_first ? x[d] * pre(d) : x[d]) * f;
         if (weight) y *= weight[weight_heads ? h * vdim + d : d];
         if (gate_mul) y *= gate_mul[item * vdim + d];
-        else if (gate_pre) {
-            const float g = to_f32(gate_pre[t * ld + (long)h * vdim + d]);
-            y *= gate_sigmoid ? sigmoid_f(g) : silu_f(g);
-        }
+        else if (gate_pre && !gate_first) y *= pre(d);
         out[item * vdim + d] = from_f32<T>(y);
     }
 }
@@ -566,7 +659,7 @@ __global__ void head_norm_gate_kernel(T* __restrict__ out, const float* __restri
 template <typename T>
 __global__ void head_norm_gate_wide_kernel(T* __restrict__ out, const float* __restrict__ o, const float* __restrict__ weight,
                                            const float* __restrict__ gate_mul, const T* __restrict__ gate_pre, long ld,
-                                           float eps, int heads, int vdim, int weight_heads, int gate_sigmoid) {
+                                           float eps, int heads, int vdim, int weight_heads, int gate_sigmoid, int gate_first) {
     extern __shared__ __align__(16) float hn_row[];
     __shared__ float scratch[33];
     const long item = blockIdx.x, t = item / heads;
@@ -574,7 +667,14 @@ __global__ void head_norm_gate_wide_kernel(T* __restrict__ out, const float* __r
     const float* x = o + item * vdim;
     float ss = 0.f;
     for (int d = threadIdx.x * 4; d < vdim; d += blockDim.x * 4) {
-        const float4 v = *(const float4*)(x + d);
+        float4 v = *(const float4*)(x + d);
+        if (gate_first) {
+            float w[4];
+            Vec4<T>::load(gate_pre + t * ld + (long)h * vdim + d, w);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) w[e] = gate_sigmoid ? sigmoid_f(w[e]) : silu_f(w[e]);
+            v.x *= w[0]; v.y *= w[1]; v.z *= w[2]; v.w *= w[3];
+        }
         *(float4*)(hn_row + d) = v;
         ss += v.x * v.x + v.y * v.y + v.z * v.z + v.w * v.w;
     }
@@ -593,7 +693,7 @@ __global__ void head_norm_gate_wide_kernel(T* __restrict__ out, const float* __r
             Vec4<float>::load(gate_mul + item * vdim + d, w);
 #pragma unroll
             for (int e = 0; e < 4; ++e) y[e] *= w[e];
-        } else if (gate_pre) {
+        } else if (gate_pre && !gate_first) {
             Vec4<T>::load(gate_pre + t * ld + (long)h * vdim + d, w);
 #pragma unroll
             for (int e = 0; e < 4; ++e) y[e] *= gate_sigmoid ? sigmoid_f(w[e]) : silu_f(w[e]);
@@ -604,23 +704,24 @@ __global__ void head_norm_gate_wide_kernel(T* __restrict__ out, const float* __r
 
 extern "C" int hb_head_norm_gate(void* out, const float* o, int dtype, const float* weight, const float* gate_mul,
                                  const void* gate_pre, long ld, float eps, int tokens, int heads, int vdim,
-                                 int weight_heads, int gate_sigmoid, hb_stream stream) {
+                                 int weight_heads, int gate_sigmoid, int gate_first, hb_stream stream) {
     const long items = (long)tokens * heads;
     if (items == 0) return 0;
+    if (gate_first && (!gate_pre || gate_mul)) HB_REFUSE("head_norm_gate: a gate ahead of the norm comes as its pre-activation");
     const unsigned blocks = (unsigned)((items + 3) / 4);
     cudaStream_t s = (cudaStream_t)stream;
     if (vdim >= 512 && vdim <= 11264 && vdim % 4 == 0 && ld % 4 == 0 && items <= 0x7fffffffL &&
         (((uintptr_t)out | (uintptr_t)o | (uintptr_t)weight | (uintptr_t)gate_mul | (uintptr_t)gate_pre) & 15) == 0) {
         const int threads = vdim >= 1024 ? 256 : 128;
         const size_t smem = (size_t)vdim * sizeof(float);
-        if (dtype == HB_F32) head_norm_gate_wide_kernel<float><<<(unsigned)items, threads, smem, s>>>((float*)out, o, weight, gate_mul, (const float*)gate_pre, ld, eps, heads, vdim, weight_heads, gate_sigmoid);
-        else if (dtype == HB_BF16) head_norm_gate_wide_kernel<bf16><<<(unsigned)items, threads, smem, s>>>((bf16*)out, o, weight, gate_mul, (const bf16*)gate_pre, ld, eps, heads, vdim, weight_heads, gate_sigmoid);
+        if (dtype == HB_F32) head_norm_gate_wide_kernel<float><<<(unsigned)items, threads, smem, s>>>((float*)out, o, weight, gate_mul, (const float*)gate_pre, ld, eps, heads, vdim, weight_heads, gate_sigmoid, gate_first);
+        else if (dtype == HB_BF16) head_norm_gate_wide_kernel<bf16><<<(unsigned)items, threads, smem, s>>>((bf16*)out, o, weight, gate_mul, (const bf16*)gate_pre, ld, eps, heads, vdim, weight_heads, gate_sigmoid, gate_first);
         else HB_REFUSE("head_norm_gate: dtype %d", dtype);
         HB_LAUNCH_CHECK("head_norm_gate");
         return 0;
     }
-    if (dtype == HB_F32) head_norm_gate_kernel<float><<<blocks, 128, 0, s>>>((float*)out, o, weight, gate_mul, (const float*)gate_pre, ld, eps, items, heads, vdim, weight_heads, gate_sigmoid);
-    else if (dtype == HB_BF16) head_norm_gate_kernel<bf16><<<blocks, 128, 0, s>>>((bf16*)out, o, weight, gate_mul, (const bf16*)gate_pre, ld, eps, items, heads, vdim, weight_heads, gate_sigmoid);
+    if (dtype == HB_F32) head_norm_gate_kernel<float><<<blocks, 128, 0, s>>>((float*)out, o, weight, gate_mul, (const float*)gate_pre, ld, eps, items, heads, vdim, weight_heads, gate_sigmoid, gate_first);
+    else if (dtype == HB_BF16) head_norm_gate_kernel<bf16><<<blocks, 128, 0, s>>>((bf16*)out, o, weight, gate_mul, (const bf16*)gate_pre, ld, eps, items, heads, vdim, weight_heads, gate_sigmoid, gate_first);
     else HB_REFUSE("head_norm_gate: dtype %d", dtype);
     HB_LAUNCH_CHECK("head_norm_gate");
     return 0;

@@ -1112,11 +1112,14 @@ class CudaKernels:
             if t is not None and t.dtype != torch.float32:
                 raise KernelError(f"{what}: 32-bit tensors expected, got {t.dtype}")
 
-    def recurrent_scan(self, out, qk, v, decay, head_decay, beta, state, rows, token_decay=None, rate=None) -> None:
+    def recurrent_scan(self, out, qk, v, decay, head_decay, beta, state, rows, token_decay=None, rate=None, take=None,
+                       skip=None) -> None:
         """The token-by-token update of a matrix state per head (csrc/api.h: hb_recurrent_scan). `rate` (float32 [tokens,
-        heads, dim], with `decay`, without `beta`): the generalized delta rule, S ← diag(decay) S − (rate ∘ k)(kᵀ S) + k vᵀ."""
-        self._check(out, qk, v, decay, head_decay, beta, state, rows.query_start, rows.row_slot, token_decay, rate)
-        self._f32("recurrent_scan", out, qk, v, decay, head_decay, beta, state, token_decay, rate)
+        heads, dim], with `decay`, without `beta`): the generalized delta rule, S ← diag(decay) S − (rate ∘ k)(kᵀ S) + k vᵀ. `take`
+        (float32 [tokens, heads]) and `skip` (float32 [heads]), with `token_decay`: what is written is take · v, and the
+        read-out gains skip · v."""
+        self._check(out, qk, v, decay, head_decay, beta, state, rows.query_start, rows.row_slot, token_decay, rate, take, skip)
+        self._f32("recurrent_scan", out, qk, v, decay, head_decay, beta, state, token_decay, rate, take, skip)
         if rate is not None and (decay is None or rate.shape != decay.shape):
             raise KernelError("recurrent_scan: rate goes with decay and has its shape")
         t, heads, vdim = v.shape
@@ -1124,11 +1127,13 @@ class CudaKernels:
         if qk.shape != (t, 2, kv_heads, dim) or out.shape != v.shape or state.shape[1:] != (heads, vdim, dim) \
                 or (decay is not None and decay.shape != (t, heads, dim)) or (beta is not None and beta.shape != (t, heads)) \
                 or (head_decay is not None and head_decay.shape != (heads,)) \
-                or (token_decay is not None and token_decay.shape != (t, heads)):
+                or (token_decay is not None and token_decay.shape != (t, heads)) \
+                or (take is not None and take.shape != (t, heads)) or (skip is not None and skip.shape != (heads,)):
             raise KernelError("recurrent_scan: qk [tokens, 2, kv_heads, dim], v and out [tokens, heads, vdim], state "
                               "[slots, heads, vdim, dim], decay [tokens, heads, dim] or head_decay [heads], beta [tokens, heads]")
         self._call("hb_recurrent_scan", self._p(out), self._p(qk), self._p(v), self._p(decay), self._p(head_decay),
-                   self._p(token_decay), self._p(beta), self._p(rate), self._p(state), self._i32(rows.query_start, "query_start"),
+                   self._p(token_decay), self._p(beta), self._p(rate), self._p(take), self._p(skip), self._p(state),
+                   self._i32(rows.query_start, "query_start"),
                    self._i32(rows.row_slot, "row_slot"), rows.n_rows, heads, kv_heads, dim, vdim,
                    int(getattr(rows, "max_q", 0) or 0))
 
@@ -1153,13 +1158,33 @@ class CudaKernels:
                    self._i32(rows.row_slot, "row_slot"), rows.n_rows, t, heads, kv_heads, dim, vdim,
                    ctypes.c_float(q_scale), ctypes.c_float(unit_eps), int(bool(carry)))
 
-    def conv_carry(self, conv_state, first, channels, taps, rows, least=0) -> None:
-        """`least`: rows of fewer tokens are passed over."""
+    def conv_carry(self, conv_state, first, channels, taps, rows, least=0, at=0) -> None:
+        """`least`: rows of fewer tokens are passed over; `at`: the column of `first` in which the channels begin."""
         if taps <= 1:
             return
         self._check(conv_state, first, rows.query_start, rows.row_slot)
-        self._call("hb_conv_carry", self._p(conv_state), self._p(first), _code(first), first.shape[1], channels, taps,
+        if conv_state.dtype != first.dtype or conv_state.shape[1:] != (taps - 1, channels) or first.shape[1] < at + channels:
+            raise KernelError("conv_carry: conv_state [slots, taps - 1, channels] of first's dtype, first [tokens, >= at + channels]")
+        self._call("hb_conv_carry", self._p(conv_state), ctypes.c_void_p(first.data_ptr() + at * first.element_size()), _code(first), first.shape[1], channels, taps,
                    self._i32(rows.query_start, "query_start"), self._i32(rows.row_slot, "row_slot"), rows.n_rows, int(least))
+
+    def state_space_prepare(self, cb, v, dt, decay, first, at, conv, conv_bias, conv_state, dt_bias, rate_log, rows) -> None:
+        """From a state-space mixer's first product to the scan's inputs (csrc/api.h: hb_state_space_prepare)."""
+        self._check(cb, v, dt, decay, first, conv, conv_bias, conv_state, dt_bias, rate_log, rows.query_start, rows.row_slot)
+        self._f32("state_space_prepare", cb, v, dt, decay, dt_bias, rate_log)
+        t, heads, vdim = v.shape
+        groups, n = cb.shape[2], cb.shape[3]
+        channels, taps = conv.shape
+        if cb.shape != (t, 2, groups, n) or channels != heads * vdim + 2 * groups * n or first.shape != (t, at + channels + heads) \
+                or dt.shape != (t, heads) or decay.shape != (t, heads) or conv_bias.shape != (channels,) \
+                or not (conv.dtype == conv_bias.dtype == first.dtype) or dt_bias.shape != (heads,) or rate_log.shape != (heads,) \
+                or (taps > 1 and (conv_state is None or conv_state.shape[1:] != (taps - 1, channels) or conv_state.dtype != first.dtype)):
+            raise KernelError("state_space_prepare: first [tokens, at + x | B | C | dt], conv [channels, taps], conv_bias [channels], "
+                              "conv_state [slots, taps - 1, channels] of one dtype, cb [tokens, 2, groups, n], v [tokens, heads, vdim]")
+        self._call("hb_state_space_prepare", self._p(cb), self._p(v), self._p(dt), self._p(decay), self._p(first), _code(first),
+                   ctypes.c_long(first.shape[1]), int(at), self._p(conv), self._p(conv_bias), taps, self._p(conv_state),
+                   self._p(dt_bias), self._p(rate_log), self._i32(rows.query_start, "query_start"),
+                   self._i32(rows.row_slot, "row_slot"), rows.n_rows, t, heads, vdim, groups, n)
 
     def retention_prepare(self, qk, v, first, positions, table, rot_dims, k_scale, silu=False) -> None:
         """`silu`: q, k and v pass silu before anything else (csrc/api.h: hb_retention_prepare)."""
@@ -1189,9 +1214,12 @@ class CudaKernels:
                    ctypes.c_long(first.shape[1]), self._p(pre), self._p(decay_bias), self._p(rate_bias), t, heads, dim,
                    ctypes.c_float(decay_scale), ctypes.c_float(unit_eps))
 
-    def head_norm_gate(self, out, o, weight, gate_mul, gate_pre, eps, gate: str = "silu") -> None:
+    def head_norm_gate(self, out, o, weight, gate_mul, gate_pre, eps, gate: str = "silu", gate_first: bool = False) -> None:
         """out = o / rms(o) · weight · gate per head; `gate_pre` may be a view into wider rows (silu of it is the gate, or
-        with `gate="sigmoid"` its sigmoid); `weight` [vdim] for all heads or [heads vdim]."""
+        with `gate="sigmoid"` its sigmoid); `weight` [vdim] for all heads or [heads vdim]. `gate_first`: the gate of
+        `gate_pre` multiplies o before its root mean square is taken."""
+        if gate_first and (gate_pre is None or gate_mul is not None):
+            raise KernelError("head_norm_gate: a gate ahead of the norm comes as its pre-activation")
         if gate not in ("silu", "sigmoid"):
             raise KernelError(f"head_norm_gate: gate {gate!r}; known: silu, sigmoid")
         self._check(out, o, weight, gate_mul)
@@ -1209,7 +1237,7 @@ class CudaKernels:
             raise KernelError("head_norm_gate: out and o [tokens, heads, vdim], weight [vdim] or [heads vdim], gate_mul of o's size")
         self._call("hb_head_norm_gate", self._p(out), self._p(o), _code(out), self._p(weight), self._p(gate_mul),
                    self._p(gate_pre), ctypes.c_long(ld), ctypes.c_float(eps), t, heads, vdim, int(per_head),
-                   int(gate == "sigmoid"))
+                   int(gate == "sigmoid"), int(bool(gate_first)))
 
     # ---- a norm without statistics and the blend with the token before (csrc/dyt.cu)
     def dyt_add_norm(self, h, y, post, out, pre, index) -> None:
@@ -1301,6 +1329,84 @@ class CudaKernels:
                    _code(bias) if bias is not None else 0, self._p(weight), _code(weight) if weight is not None else 0,
                    ctypes.c_float(eps), ctypes.c_float(offset), self._p(hist), ctypes.c_long(rows * dim), int(n_hist),
                    self._p(coef), self._p(avg), self._p(cast), _code(cast) if cast is not None else 0, rows, dim)
+
+    def out_norm_pair_add(self, dst, src, pair, weight, eps, offset, cast=None) -> None:
+        """dst = src + N(pair put together) for a parts.base.NormedPair, in one kernel; `cast` gets dst in the pair's dtype."""
+        a, b = pair.a, pair.b
+        self._check(dst, src, a, b, pair.a_weight, pair.b_weight, weight, cast)
+        self._f32("out_norm_pair_add", dst, src)
+        rows, dim = dst.shape
+        if any(x.shape != dst.shape for x in (src, a, b)) or any(w.shape != (dim,) for w in (pair.a_weight, pair.b_weight, weight)) \
+                or a.dtype != b.dtype or pair.a_weight.dtype != pair.b_weight.dtype or (cast is not None and (cast.shape != dst.shape or cast.dtype != a.dtype)):
+            raise KernelError("out_norm_pair_add: dst, src, a, b, cast [rows, dim], weights [dim]; a, b and cast of one dtype")
+        self._call("hb_out_norm_pair_add", self._p(dst), self._p(src), self._p(a), self._p(b), _code(a), self._p(pair.a_weight),
+                   self._p(pair.b_weight), _code(pair.a_weight), ctypes.c_float(pair.eps), ctypes.c_float(pair.scale), self._p(weight),
+                   _code(weight), ctypes.c_float(eps), ctypes.c_float(offset), self._p(cast), rows, dim)
+
+    # ---- attention with one or two maps a head (csrc/attention_maps.cu, csrc/attention_maps_tcgen05.cu)
+    QK_NORMS = {None: 0, "before": 1, "after": 2}       # where q and k are normed, seen from the rotation
+
+    def qkv_maps_prepare(self, q_out, kv, first, q_weight, k_weight, eps, norm, positions, table, rot_dims, write_index, kv_heads,
+                         value_dim) -> None:
+        """csrc/api.h: hb_qkv_maps_prepare; q_out [tokens, heads, maps, dim], kv the cache's rows or None."""
+        self._check(q_out, kv, first, q_weight, k_weight, positions, table, write_index)
+        self._f32("qkv_maps_prepare", q_weight, k_weight, table)
+        t, heads, maps, dim = q_out.shape
+        rowlen = maps * dim + value_dim
+        if first.shape[0] != t or first.shape[1] < heads * maps * dim + kv_heads * rowlen or first.dtype != q_out.dtype \
+                or (kv is not None and (kv.dtype != first.dtype or kv.shape[1] != kv_heads or kv.shape[3] != rowlen or write_index is None)) \
+                or any(w is not None and w.shape != (dim,) for w in (q_weight, k_weight)) \
+                or (rot_dims and (table is None or table.shape[1] != rot_dims)):
+            raise KernelError("qkv_maps_prepare: first [tokens, >= q | k | v], q_out [tokens, heads, maps, dim], cache [pages, "
+                              "kv_heads, page, maps dim + value_dim] of one dtype")
+        self._call("hb_qkv_maps_prepare", self._p(q_out), self._p(kv), self._p(first), _code(first), ctypes.c_long(first.shape[1]),
+                   self._p(q_weight), self._p(k_weight), ctypes.c_float(eps), self.QK_NORMS[norm],
+                   self._i32(positions, "positions"), self._p(table), int(rot_dims), table.shape[0] if table is not None else 0,
+                   self._i32(write_index, "write_index"), kv.shape[0] - 1 if kv is not None else 0,
+                   kv.shape[2] if kv is not None else 1, t, heads, kv_heads, maps, dim, value_dim)
+
+    MAPS_CLUSTER = 8                          # parts a one-token row's keys are cut into at most (one cluster)
+
+    def attention_maps(self, out, q, kv, block_table, rows, scale, cap, window, keep_first, diff, eps, gate) -> None:
+        """out [tokens, heads, value_dim] from q [tokens, heads, maps, dim] over the cache's rows; `diff` (λ, d) for two maps;
+        `gate` [tokens, heads value_dim], a view into wider rows, or None. In bfloat16 rows of one token run on mma.sync tiles
+        with their keys in parts, rows of several tokens on tcgen05; sizes these refuse, and float32, on CUDA cores."""
+        self._check(out, q, kv, block_table, rows.row_slot, rows.query_start, rows.kv_len)
+        t, heads, maps, dim = q.shape
+        vd, kv_heads, page = out.shape[2], kv.shape[1], kv.shape[2]
+        if out.shape != (t, heads, vd) or kv.shape[3] != maps * dim + vd or not (out.dtype == q.dtype == kv.dtype) \
+                or (maps == 2) != (diff is not None):
+            raise KernelError("attention_maps: q [tokens, heads, maps, dim], out [tokens, heads, value_dim], cache [pages, kv_heads, "
+                              "page, maps dim + value_dim] of one dtype; two maps with their λ and factor")
+        if gate is not None and (gate.shape != (t, heads * vd) or gate.dtype != q.dtype or gate.stride(1) != 1 or gate.get_device() != self._index):
+            raise KernelError("attention_maps: gate must be [tokens, heads value_dim] of q's dtype, innermost stride 1")
+        lam, d = diff if diff is not None else (0.0, 0.0)
+        common = (self._i32(block_table, "block_table"), block_table.shape[1], self._i32(rows.row_slot, "row_slot"),
+                  self._i32(rows.query_start, "query_start"), self._i32(rows.kv_len, "kv_len"))
+        rules = (ctypes.c_float(scale), ctypes.c_float(cap or 0.0), int(window), int(keep_first), ctypes.c_float(lam),
+                 ctypes.c_float(1.0 - d), ctypes.c_float(eps), self._p(gate), ctypes.c_long(gate.stride(0) if gate is not None else 0))
+        sizes = (heads, kv_heads, maps, dim, vd, kv.shape[0] - 1, page)
+        head = (self._p(out), self._p(q), self._p(kv))
+        fast = q.dtype == torch.bfloat16 and self.attention_bf16 == "fast"
+        ones, portions = rows.n_decode, rows.n_rows > rows.n_decode
+        decode = fast and dim % 8 == 0 and vd % 8 == 0 and maps * dim <= 256 and vd <= 256
+        if not decode and not (fast and portions and self._maps_tcgen05(dim, vd, page)):
+            return self._call("hb_attention_maps", *head, _code(q), *common, rows.n_rows, t, *sizes, *rules)
+        if ones and decode:
+            self._call("hb_attention_maps_decode", *head, *common, ones, *sizes, *rules,
+                       self._maps_splits(ones, heads // kv_heads, kv_heads, maps, rows.max_kv, window, keep_first))
+        if portions:
+            self._call("hb_attention_maps", *head, _code(q), *common, rows.n_rows, t, *sizes, *rules)
+
+    def _maps_tcgen05(self, dim: int, vd: int, page: int) -> bool:
+        return False
+
+    def _maps_splits(self, rows: int, group: int, kv_heads: int, maps: int, max_kv: int, window: int, keep: int) -> int:
+        """Parts a one-token row's keys are cut into: enough for two CTAs an SM, each part at least one tile of 64 keys. A
+        function of the batch's size and the longest row only (under a CUDA graph: of the bucket its plan pinned)."""
+        keys = min(max_kv, window + keep + 63) if window else max_kv
+        ctas = rows * kv_heads * -(-group // (16 // maps))
+        return max(1, min(self.MAPS_CLUSTER, -(-keys // 64), -(-2 * self.sms // ctas)))
 
     # ---- attention whose heads share their weights after the softmax (csrc/attention_talking.cu)
     def qkv_talking_prepare(self, q_out, kv, keep, qkv, bias, q_weight, k_weight, eps, positions, table, rot_dims, interleaved,

@@ -1,2 +1,2 @@
 """Built-in architectures; importing this package registers them."""
-from . import gegunex, kasovik, qwen3, rulorax, tilarax, vobosun  # noqa: F401
+from . import bukuvik, gegunex, kasovik, qwen3, rulorax, tilarax, vobosun  # noqa: F401

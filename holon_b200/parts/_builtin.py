@@ -1,5 +1,5 @@
 """Registers the parts that ship with the framework."""
-from .attention import GQA, TalkingAttention
+from .attention import GQA, MapAttention, TalkingAttention
 from .base import register_part
 from .block import OutNorm, PreNorm, Sandwich
 from .embedding import Embedding, Head, PairEmbedding
@@ -10,7 +10,7 @@ from .latent import LatentAttention
 from .norm import DynamicTanh, LayerNorm, RMSNorm
 from .parallel import ParallelBlock, SideBySide
 from .position import Rope
-from .recurrent import MLSTM, GatedDelta, GeneralDelta, Lightning, Retention
+from .recurrent import MLSTM, GatedDelta, GeneralDelta, Lightning, Retention, StateSpace
 
 register_part("norm", "rmsnorm", RMSNorm, replace=True)
 register_part("position", "rope", Rope, replace=True)
@@ -37,3 +37,5 @@ register_part("block", "sandwich", Sandwich, replace=True)
 register_part("mixer", "general_delta", GeneralDelta, replace=True)
 register_part("norm", "layernorm", LayerNorm, replace=True)
 register_part("mixer", "lightning", Lightning, replace=True)
+register_part("mixer", "maps", MapAttention, replace=True)
+register_part("mixer", "state_space", StateSpace, replace=True)

@@ -219,3 +219,92 @@ class TalkingAttention(Part):
     def forward(self, x: torch.Tensor, step, cache) -> torch.Tensor:
         y, bias = self.forward_biased(x, step, cache)
         return y if bias is None else y + bias
+
+
+class MapAttention(Part):
+    """Grouped-query attention with keys and values of unequal sizes over a window, one or two maps a head, and an output gate.
+
+        s_hm(i, j) = q_hm(i) · k_gm(j) · scale, with `softcap` c: c tanh(s / c);    a_hm(i) = Σ_j softmax_j(s_hm(i, ·)) v_g(j)
+
+    for the keys j ≤ i with i − j < window (0: all) or j < keep_first; g is the head's key/value head. `maps` = 1: the head's
+    result is a_h. `maps` = 2 with `diff` d (differential attention): a_h1 − λ a_h2 divided by its root mean square over the
+    head (eps), times 1 − d, where λ = exp(Σ lq1 lk1) − exp(Σ lq2 lk2) + d is one number for the layer, worked out once when
+    the weights are loaded. `gate`: the heads' results times sigmoid(W_g x), in the attention kernels. `qk_norm` "before":
+    per head and map an RMS norm with one weight shared by all (q.norm, k.norm), then the position's rotation; "after": the
+    rotation, then a division by the root mean square without a weight. Scores, softmax, the two maps' difference and its norm
+    are 32-bit; q, keys, values and the softmax weights as the tensor cores' operands are kept in the engine's dtype.
+
+    q, k, v and g are one merged product. The cache keeps per token and kv head one row [key of map 1 | key of map 2 | value]
+    (`PagedRows`)."""
+
+    def __init__(self, ctx: BuildContext, *, heads: int, kv_heads: int, key_dim: int, value_dim: int, hidden: int, scale: float,
+                 eps: float, maps: int = 1, diff: float | None = None, softcap: float | None = None, window: int = 0,
+                 keep_first: int = 0, qk_norm: str | None = None, gate: bool = True, position: PartRef | None = None,
+                 layer: int = 0) -> None:
+        super().__init__()
+        if heads % kv_heads:
+            raise ValueError(f"map attention: {heads} heads are no multiple of {kv_heads} kv heads")
+        if maps not in (1, 2) or (maps == 2) != (diff is not None):
+            raise ValueError(f"map attention: {maps} maps with diff {diff}; two maps are combined with one, one map has none")
+        if qk_norm not in (None, "before", "after"):
+            raise ValueError(f"map attention: qk_norm {qk_norm!r}; known: None, 'before', 'after' (the rotation)")
+        self.ctx, self.heads, self.kv_heads, self.key_dim, self.value_dim = ctx, heads, kv_heads, key_dim, value_dim
+        self.scale, self.eps, self.maps, self.diff, self.cap = float(scale), float(eps), maps, diff, softcap
+        self.window, self.keep_first, self.qk_norm = int(window), int(keep_first) if window else 0, qk_norm
+        pieces = {"q": heads * maps * key_dim, "k": kv_heads * maps * key_dim, "v": kv_heads * value_dim}
+        self.gate_at = sum(pieces.values()) if gate else None
+        if gate:
+            pieces["g"] = heads * value_dim
+        self.first = self.add_child("first", Linear(ctx, "weight", hidden, pieces))
+        self.out = self.add_child("out", Linear(ctx, "weight", heads * value_dim, {"o": hidden}))
+        before = qk_norm == "before"
+        self.q_gain = self.add_param("q.norm", (key_dim,), "coef") if before else None
+        self.k_gain = self.add_param("k.norm", (key_dim,), "coef") if before else None
+        self.lam_parts = tuple(self.add_param(n, (key_dim,), "coef") for n in ("lq1", "lk1", "lq2", "lk2")) if maps == 2 else ()
+        self.lam = None                          # the layer's λ (finalize)
+        self.position = self.add_child("position", ctx.part(position, head_dim=key_dim)) if position else None
+        if self.position is not None and self.position.interleaved:
+            raise ValueError("map attention: the rotation's pairs are half-split")
+
+    def loadables(self, prefix: str = ""):
+        for name, p, rows in super().loadables(prefix):
+            for child in ("first.", "out."):
+                if name.startswith(prefix + child):
+                    name = prefix + name[len(prefix + child):]
+            yield name, p, rows
+
+    def finalize(self) -> None:
+        super().finalize()
+        if self.lam_parts and self.lam_parts[0].tensor is not None:
+            q1, k1, q2, k2 = (p.tensor.double() for p in self.lam_parts)
+            self.lam = float((q1 * k1).sum().exp() - (q2 * k2).sum().exp()) + self.diff
+
+    @property
+    def plan_group(self):
+        return "maps", self.heads, self.kv_heads, self.key_dim, self.value_dim, self.maps, self.window, self.keep_first
+
+    def capture_plan(self, step, max_model_len: int):
+        """What the attention kernels pin for a step that is captured as a CUDA graph (see base.Part)."""
+        plan = getattr(self.ctx.kernels, "attention_capture_plan", None)
+        return plan(step.rows, max_model_len) if plan is not None else None
+
+    def cache(self) -> PagedRows:
+        return PagedRows(self.kv_heads, self.maps * self.key_dim, self.value_dim, self.window, self.keep_first)
+
+    def slot_states(self):
+        return ()
+
+    def forward(self, x: torch.Tensor, step, cache) -> torch.Tensor:
+        t, k, ctx = x.shape[0], self.ctx.kernels, self.ctx
+        heads, vd, pos = self.heads, self.value_dim, self.position
+        first = self.first.forward(x)                                    # [t, q | k | v | g]
+        q = ctx.empty(t, heads, self.maps, self.key_dim)
+        k.qkv_maps_prepare(q, cache.kv if cache.fills else None, first, self.q_gain.tensor if self.q_gain else None,
+                           self.k_gain.tensor if self.k_gain else None, self.eps, self.qk_norm, step.positions,
+                           pos.table if pos else None, pos.rotary_dim if pos else 0,
+                           cache.group.write_index if cache.fills else None, self.kv_heads, vd)
+        o = ctx.empty(t, heads, vd)
+        gate = first[:, self.gate_at:self.gate_at + heads * vd] if self.gate_at is not None else None
+        k.attention_maps(o, q, cache.kv, cache.group.block_table, step.rows, self.scale, self.cap, self.window, self.keep_first,
+                         (self.lam, self.diff) if self.maps == 2 else None, self.eps, gate)
+        return self.out.forward(o.view(t, heads * vd))

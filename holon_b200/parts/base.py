@@ -108,12 +108,15 @@ class PagedLatent:
 @dataclasses.dataclass(frozen=True)
 class PagedRows:
     """Per token and kv head one row [key (key_dim) | value (value_dim)], in pages: for mixers whose keys and values
-    differ in size, and whose kernels read a token's key and value of all kv heads in one sweep. `window` as for PagedKV."""
+    differ in size, and whose kernels read a token's key and value of all kv heads in one sweep. `window` as for PagedKV;
+    `keep_first` K beside a window: the sequence's first K positions are read for as long as it lives, so the pages that
+    hold them stay."""
 
     kv_heads: int
     key_dim: int
     value_dim: int
     window: int = 0
+    keep_first: int = 0
 
     def page_shape(self, page_size: int) -> tuple[int, ...]:
         return (self.kv_heads, page_size, self.key_dim + self.value_dim)
@@ -216,6 +219,22 @@ class PairRows:
         out = self.ctx.empty(self.tokens, self.y.shape[1])
         self.ctx.kernels.expert_combine(out, self.y, self.place, None, None, None, 0)
         return out
+
+
+class NormedPair:
+    """A mixer's output before it is put together: scale · (R(a) · a_weight + R(b) · b_weight) with R(y) = y / sqrt(mean y² + eps)
+    row by row. A block that says so to the mixer (`pair_out`) norms and adds the two rows in the kernel that adds the sum."""
+
+    __slots__ = ("a", "a_weight", "b", "b_weight", "eps", "scale")
+
+    def __init__(self, a: torch.Tensor, a_weight: torch.Tensor, b: torch.Tensor, b_weight: torch.Tensor, eps: float,
+                 scale: float) -> None:
+        self.a, self.a_weight, self.b, self.b_weight, self.eps, self.scale = a, a_weight, b, b_weight, eps, scale
+
+    def combined(self) -> torch.Tensor:
+        unit = lambda y: y.float() * torch.rsqrt(y.float().pow(2).mean(-1, keepdim=True) + self.eps)      # noqa: E731
+        out = self.scale * (unit(self.a) * self.a_weight.float() + unit(self.b) * self.b_weight.float())
+        return out.to(self.a.dtype)
 
 
 class Scaled:

@@ -7,7 +7,9 @@ mixer(...), h += m · ffn(...); the factor waits on the stream beside the output
 OutNorm: the norm stands on a sublayer's OUTPUT, and the sublayers read the stream itself: x ← x + N(mixer(x)), then
 x ← x + N(ffn(x)). With `average` = n the block ends with an average over depth: with X_0 the embedding's rows and X_j
 what the j-th block before left (before ITS averaging), what goes on is Σ_j c[j] X_j over the n results so far, c the
-block's stored `depth` coefficients. The results of a step's blocks wait on the step (`step.shared`), 32-bit.
+block's stored `depth` coefficients. The results of a step's blocks wait on the step (`step.shared`), 32-bit. `residual_mult` m
+and `layer_scale` (a stored vector a per sublayer: `mixer_scale`, `ffn_scale`): x ← x + m · a ∘ N(mixer(x)); m, a and the norm's
+weight are multiplied into one 32-bit vector when the weights are loaded.
 
 Sandwich: a norm before and behind each sublayer, x ← x + N1b(mixer(N1(x))), then x ← x + N2b(ffn(N2(x))). With `shift`
 the mixer reads each token's normed row blended with the row of the token before, m_t = n_t + (n_(t−1) − n_t) · mix with a
@@ -20,7 +22,7 @@ from __future__ import annotations
 import torch
 
 from ..config.spec import PartRef
-from .base import BuildContext, Link, Part, Residual, SlotState
+from .base import BuildContext, Link, NormedPair, Part, Residual, SlotState
 
 
 class PreNorm(Part):
@@ -73,7 +75,7 @@ class OutNorm(Part):
     KEY = "outnorm"                # step.shared: {"x": the stream's rows as the sublayers read them, "hist", "n"}
 
     def __init__(self, ctx: BuildContext, *, layer: int, hidden: int, mixer: PartRef, ffn: PartRef | None, norm: PartRef,
-                 average: int | None = None, results: int = 0) -> None:
+                 average: int | None = None, results: int = 0, residual_mult: float = 1.0, layer_scale: bool = False) -> None:
         super().__init__()
         if average is not None and not 1 <= average <= results:
             raise ValueError(f"outnorm: an average over {average} of {results} results")
@@ -85,6 +87,27 @@ class OutNorm(Part):
             self.ffn_norm = self.add_child("ffn_norm", ctx.part(norm, dim=hidden))
             self.ffn = self.add_child("ffn", ctx.part(ffn, layer=layer, hidden=hidden))
         self.coef = self.add_param("depth", (average,), "coef") if average is not None else None
+        self.mult, self._gains = float(residual_mult), {}
+        self._scales = ()
+        if layer_scale:
+            self._scales = tuple((norm, self.add_param(name, (hidden,), "gain")) for name, norm in
+                                 (("mixer_scale", self.mixer_norm), ("ffn_scale", self.ffn_norm)) if norm is not None)
+
+    def finalize(self) -> None:
+        super().finalize()
+        scales = {id(norm): p.tensor for norm, p in self._scales}
+        for norm in (self.mixer_norm, self.ffn_norm):
+            w = norm.weight.tensor if norm is not None else None
+            if w is not None and (scales or self.mult != 1.0):
+                gain = self.mult * (w.float() + norm.offset)
+                if id(norm) in scales:
+                    gain = gain * scales[id(norm)].float()
+                self._gains[id(norm)] = gain.contiguous()
+
+    def _norm(self, norm):
+        """(weight, eps, offset) of what a sublayer's output passes: the norm with the multipliers behind it."""
+        gain = self._gains.get(id(norm))
+        return (norm.weight.tensor, norm.eps, norm.offset) if gain is None else (gain, norm.eps, 0.0)
 
     def _rows(self, t: int, hidden: int):
         """A place for the stream's rows in the engine's dtype (None where that is 32-bit: the stream itself is read)."""
@@ -112,7 +135,9 @@ class OutNorm(Part):
         if self.average is not None and (hist is None or n + 1 != self.average or n >= hist.shape[0]):
             raise RuntimeError(f"outnorm: this block averages {self.average} results, the step holds {n} before it")
         mixer, norm = self.mixer, self.mixer_norm
-        if hasattr(mixer, "forward_biased"):                             # the last product's bias rides in the norm's kernel
+        if self.average is None and getattr(mixer, "out_eps", None) is not None:     # two outputs, their norms and their sum
+            y, bias = mixer.pair_out(state["x"], step, cache), None
+        elif hasattr(mixer, "forward_biased"):                             # the last product's bias rides in the norm's kernel
             y, bias = mixer.forward_biased(state["x"], step, cache)
         else:
             y, bias = mixer.forward(state["x"], step, cache), None
@@ -120,18 +145,26 @@ class OutNorm(Part):
         src = stream.h
         if self.ffn is not None:
             mid = self._rows(t, hidden)
-            k.out_norm_add(own, src, y, bias, norm.weight.tensor, norm.eps, norm.offset, cast=mid)
+            self._add(own, src, y, bias, norm, mid)
             y, bias, norm, src = self.ffn.forward(mid if mid is not None else own, step), None, self.ffn_norm, own
         cast = self._rows(t, hidden)
         if self.average is not None:
             go = ctx.empty(t, hidden, dtype=torch.float32)
-            k.out_norm_add(own, src, y, bias, norm.weight.tensor, norm.eps, norm.offset, hist=hist, n_hist=n + 1,
+            k.out_norm_add(own, src, y, bias, *self._norm(norm), hist=hist, n_hist=n + 1,
                            coef=self.coef.tensor, avg=go, cast=cast)
             stream.h, state["n"] = go, n + 1
         else:
-            k.out_norm_add(own, src, y, bias, norm.weight.tensor, norm.eps, norm.offset, cast=cast)
+            self._add(own, src, y, bias, norm, cast)
         state["x"] = cast if cast is not None else stream.h
         return stream
+
+    def _add(self, dst, src, y, bias, norm, cast) -> None:
+        """dst = src + norm(y + bias), or of a pair of outputs put together (base.NormedPair); `cast` gets it too."""
+        weight, eps, offset = self._norm(norm)
+        if isinstance(y, NormedPair):
+            self.ctx.kernels.out_norm_pair_add(dst, src, y, weight, eps, offset, cast=cast)
+        else:
+            self.ctx.kernels.out_norm_add(dst, src, y, bias, weight, eps, offset, cast=cast)
 
 
 class Sandwich(Part):

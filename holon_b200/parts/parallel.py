@@ -7,7 +7,9 @@ has one launch for its sum and the next layer's norm.
 
 `SideBySide`: a mixer made of two mixers that read the same input, result = left_scale · left + right_scale · right.
 At most one of the two may ask for a paged cache; their fixed-size states are kept under `left.` and `right.` names.
-Inside a `ParallelBlock` its two outputs go into the block's one sum as terms of their own.
+Inside a `ParallelBlock` its two outputs go into the block's one sum as terms of their own. With `out_eps` each output first
+passes an RMS norm over its row with a weight of its own (stored `left.out`, `right.out`), and the two scales are equal; an
+`OutNorm` block then takes both rows as they are (`pair_out`: base.NormedPair) and does everything up to the stream in one kernel.
 """
 from __future__ import annotations
 
@@ -16,20 +18,24 @@ import dataclasses
 import torch
 
 from ..config.spec import PartRef
-from .base import BuildContext, Part, Residual
+from .base import BuildContext, NormedPair, Part, Residual
 from .model import LayerCache
 
 
 class SideBySide(Part):
     def __init__(self, ctx: BuildContext, *, left: PartRef, right: PartRef, left_scale: float, right_scale: float,
-                 hidden: int, layer: int = 0) -> None:
+                 hidden: int, layer: int = 0, out_eps: float | None = None) -> None:
         super().__init__()
-        self.ctx = ctx
+        self.ctx, self.out_eps = ctx, out_eps
         self.left = self.add_child("left", ctx.part(left, layer=layer, hidden=hidden))
         self.right = self.add_child("right", ctx.part(right, layer=layer, hidden=hidden))
         self.scales = (float(left_scale), float(right_scale))
         if self.left.cache() is not None and self.right.cache() is not None:
             raise ValueError("side by side: only one of the two mixers may keep a paged cache")
+        if out_eps is not None:
+            if self.scales[0] != self.scales[1]:
+                raise ValueError("side by side: normed outputs go with equal scales")
+            self.out_gain = tuple(self.add_param(f"{side}.out", (hidden,), "gain") for side in ("left", "right"))
 
     def _sides(self):
         return (("left", self.left), ("right", self.right))
@@ -51,6 +57,16 @@ class SideBySide(Part):
 
     def terms(self, x: torch.Tensor, step, cache) -> list:
         """[(output, scale)] of the two mixers."""
+        if self.out_eps is not None:
+            return [(self.pair_out(x, step, cache).combined(), 1.0)]
+        return self._run(x, step, cache)
+
+    def pair_out(self, x: torch.Tensor, step, cache) -> NormedPair:
+        """The two outputs with the norms they have yet to pass (with `out_eps`)."""
+        (a, scale), (b, _) = self._run(x, step, cache)
+        return NormedPair(a, self.out_gain[0].tensor, b, self.out_gain[1].tensor, self.out_eps, scale)
+
+    def _run(self, x: torch.Tensor, step, cache) -> list:
         out = []
         for (side, part), scale in zip(self._sides(), self.scales):
             slots = {name[len(side) + 1:]: t for name, t in cache.slots.items() if name.startswith(side + ".")}
@@ -60,6 +76,8 @@ class SideBySide(Part):
         return out
 
     def forward(self, x: torch.Tensor, step, cache) -> torch.Tensor:
+        if self.out_eps is not None:
+            return self.pair_out(x, step, cache).combined()
         (a, sa), (b, sb) = self.terms(x, step, cache)
         return (sa * a.float() + sb * b.float()).to(a.dtype)
 

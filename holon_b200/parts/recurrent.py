@@ -36,6 +36,15 @@ all heads' channels, times sigmoid(W_g x), then W_o.
 projections, no rotation, no scale, o = Sᵀ q; all heads' o together under one RMS norm with a weight over all their channels,
 times sigmoid(W_g x), then W_o.
 
+`StateSpace`: a selective state space in its matrix form (Mamba-2). Per head with a rate exp(A_log), a skip D and a step size
+dt = softplus(its projection + dt_bias) per token, and B, C [state] shared by the heads of a group:
+
+    S ← exp(−exp(A_log) dt) S + dt B xᵀ,   y = Sᵀ C + D x.
+
+x, B and C pass one short causal convolution over time with a bias (its last taps − 1 inputs are carried per request) and silu;
+all heads' y times silu(z), then an RMS norm over each of `norm_groups` equal parts of the row with a weight over the whole of
+it, then W_o. dt is a factor on what the scan writes (`recurrent_scan(take=)`), D a skip in its read-out.
+
 Everything that enters the recurrence is 32-bit (the scan's inputs are made in 32-bit from the first product's rows);
 the products themselves are the engine's. All first projections of a mixer are one merged product.
 """
@@ -277,3 +286,53 @@ class GeneralDelta(_MatrixState):
         y = ctx.empty(t, heads, dim)
         k.head_norm_gate(y, o, self.gain.tensor, None, first[:, 3 * n:4 * n], self.eps, gate="sigmoid")
         return self.out.forward(y.view(t, n), link=take_link(step))
+
+
+class StateSpace(_MatrixState):
+    def __init__(self, ctx: BuildContext, *, heads: int, vdim: int, state: int, groups: int, taps: int, norm_groups: int, eps: float,
+                 hidden: int, layer: int = 0) -> None:
+        super().__init__()
+        if heads % groups:
+            raise ValueError(f"state space: {heads} heads are no multiple of {groups} groups")
+        if taps < 1:
+            raise ValueError("state space: the convolution has at least one tap")
+        if (heads * vdim) % norm_groups:
+            raise ValueError(f"state space: rows of {heads * vdim} numbers do not fall into {norm_groups} equal parts")
+        self.ctx, self.heads, self.vdim, self.state, self.groups = ctx, heads, vdim, state, groups
+        self.taps, self.norm_groups, self.eps = int(taps), int(norm_groups), float(eps)
+        self.inner = heads * vdim
+        self.channels = self.inner + 2 * groups * state                  # what passes the convolution: x | B | C
+        self.first = self.add_child("first", Linear(ctx, "weight", hidden, {"in": self.inner + self.channels + heads}))
+        self.conv = self.add_param("conv", (self.channels, taps), "matrix")
+        self.conv_bias = self.add_param("conv.b", (self.channels,), "matrix")
+        self.dt_bias = self.add_param("dt_bias", (heads,), "coef")
+        self.rate_log = self.add_param("A_log", (heads,), "coef")
+        self.skip = self.add_param("D", (heads,), "coef")
+        self.gain = self.add_param("norm", (self.inner,), "coef")
+        self.out = self.add_child("out", Linear(ctx, "weight", self.inner, {"o": hidden}))
+
+    def slot_states(self):
+        states = [SlotState("state", (self.heads, self.vdim, self.state))]
+        if self.taps > 1:
+            states.append(SlotState("conv", (self.taps - 1, self.channels), str(self.ctx.dtype).replace("torch.", "")))
+        return tuple(states)
+
+    def forward(self, x: torch.Tensor, step, cache) -> torch.Tensor:
+        t, k, ctx, f32 = x.shape[0], self.ctx.kernels, self.ctx, torch.float32
+        heads, vdim, inner = self.heads, self.vdim, self.inner
+        first = self.first.forward(x)                                    # [t, z | x | B | C | dt]
+        cb = ctx.empty(t, 2, self.groups, self.state, dtype=f32)         # C in the queries' place, B in the keys'
+        v = ctx.empty(t, heads, vdim, dtype=f32)
+        dt, decay = ctx.empty(t, heads, dtype=f32), ctx.empty(t, heads, dtype=f32)
+        carried = cache.slots.get("conv")
+        k.state_space_prepare(cb, v, dt, decay, first, inner, self.conv.tensor, self.conv_bias.tensor, carried,
+                              self.dt_bias.tensor, self.rate_log.tensor, step.rows)
+        if step.rows.n_rows > step.rows.n_decode:                        # (rows of one token: moved on by the kernel above)
+            k.conv_carry(carried, first, self.channels, self.taps, step.rows, least=2, at=inner)
+        y = ctx.empty(t, heads, vdim, dtype=f32)
+        k.recurrent_scan(y, cb, v, None, None, None, cache.slots["state"], step.rows, token_decay=decay, take=dt,
+                         skip=self.skip.tensor)
+        n = self.norm_groups
+        out = ctx.empty(t, n, inner // n)
+        k.head_norm_gate(out, y.view(t, n, inner // n), self.gain.tensor, None, first[:, :inner], self.eps, gate_first=True)
+        return self.out.forward(out.view(t, inner))

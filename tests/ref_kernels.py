@@ -127,7 +127,7 @@ class RefKernels:
         x = table[ids.long()].float() * scale
         for b in range(rows.n_rows):
             for t in range(qs[b], qs[b + 1]):
-                before = ids_[t - 1] if t > qs[b] else int(prev[slots[b]])
+                before = ids_[t - 1] if t > qs[b] else int(prev[slots[b]]) if prev is not None else 0
                 if pair is not None:
                     r = buckets if pos[t] == 0 else (before * mul_prev + ids_[t] * mul_cur) % buckets
                     x[t] += pair[r].float()
@@ -157,7 +157,7 @@ class RefKernels:
         g, u = g.clamp(max=limit), u.clamp(-limit, limit)
         out.copy_((g * torch.sigmoid(alpha * g) * (u + 1)).to(out.dtype))
 
-    def recurrent_scan(self, out, qk, v, decay, head_decay, beta, state, rows, token_decay=None, rate=None):
+    def recurrent_scan(self, out, qk, v, decay, head_decay, beta, state, rows, token_decay=None, rate=None, take=None, skip=None):
         t, heads, vdim = v.shape
         group = heads // qk.shape[2]
         qs, slots = rows.query_start.tolist(), rows.row_slot.tolist()
@@ -173,8 +173,10 @@ class RefKernels:
                     s = s * (decay[i, h][:, None] if decay is not None else
                              token_decay[i, h] if token_decay is not None else head_decay[h])
                     u = v[i, h] if beta is None else beta[i, h] * (v[i, h] - s.T @ k)
+                    if take is not None:                       # a factor per head and token on what is written
+                        u = u * take[i, h]
                     s = s + torch.outer(k, u)
-                    out[i, h] = s.T @ q
+                    out[i, h] = s.T @ q + (skip[h] * v[i, h] if skip is not None else 0.0)
                 state[slots[b], h] = s.T
 
     def delta_prepare(self, qk, v, beta, decay, gate, first, conv, conv_state, low2, dt_bias, rate_log, rows, q_scale,
@@ -206,14 +208,36 @@ class RefKernels:
         decay.copy_(torch.exp(-torch.exp(rate_log)[None, :, None] * torch.nn.functional.softplus(a).view(t, heads, dim)))
         gate.copy_(torch.sigmoid(low2[:, heads * dim:]).view(gate.shape))
 
-    def conv_carry(self, conv_state, first, channels, taps, rows, least=0):
+    def state_space_prepare(self, cb, v, dt, decay, first, at, conv, conv_bias, conv_state, dt_bias, rate_log, rows):
+        t, heads, vdim = v.shape
+        groups, n = cb.shape[2], cb.shape[3]
+        channels, taps = conv.shape
+        x = first[:, at:at + channels]
+        y = torch.zeros(t, channels)
+        qs, slots = rows.query_start.tolist(), rows.row_slot.tolist()
+        for b in range(rows.n_rows):
+            s, e = qs[b], qs[b + 1]
+            carried = conv_state[slots[b]] if taps > 1 else x[:0]
+            seq = torch.cat((carried, x[s:e]), 0)
+            y[s:e] = sum(seq[j:j + e - s].float() * conv.float()[:, j] for j in range(taps)) + conv_bias.float()
+            if taps > 1 and e - s == 1:
+                conv_state[slots[b]] = seq[-(taps - 1):]
+        y = y * torch.sigmoid(y)
+        inner, gn = heads * vdim, groups * n
+        v.copy_(y[:, :inner].view(t, heads, vdim))
+        cb[:, 1] = y[:, inner:inner + gn].view(t, groups, n)
+        cb[:, 0] = y[:, inner + gn:].view(t, groups, n)
+        dt.copy_(torch.nn.functional.softplus(first[:, at + channels:].float() + dt_bias))
+        decay.copy_(torch.exp(-torch.exp(rate_log) * dt))
+
+    def conv_carry(self, conv_state, first, channels, taps, rows, least=0, at=0):
         if taps <= 1:
             return
         qs, slots = rows.query_start.tolist(), rows.row_slot.tolist()
         for b in range(rows.n_rows):
             if qs[b + 1] - qs[b] < least:
                 continue
-            seq = torch.cat((conv_state[slots[b]], first[qs[b]:qs[b + 1], :channels]), 0)
+            seq = torch.cat((conv_state[slots[b]], first[qs[b]:qs[b + 1], at:at + channels]), 0)
             conv_state[slots[b]] = seq[-(taps - 1):]
 
     def retention_prepare(self, qk, v, first, positions, table, rot_dims, k_scale, silu=False):
@@ -229,7 +253,10 @@ class RefKernels:
             qk[:, which] = z * (k_scale if which else 1.0)
         v.copy_(x[:, 2 * heads * dim:2 * heads * dim + heads * vdim].view(t, heads, vdim))
 
-    def head_norm_gate(self, out, o, weight, gate_mul, gate_pre, eps, gate="silu"):
+    def head_norm_gate(self, out, o, weight, gate_mul, gate_pre, eps, gate="silu", gate_first=False):
+        if gate_first:                                         # the gate is part of what is normed
+            g = gate_pre.float().reshape(o.shape)
+            o, gate_pre = o * (g * torch.sigmoid(g) if gate == "silu" else torch.sigmoid(g)), None
         y = o * torch.rsqrt((o * o).mean(-1, keepdim=True) + eps)
         if weight is not None:                                 # one weight for all heads, or one per head and channel
             y = y * (weight.view(o.shape[1:]) if weight.numel() == o.shape[1] * o.shape[2] else weight)
@@ -496,6 +523,69 @@ class RefKernels:
             avg.copy_(go)
         if cast is not None:
             cast.copy_(go.to(cast.dtype))
+
+    def out_norm_pair_add(self, dst, src, pair, weight, eps, offset, cast=None):
+        unit = lambda y, e: y.float() * torch.rsqrt((y.float() ** 2).mean(-1, keepdim=True) + e)      # noqa: E731
+        z = pair.scale * (unit(pair.a, pair.eps) * pair.a_weight.float() + unit(pair.b, pair.eps) * pair.b_weight.float())
+        self.out_norm_add(dst, src, z, None, weight, eps, offset, cast=cast)
+
+    # ---- attention with one or two maps a head
+    def qkv_maps_prepare(self, q_out, kv, first, q_weight, k_weight, eps, norm, positions, table, rot_dims, write_index, kv_heads,
+                         value_dim):
+        t, heads, maps, dim = q_out.shape
+        nq, nk, nv = heads * maps * dim, kv_heads * maps * dim, kv_heads * value_dim
+        x = first.float()
+
+        def prepare(u, weight):
+            if norm == "before":
+                u = u * torch.rsqrt((u * u).mean(-1, keepdim=True) + eps) * weight.float()
+            if rot_dims:
+                u = self._turn(u, table[positions.long()][:, None, None, :], rot_dims)
+            if norm == "after":
+                u = u * torch.rsqrt((u * u).mean(-1, keepdim=True) + eps)
+            return u
+
+        q_out.copy_(prepare(x[:, :nq].view(t, heads, maps, dim), q_weight).to(q_out.dtype))
+        if kv is not None:
+            k = prepare(x[:, nq:nq + nk].view(t, kv_heads, maps, dim), k_weight).reshape(t, kv_heads, maps * dim)
+            v = x[:, nq + nk:nq + nk + nv].view(t, kv_heads, value_dim)
+            page, w = kv.shape[2], write_index.long()
+            rows = torch.cat((k, v), dim=-1).to(kv.dtype)
+            for i in torch.nonzero((w >= 0) & (w < (kv.shape[0] - 1) * page)).flatten().tolist():
+                kv[int(w[i]) // page, :, int(w[i]) % page] = rows[i]
+
+    def attention_maps(self, out, q, kv, block_table, rows, scale, cap, window, keep_first, diff, eps, gate):
+        t, heads, maps, dim = q.shape
+        vd, kvh, page = out.shape[2], kv.shape[1], kv.shape[2]
+        null = kv.shape[0] - 1
+        qs, slots, lens = rows.query_start.tolist(), rows.row_slot.tolist(), rows.kv_len.tolist()
+        for b in range(rows.n_rows):
+            n, s, e = lens[b], qs[b], qs[b + 1]
+            if e == s:
+                continue
+            pages = block_table[slots[b], :-(-n // page)].long()
+            held = kv[pages].float().permute(1, 0, 2, 3).reshape(kvh, -1, kv.shape[3])[:, :n]      # [kvh, n, maps dim + vd]
+            gone = (pages == null).repeat_interleave(page)[:n]
+            pos, key = torch.arange(n - (e - s), n)[:, None], torch.arange(n)[None]
+            hidden = key > pos
+            if window > 0:
+                hidden = hidden | ((pos - key >= window) & (key >= keep_first))
+            assert not (~hidden & gone[None]).any(), "a visible key lies in a page that was given back"
+            for h in range(heads):
+                rows_g = held[h // (heads // kvh)]
+                o = []
+                for m in range(maps):
+                    sc = (q[s:e, h, m].float() @ rows_g[:, m * dim:(m + 1) * dim].T) * scale
+                    if cap:
+                        sc = cap * torch.tanh(sc / cap)
+                    o.append(torch.softmax(sc.masked_fill(hidden, float("-inf")), -1) @ rows_g[:, maps * dim:])
+                y = o[0]
+                if diff is not None:
+                    y = o[0] - diff[0] * o[1]
+                    y = y * torch.rsqrt((y * y).mean(-1, keepdim=True) + eps) * (1.0 - diff[1])
+                if gate is not None:
+                    y = y * torch.sigmoid(gate[s:e, h * vd:(h + 1) * vd].float())
+                out[s:e, h] = y.to(out.dtype)
 
     # ---- attention whose heads share their weights after the softmax
     def qkv_talking_prepare(self, q_out, kv, keep, qkv, bias, q_weight, k_weight, eps, positions, table, rot_dims, interleaved,
