@@ -37,41 +37,6 @@
 #define AT_MMA_WARP1 10                            // warps 10, 11: the groups' P V issuing warps; warps 2-9 are the softmax
 #define AT_THREADS 384
 
-__device__ __forceinline__ float at_ex2(float x) {
-    float y;
-    asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
-    return y;
-}
-__device__ __forceinline__ void tc_mma_f16(uint32_t tmem_d, uint64_t desc_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
-    asm volatile("{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
-                 "tcgen05.mma.cta_group::1.kind::f16 [%0], %1, %2, %3, p;\n\t}\n"
-                 ::"r"(tmem_d), "l"(desc_a), "l"(desc_b), "r"(idesc), "r"(accumulate) : "memory");
-}
-
-// Two float32 in one 64-bit register, for the packed arithmetic of sm_100 (one instruction, two results).
-__device__ __forceinline__ uint64_t pack2(float lo, float hi) {
-    uint64_t r;
-    asm("mov.b64 %0, {%1, %2};\n" : "=l"(r) : "f"(lo), "f"(hi));
-    return r;
-}
-__device__ __forceinline__ void unpack2(uint64_t v, float& lo, float& hi) { asm("mov.b64 {%0, %1}, %2;\n" : "=f"(lo), "=f"(hi) : "l"(v)); }
-__device__ __forceinline__ uint64_t fma2(uint64_t a, uint64_t b, uint64_t c) {
-    uint64_t d;
-    asm("fma.rn.f32x2 %0, %1, %2, %3;\n" : "=l"(d) : "l"(a), "l"(b), "l"(c));
-    return d;
-}
-__device__ __forceinline__ uint64_t add2(uint64_t a, uint64_t b) {
-    uint64_t d;
-    asm("add.rn.f32x2 %0, %1, %2;\n" : "=l"(d) : "l"(a), "l"(b));
-    return d;
-}
-// The same with the A operand in tensor memory (128 lanes x K/2 columns, two bfloat16 per column).
-__device__ __forceinline__ void tc_mma_f16_ts(uint32_t tmem_d, uint32_t tmem_a, uint64_t desc_b, uint32_t idesc, uint32_t accumulate) {
-    asm volatile("{\n\t.reg .pred p;\n\tsetp.ne.b32 p, %4, 0;\n\t"
-                 "tcgen05.mma.cta_group::1.kind::f16 [%0], [%1], %2, %3, p;\n\t}\n"
-                 ::"r"(tmem_d), "r"(tmem_a), "l"(desc_b), "r"(idesc), "r"(accumulate) : "memory");
-}
-
 // Two groups of 128 queries share the CTA's key and value tiles; each has its own softmax warps (2-5 and 6-9), its own
 // S, P and O, so that one group's softmax runs while the tensor cores work for the other.
 __global__ void __launch_bounds__(AT_THREADS, 1) prefill_tcgen05_kernel(
@@ -194,7 +159,7 @@ __global__ void __launch_bounds__(AT_THREADS, 1) prefill_tcgen05_kernel(
 #pragma unroll
                         for (int kk = 0; kk < AT_D / 16; ++kk) {      // d 0..63 in the first block, 64..127 in the second
                             const uint32_t blk = kk >> 2, within = (kk & 3) * 2;
-                            tc_mma_f16(s_t, tc_smem_desc(q_s + g * AT_Q_BYTES + blk * (AT_Q_BYTES / 2)) + within,
+                            tc_mma(s_t, tc_smem_desc(q_s + g * AT_Q_BYTES + blk * (AT_Q_BYTES / 2)) + within,
                                        tc_smem_desc(k_src + blk * (AT_KV_BYTES / 2)) + within, idesc_qk, kk != 0);
                         }
                         tc_commit(s_full0 + 8 * gb);

@@ -7,6 +7,7 @@
 #include "tcgen05.cuh"
 
 extern "C" int hb_attention_tcgen05_status_mirror(unsigned int* word);
+extern "C" int hb_attention_maps_status_mirror(unsigned int* word);
 extern "C" int hb_gemm_tcgen05_status_mirror(unsigned int* word);
 extern "C" int hb_gemm_tcgen05_pair_status_mirror(unsigned int* word);
 extern "C" int hb_gemm_chain_status_mirror(unsigned int* word);
@@ -31,7 +32,7 @@ extern "C" int hb_status_word(unsigned int** host) {
         if (hb_attention_tcgen05_status_mirror(device) || hb_gemm_tcgen05_status_mirror(device) ||
             hb_gemm_tcgen05_pair_status_mirror(device) || hb_gemm_chain_status_mirror(device) ||
             hb_gemm_tickets_status_mirror(device) || hb_gemm_mid_status_mirror(device) ||
-            hb_experts_tcgen05_status_mirror(device) ||
+            hb_experts_tcgen05_status_mirror(device) || hb_attention_maps_status_mirror(device) ||
             hb_status_selftest_mirror(device))
             return HB_ERR_CUDA;
         g_word_host = word;

@@ -770,7 +770,7 @@ class CudaKernels:
         up their barrier and flags are put back to zero, so that the next launch starts clean."""
         out = 0
         for name in ("hb_gemm_tcgen05_status", "hb_gemm_tcgen05_pair_status", "hb_attention_tcgen05_status",
-                     "hb_gemm_chain_status", "hb_gemm_tickets_status", "hb_gemm_mid_status", "hb_experts_tcgen05_status"):
+                     "hb_gemm_chain_status", "hb_gemm_tickets_status", "hb_gemm_mid_status", "hb_experts_tcgen05_status", "hb_attention_maps_status"):
             status = ctypes.c_uint(0)
             if getattr(self.lib, name)(ctypes.byref(status)):
                 raise KernelError(self.lib.hb_last_error().decode())
@@ -1389,17 +1389,17 @@ class CudaKernels:
         head = (self._p(out), self._p(q), self._p(kv))
         fast = q.dtype == torch.bfloat16 and self.attention_bf16 == "fast"
         ones, portions = rows.n_decode, rows.n_rows > rows.n_decode
-        decode = fast and dim % 8 == 0 and vd % 8 == 0 and maps * dim <= 256 and vd <= 256
-        if not decode and not (fast and portions and self._maps_tcgen05(dim, vd, page)):
+        tiles16 = fast and self.prefill_attention == "tcgen05" and dim % 16 == 0 and vd % 16 == 0 and max(dim, vd) <= 128 and page % 64 == 0
+        if not (fast and dim % 8 == 0 and vd % 8 == 0 and max(maps * dim, vd) <= 256) or (portions and not tiles16):
             return self._call("hb_attention_maps", *head, _code(q), *common, rows.n_rows, t, *sizes, *rules)
-        if ones and decode:
+        if ones:
             self._call("hb_attention_maps_decode", *head, *common, ones, *sizes, *rules,
                        self._maps_splits(ones, heads // kv_heads, kv_heads, maps, rows.max_kv, window, keep_first))
         if portions:
-            self._call("hb_attention_maps", *head, _code(q), *common, rows.n_rows, t, *sizes, *rules)
-
-    def _maps_tcgen05(self, dim: int, vd: int, page: int) -> bool:
-        return False
+            tile_q, tiles = 128, self._query_tiles(rows, 128)
+            if maps == 1 and self.prefill_tile != 128 and (self.prefill_tile == 256 or 4 * heads * self._query_tiles(rows, 256) >= 3 * self.sms):
+                tile_q, tiles = 256, self._query_tiles(rows, 256)     # (fewer tiles would leave SMs idle)
+            self._call("hb_attention_maps_prefill", *head, *common, ones, rows.n_rows, tiles, t, *sizes, *rules, tile_q)
 
     def _maps_splits(self, rows: int, group: int, kv_heads: int, maps: int, max_kv: int, window: int, keep: int) -> int:
         """Parts a one-token row's keys are cut into: enough for two CTAs an SM, each part at least one tile of 64 keys. A
