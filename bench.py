@@ -201,6 +201,34 @@ GEGUNEX_SIZES = {
 }
 
 
+def bukuvik_config(width: int, heads: int, kv_heads: int, map_dim: int, dim: int, vdim: int, window: int, keep: int, ff: int,
+                   state_heads: int, groups: int, state: int, state_vdim: int, layers: int, taps: int = 4, vocab: int = 32768) -> dict:
+    """A Bukuvik model for `--only bukuvik`: of every three layers two are parallel ones (attention over a window that keeps the
+    first tokens beside a state space) and the third differential attention; dense squared-relu feed-forwards."""
+    two_maps = {"heads": heads, "kv_heads": kv_heads, "dim": map_dim, "vdim": vdim, "scale": map_dim ** -0.5, "softcap": 50.0,
+                "diff": 0.5, "mask": {"size": window}, "rot": {"base": 1000000.0, "dims": map_dim // 2}}
+    left = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": vdim, "scale": dim ** -0.5, "mask": {"size": window, "keep_first": keep},
+            "rot": {"base": 1000000.0, "dims": dim, "scaling": {"factor": 16.0, "original": 4096, "fast": 32.0, "slow": 1.0}}}
+    right = {"heads": state_heads, "groups": groups, "state": state, "vdim": state_vdim, "conv": taps, "norm_groups": groups}
+    mlp = {"kind": "dense", "ff": ff}
+    parallel = {"type": "parallel", "mixer": {"left": left, "right": right}, "mlp": mlp}
+    listed = [{"type": "attention", "mixer": two_maps, "mlp": mlp} if i % 3 == 2 else parallel for i in range(layers)]
+    return {"architecture": "Bukuvik", "width": width, "vocab": vocab, "norm": {"eps": 1e-6}, "residual_mult": 0.5,
+            "embedding": {"scale": width ** 0.5}, "layers": listed}
+
+
+# Layers of the sizes of published decoders of 1.5 and 8 billion parameters (as Kasovik's, the ungated feed-forward as large as its
+# gated one), maps of 64 over values of 128, a state space as wide as the model (heads of 64 over a state of 128), windows of 1,024
+# and 2,048 tokens that keep the first 16. Beside each the Kasovik model of `KASOVIK_SIZES` (windowed attention beside a matrix state:
+# the closest design here) and the Qwen3 decoder of the same width, heads, key heads and layers.
+BUKUVIK_SIZES = {
+    "base": (dict(width=2048, heads=16, kv_heads=4, map_dim=64, dim=128, vdim=128, window=1024, keep=16, ff=9216, state_heads=32,
+                  groups=4, state=128, state_vdim=64, layers=6), "base"),
+    "wide": (dict(width=4096, heads=32, kv_heads=8, map_dim=64, dim=128, vdim=128, window=2048, keep=16, ff=18432, state_heads=64,
+                  groups=8, state=128, state_vdim=64, layers=6), "wide"),
+}
+
+
 def _find_number(data, key: str):
     """The first number stored under `key` anywhere in a nested JSON value (a dict under the key: its "value")."""
     if isinstance(data, dict):
@@ -679,6 +707,13 @@ def gegunex_run(args) -> dict:
     return beside_qwen3(args, "gegunex", table, gegunex_config, args.gegunex_sizes)
 
 
+def bukuvik_run(args) -> dict:
+    """The same for Bukuvik beside the Kasovik model and the Qwen3 decoder of the same width, heads, key heads and layers."""
+    table = {name: (ours, KASOVIK_SIZES[like][1], {"kasovik": kasovik_config(**KASOVIK_SIZES[like][0])})
+             for name, (ours, like) in BUKUVIK_SIZES.items()}
+    return beside_qwen3(args, "bukuvik", table, bukuvik_config, args.bukuvik_sizes)
+
+
 def beside_qwen3(args, design: str, table: dict, make_config, chosen: str, context: int = 2048) -> dict:
     import gc
     import torch
@@ -831,6 +866,8 @@ def run_ours(args) -> dict:
         return vobosun_run(args)
     if args.only == "gegunex":
         return gegunex_run(args)
+    if args.only == "bukuvik":
+        return bukuvik_run(args)
     cfg = dict(QWEN3_8B, num_hidden_layers=args.layers)
     context, batch = args.context, args.batch
     engine = Engine(EngineConfig(model="random weights, seed 2", device="cuda:0", dtype="bfloat16", page_size=64,
@@ -953,7 +990,7 @@ def main() -> int:
                          "several passes should hold a few GB only (e.g. 0.03 with --layers 4 --batch 8)")
     ap.add_argument("--batch", type=int, default=8)
     ap.add_argument("--context", type=int, default=8192)
-    ap.add_argument("--only", default="all", choices=("all", "decode", "prefill", "long_prompt", "sizes", "shared_prompt", "rulorax", "kasovik", "tilarax", "vobosun", "gegunex"),
+    ap.add_argument("--only", default="all", choices=("all", "decode", "prefill", "long_prompt", "sizes", "shared_prompt", "rulorax", "kasovik", "tilarax", "vobosun", "gegunex", "bukuvik"),
                     help="run one part only (for profiling a small case); the JSON line then lacks the other parts. "
                          "long_prompt: time to first token of a 30,000-token prompt behind three decoding requests; "
                          "sizes: the workloads of the Qwen3-32B and Qwen3-0.6B configurations (--sizes); "
@@ -965,6 +1002,7 @@ def main() -> int:
     ap.add_argument("--tilarax-sizes", default="", help="with --only tilarax: which sizes (base, wide; default both)")
     ap.add_argument("--vobosun-sizes", default="", help="with --only vobosun: which sizes (base, wide; default both)")
     ap.add_argument("--gegunex-sizes", default="", help="with --only gegunex: which sizes (base, wide; default both)")
+    ap.add_argument("--bukuvik-sizes", default="", help="with --only bukuvik: which sizes (base, wide; default both)")
     ap.add_argument("--no-points", action="store_true", help="leave out the points at other batch sizes and contexts")
     ap.add_argument("--no-kernels", action="store_true", help="leave out the per-kernel table")
     args = ap.parse_args()

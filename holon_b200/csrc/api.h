@@ -238,7 +238,8 @@ int hb_dyt_shift(void* out, int out_dtype, float* into, const float* h, const vo
 
 // bfloat16 product for at most 16 rows of x, bound by reading w once. mode 0: out [m, n] (bfloat16, or float32 when
 // out_f32) = x [m, k] · w [n, k]ᵀ. mode 1: w is [2 inter, k], gate rows first; out [m, inter] = silu(x · gateᵀ) ·
-// (x · upᵀ). k a multiple of 8; pointers 16-byte aligned.
+// (x · upᵀ). mode 5: mode 0 under a squared relu, max(., 0)^2. k a multiple of 8; pointers 16-byte aligned. (Modes 0, 1 and 5 are
+// those of the tcgen05 products below too.)
 int hb_gemm_bf16_skinny(void* out, int out_f32, const void* x, const void* w, int m, int n, int k, int mode, int inter,
                         hb_stream stream);
 
@@ -435,6 +436,14 @@ int hb_state_space_prepare(float* cb, float* v, float* dt, float* decay, const v
                            const void* conv, const void* conv_bias, int taps, void* conv_state, const float* dt_bias,
                            const float* rate_log, const int32_t* query_start, const int32_t* row_slot, int rows, int tokens,
                            int heads, int vdim, int groups, int n, hb_stream stream);
+// The state-space recurrence for rows row0 .. rows - 1, in chunks of 64 tokens (csrc/state_space.cu), all 32-bit: S <- exp(-exp(
+// rate_log[h]) dt) S + dt B x^T, y = S^T C + skip[h] x, with cb [tokens, 2, groups, n] = (C, B), x [tokens, heads, vdim], dt [tokens,
+// heads], state [slots, heads, vdim, n] read at a row's start and written at its end. tiles: at least the sum over the rows of
+// ceil(tokens / 64); scratch: hb_state_space_prompt_scratch_floats(tiles, ...) floats on a 16-byte boundary.
+size_t hb_state_space_prompt_scratch_floats(int tiles, int heads, int groups, int n, int vdim);
+int hb_state_space_prompt(float* y, const float* cb, const float* x, const float* dt, const float* rate_log, const float* skip,
+                          float* state, float* scratch, const int32_t* query_start, const int32_t* row_slot, int row0, int rows,
+                          int tiles, int heads, int groups, int n, int vdim, hb_stream stream);
 
 // ---- the matrix memory with exponential gates (csrc/mlstm.cu): the kernels around hb_recurrent_scan with token_decay.
 // pre [tokens, ld] 32-bit: the input gate's pre-activations of the heads, then the forget gate's; bias [2 heads] likewise.

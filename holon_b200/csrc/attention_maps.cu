@@ -26,7 +26,7 @@ __device__ __forceinline__ float mp_sigmoid(float x) { return 1.f / (1.f + expf(
 // `table` holds, per position, the rot_dims / 2 cosines and then the sines. One rounding, at the end. PAIR: a lane owns runs of
 // two neighbouring channels (dim, vdim, the rows and the cache even), else every 32nd channel.
 #define MP_WARPS 4
-#define MP_PER_LANE 16            // sizes up to 512
+#define MP_PER_LANE 16            // sizes up to 512 (PL: numbers a lane holds, 4 for sizes up to 128)
 template <typename T> struct Two;
 template <> struct Two<float> {
     static __device__ __forceinline__ float2 load(const float* p) { return *(const float2*)p; }
@@ -37,19 +37,18 @@ template <> struct Two<bf16> {
     static __device__ __forceinline__ void store(bf16* p, float a, float b) { *(__nv_bfloat162*)p = __floats2bfloat162_rn(a, b); }
 };
 
-template <typename T, bool PAIR>
+template <typename T, bool PAIR, int PL>
 __global__ void maps_prepare_kernel(T* __restrict__ q_out, T* __restrict__ kv, const T* __restrict__ first, long ld,
                                     const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps, int norm,
                                     const int32_t* __restrict__ positions, const float* __restrict__ table, int rot_dims,
                                     int table_rows, const int32_t* __restrict__ write_index, int pages, int page_size,
-                                    long items, int heads, int kv_heads, int maps, int dim, int vdim) {
+                                    int heads, int kv_heads, int maps, int dim, int vdim) {
     extern __shared__ __align__(16) float mp_smem[];
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int nq = heads * maps, nk = kv_heads * maps, slots = nq + nk + kv_heads;
-    const long item = (long)blockIdx.x * MP_WARPS + warp;
-    if (item >= items) return;
-    const long t = item / slots;
-    const int slot = (int)(item - t * slots);
+    const long t = blockIdx.x;
+    const int slot = (int)blockIdx.y * MP_WARPS + warp;
+    if (slot >= slots) return;
     const int rowlen = maps * dim + vdim;
     const long w = write_index ? write_index[t] : -1;
     const bool stored = w >= 0 && w < (long)pages * page_size;
@@ -78,11 +77,11 @@ __global__ void maps_prepare_kernel(T* __restrict__ q_out, T* __restrict__ kv, c
     if (!dst) return;
     const float* weight = is_q ? q_weight : k_weight;
     float* ys = mp_smem + (size_t)warp * ((dim + 3) & ~3);
-    float x[MP_PER_LANE];
+    float x[PL];
     auto at = [&](int i) -> int { return PAIR ? 2 * lane + 64 * (i >> 1) + (i & 1) : lane + 32 * i; };
     float ss = 0.f;
 #pragma unroll
-    for (int i = 0; i < MP_PER_LANE; i += PAIR ? 2 : 1) {
+    for (int i = 0; i < PL; i += PAIR ? 2 : 1) {
         const int d = at(i);
         if (PAIR) {
             const float2 v = d < dim ? Two<T>::load(src + d) : make_float2(0.f, 0.f);
@@ -96,7 +95,7 @@ __global__ void maps_prepare_kernel(T* __restrict__ q_out, T* __restrict__ kv, c
     if (norm == 1) {
         const float r = rsqrtf(warp_sum(ss) / (float)dim + eps);
 #pragma unroll
-        for (int i = 0; i < MP_PER_LANE; ++i) { const int d = at(i); if (d < dim) x[i] *= r * weight[d]; }
+        for (int i = 0; i < PL; ++i) { const int d = at(i); if (d < dim) x[i] *= r * weight[d]; }
     }
     if (rot_dims) {
         int pos = positions[t];
@@ -104,11 +103,11 @@ __global__ void maps_prepare_kernel(T* __restrict__ q_out, T* __restrict__ kv, c
         const float* cs = table + (size_t)pos * rot_dims;
         const int half = rot_dims >> 1;
 #pragma unroll
-        for (int i = 0; i < MP_PER_LANE; ++i) { const int d = at(i); if (d < rot_dims) ys[d] = x[i]; }
+        for (int i = 0; i < PL; ++i) { const int d = at(i); if (d < rot_dims) ys[d] = x[i]; }
         __syncwarp();
         ss = 0.f;
 #pragma unroll
-        for (int i = 0; i < MP_PER_LANE; ++i) {
+        for (int i = 0; i < PL; ++i) {
             const int d = at(i);
             if (d < rot_dims) {
                 const bool lead = d < half;                           // u of the pair (u, v), or v
@@ -122,10 +121,10 @@ __global__ void maps_prepare_kernel(T* __restrict__ q_out, T* __restrict__ kv, c
     if (norm == 2) {
         const float r = rsqrtf(warp_sum(ss) / (float)dim + eps);
 #pragma unroll
-        for (int i = 0; i < MP_PER_LANE; ++i) x[i] *= r;
+        for (int i = 0; i < PL; ++i) x[i] *= r;
     }
 #pragma unroll
-    for (int i = 0; i < MP_PER_LANE; i += PAIR ? 2 : 1) {
+    for (int i = 0; i < PL; i += PAIR ? 2 : 1) {
         const int d = at(i);
         if (d < dim) { if (PAIR) Two<T>::store(dst + d, x[i], x[i + 1]); else dst[d] = from_f32<T>(x[i]); }
     }
@@ -141,22 +140,21 @@ extern "C" int hb_qkv_maps_prepare(void* q_out, void* kv, const void* first, int
     if (rot_dims && (!table || table_rows < 1)) HB_REFUSE("qkv_maps_prepare: a rotation needs its table");
     if (norm < 0 || norm > 2 || (norm == 1 && (!q_weight || !k_weight))) HB_REFUSE("qkv_maps_prepare: norm %d needs both weights", norm);
     if (maps < 1 || kv_heads < 1 || heads % kv_heads) HB_REFUSE("qkv_maps_prepare: %d heads, %d kv heads, %d maps", heads, kv_heads, maps);
-    const long items = (long)tokens * (heads * maps + kv_heads * maps + kv_heads);
-    const long blocks = (items + MP_WARPS - 1) / MP_WARPS;
-    if (blocks > 0x7fffffffL) HB_REFUSE("qkv_maps_prepare: %d tokens", tokens);
+    const long slots = (long)heads * maps + (long)kv_heads * maps + kv_heads;
+    if (slots > 65535L * MP_WARPS) HB_REFUSE("qkv_maps_prepare: %ld heads a token", slots);
+    const dim3 grid(tokens, (unsigned)((slots + MP_WARPS - 1) / MP_WARPS));
     const size_t smem = (size_t)MP_WARPS * ((dim + 3) & ~3) * sizeof(float);
     cudaStream_t s = (cudaStream_t)stream;
     const size_t two = dtype == HB_F32 ? 8 : 4;
     const bool pair = dim % 2 == 0 && vdim % 2 == 0 && ld % 2 == 0 && (((uintptr_t)q_out | (uintptr_t)kv | (uintptr_t)first) % two) == 0;
 #define HB_ARGS(T) (T*)q_out, (T*)kv, (const T*)first, ld, q_weight, k_weight, eps, norm, positions, table, rot_dims, table_rows, \
-    write_index, pages, page_size, items, heads, kv_heads, maps, dim, vdim
-    if (dtype == HB_F32) {
-        if (pair) maps_prepare_kernel<float, true><<<(unsigned)blocks, MP_WARPS * 32, smem, s>>>(HB_ARGS(float));
-        else maps_prepare_kernel<float, false><<<(unsigned)blocks, MP_WARPS * 32, smem, s>>>(HB_ARGS(float));
-    } else if (dtype == HB_BF16) {
-        if (pair) maps_prepare_kernel<bf16, true><<<(unsigned)blocks, MP_WARPS * 32, smem, s>>>(HB_ARGS(bf16));
-        else maps_prepare_kernel<bf16, false><<<(unsigned)blocks, MP_WARPS * 32, smem, s>>>(HB_ARGS(bf16));
-    } else HB_REFUSE("qkv_maps_prepare: dtype %d", dtype);
+    write_index, pages, page_size, heads, kv_heads, maps, dim, vdim
+#define HB_RUN(T, P) do { if (dim <= 128) maps_prepare_kernel<T, P, 4><<<grid, MP_WARPS * 32, smem, s>>>(HB_ARGS(T)); \
+                          else maps_prepare_kernel<T, P, MP_PER_LANE><<<grid, MP_WARPS * 32, smem, s>>>(HB_ARGS(T)); } while (0)
+    if (dtype == HB_F32) { if (pair) HB_RUN(float, true); else HB_RUN(float, false); }
+    else if (dtype == HB_BF16) { if (pair) HB_RUN(bf16, true); else HB_RUN(bf16, false); }
+    else HB_REFUSE("qkv_maps_prepare: dtype %d", dtype);
+#undef HB_RUN
 #undef HB_ARGS
     HB_LAUNCH_CHECK("qkv_maps_prepare");
     return 0;
@@ -298,7 +296,8 @@ extern "C" int hb_attention_maps(void* out, const void* q, const void* kv, int d
 // mma.sync m16n8k16 holds 16 / maps heads of the kv head's group for each map: the query of map m lies in the columns of that
 // map's key and the rest of its row is zero, so one product over the whole key row [key 1 | key 2] scores every map, and the
 // 16 rows share one sweep over the values. The parts' CTAs form a cluster; after a barrier each takes a share of the heads,
-// merges the parts through distributed shared memory and does the heads' epilogue, a warp a head.
+// merges the parts through distributed shared memory and does the heads' epilogue.
+#define MD_PARTS 8                 // parts a row's keys are cut into at most
 struct MapsArgs {
     bf16* out;
     const bf16* q;
@@ -326,27 +325,37 @@ __device__ __forceinline__ void load_maps_tile(uint32_t k_s, uint32_t v_s, const
     if (c >= want) return;                                    // (columns no product reads)
     const int x = (is_k ? 0 : kd) + c * 8;
     const uint32_t base = is_k ? k_s : v_s;
-    const bool in_page = a.page_shift >= 6;
+    const int j0 = tile * TILE_N;
+    if (a.page_shift >= 6) {                                  // the tile lies in one page: its rows follow one another
+        const bool page_ok = page_of_tile >= 0 && page_of_tile < a.pages && c < have;
+        const bool whole = j0 >= lo && j0 + TILE_N <= n;      // no key of the tile is outside the row's range
+        const bf16* src = a.kv + (((long)(page_ok ? page_of_tile : 0) * a.kv_heads + hk) * a.page_size + (j0 & (a.page_size - 1))) * rowlen + (page_ok ? x : 0);
+#pragma unroll
+        for (int r = r0; r < TILE_N; r += STEP) {
+            const int j = j0 + r;
+            const bool ok = page_ok && (whole || (j < n && (j >= lo || j < keep)));
+            cp_async16(base + (is_k ? tile_off<KP>(r, c) : tile_off<VP>(r, c)), src + (ok ? r * rowlen : 0), ok);
+        }
+        return;
+    }
 #pragma unroll 4
     for (int r = r0; r < TILE_N; r += STEP) {
-        const int j = tile * TILE_N + r;
+        const int j = j0 + r;
         bool ok = j < n && (j >= lo || j < keep) && c < have;
         const bf16* src = a.kv;
         if (ok) {
-            int page, po;
-            if (in_page) { page = page_of_tile; po = j & (a.page_size - 1); }
-            else { const int pi = a.page_shift >= 0 ? j >> a.page_shift : j / a.page_size; po = j - pi * a.page_size; page = table[pi]; }
+            const int pi = a.page_shift >= 0 ? j >> a.page_shift : j / a.page_size, po = j - pi * a.page_size, page = table[pi];
             ok = page >= 0 && page < a.pages;
             if (ok) src = a.kv + (((long)page * a.kv_heads + hk) * a.page_size + po) * rowlen + x;
         }
-        const uint32_t d = is_k ? tile_off<KP>(r, c) : tile_off<VP>(r, c);
-        cp_async16(base + d, src, ok);
+        cp_async16(base + (is_k ? tile_off<KP>(r, c) : tile_off<VP>(r, c)), src, ok);
     }
 }
 
 template <int KP, int VP, int STAGES>
 __global__ void __launch_bounds__(128) maps_decode_kernel(const MapsArgs a) {
     extern __shared__ __align__(128) unsigned char smem_raw[];
+    __shared__ float scratch[33];
     constexpr uint32_t K_BYTES = TILE_N * KP * 2, V_BYTES = TILE_N * VP * 2;
     const uint32_t q_s = smem_u32(smem_raw), k_s = q_s + 16 * KP * 2, v_s = k_s + STAGES * K_BYTES;
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -485,43 +494,60 @@ __global__ void __launch_bounds__(128) maps_decode_kernel(const MapsArgs a) {
     __syncthreads();
     __syncwarp();
     cluster_barrier();                                               // every part of the cluster lies in its shared memory
-    // ---- a warp a head: the parts in their order, the maps, the norm, the gate
+    // ---- a head at a time, a channel (VP 256: two) a thread: the parts in their order, all their loads in flight at once; then the
+    // maps, the norm, the gate
+    constexpr int PER = VP > 128 ? 2 : 1;
     const uint32_t po = smem_u32(part_o), pml = smem_u32(part_ml);
-    for (int x = split + splits * warp; x < g; x += splits * 4) {
+    for (int x = split; x < g; x += splits) {
         const int h = hk * group + g0 + x;
-        float res[VP / 32];
+        float res[PER];
         for (int m = 0; m < a.maps; ++m) {
             const int r = m * hpm + x;
-            float mm = -INFINITY, l = 0.f, acc[VP / 32];
+            float ms[MD_PARTS], ls[MD_PARTS], os[MD_PARTS][PER];
 #pragma unroll
-            for (int i = 0; i < VP / 32; ++i) acc[i] = 0.f;
-            for (int s2 = 0; s2 < splits; ++s2) mm = fmaxf(mm, ld_cluster_f32(pml + r * 8, s2));
-            for (int s2 = 0; s2 < splits; ++s2) {
-                const float ms = ld_cluster_f32(pml + r * 8, s2);
-                const float f = ms == -INFINITY ? 0.f : ex2(ms - mm);
-                l += f * ld_cluster_f32(pml + r * 8 + 4, s2);
+            for (int s2 = 0; s2 < MD_PARTS; ++s2) {
+                ms[s2] = -INFINITY; ls[s2] = 0.f;
+                if (s2 < splits) {
+                    ms[s2] = ld_cluster_f32(pml + r * 8, s2);
+                    ls[s2] = ld_cluster_f32(pml + r * 8 + 4, s2);
+                }
 #pragma unroll
-                for (int i = 0; i < VP / 32; ++i)
-                    if (lane + 32 * i < a.vdim) acc[i] += f * ld_cluster_f32(po + (r * VP + lane + 32 * i) * 4, s2);
+                for (int i = 0; i < PER; ++i) {
+                    os[s2][i] = 0.f;
+                    if (s2 < splits && (int)threadIdx.x + 128 * i < a.vdim) os[s2][i] = ld_cluster_f32(po + (r * VP + threadIdx.x + 128 * i) * 4, s2);
+                }
+            }
+            float mm = -INFINITY, l = 0.f, acc[PER];
+#pragma unroll
+            for (int i = 0; i < PER; ++i) acc[i] = 0.f;
+#pragma unroll
+            for (int s2 = 0; s2 < MD_PARTS; ++s2) mm = fmaxf(mm, ms[s2]);
+#pragma unroll
+            for (int s2 = 0; s2 < MD_PARTS; ++s2) {
+                const float f = ms[s2] == -INFINITY ? 0.f : ex2(ms[s2] - mm);
+                l += f * ls[s2];
+#pragma unroll
+                for (int i = 0; i < PER; ++i) acc[i] += f * os[s2][i];
             }
             const float inv = l > 0.f ? 1.f / l : 0.f;
 #pragma unroll
-            for (int i = 0; i < VP / 32; ++i) res[i] = m == 0 ? acc[i] * inv : res[i] - a.lam * (acc[i] * inv);
+            for (int i = 0; i < PER; ++i) res[i] = m == 0 ? acc[i] * inv : res[i] - a.lam * (acc[i] * inv);
         }
         if (a.maps > 1) {
             float ss = 0.f;
 #pragma unroll
-            for (int i = 0; i < VP / 32; ++i) ss += res[i] * res[i];
-            const float f = rsqrtf(warp_sum(ss) / (float)a.vdim + a.eps) * a.factor;
+            for (int i = 0; i < PER; ++i) ss += res[i] * res[i];     // (channels past vdim hold zeros)
+            const float f = rsqrtf(block_sum(ss, scratch) / (float)a.vdim + a.eps) * a.factor;
 #pragma unroll
-            for (int i = 0; i < VP / 32; ++i) res[i] *= f;
+            for (int i = 0; i < PER; ++i) res[i] *= f;
         }
-        bf16* dst = a.out + ((size_t)t * a.heads + h) * a.vdim;
-        const bf16* gr = a.gate ? a.gate + (size_t)t * a.gate_ld + (size_t)h * a.vdim : nullptr;
 #pragma unroll
-        for (int i = 0; i < VP / 32; ++i) {
-            const int d = lane + 32 * i;
-            if (d < a.vdim) dst[d] = __float2bfloat16_rn(gr ? res[i] * mp_sigmoid(to_f32(gr[d])) : res[i]);
+        for (int i = 0; i < PER; ++i) {
+            const int d = threadIdx.x + 128 * i;
+            if (d < a.vdim) {
+                const float y = a.gate ? res[i] * mp_sigmoid(to_f32(a.gate[(size_t)t * a.gate_ld + (size_t)h * a.vdim + d])) : res[i];
+                a.out[((size_t)t * a.heads + h) * a.vdim + d] = __float2bfloat16_rn(y);
+            }
         }
     }
     __syncwarp();

@@ -8,6 +8,7 @@
 // 32 rows and add their partial sums through shared memory in a fixed order.
 // mode 1 computes SwiGLU's activation in the epilogue: the CTA's first tile holds 16 gate rows, its second the 16 up
 // rows of the same columns, and it writes silu(gate) * up.
+// mode 5 is the plain product under a squared relu (an ungated feed-forward's first product with its activation).
 // mode 2 is the attention's first product with what follows it folded in: w is [q heads; k heads; v heads] x head_dim
 // rows, the head_dim / 16 CTAs of a head form a thread-block cluster, and after the product they norm the head
 // (RMSNorm over head_dim with the q or k weight), rotate it by its token's position (half-split pairs, whole head)
@@ -333,6 +334,7 @@ __global__ void __launch_bounds__(SK_WARPS * 32, MIN_CTAS) gemm_skinny_kernel(vo
             for (int wv = 0; wv < SK_WARPS; ++wv) u += red[wv][HALF * 16 + rr][tok];
             v = v / (1.f + expf(-v)) * (u * scale_in[tok]);
         }
+        if (mode == 5) { v = fmaxf(v, 0.f); v *= v; }
         if (col < width) {
             if (out_f32) ((float*)out)[(size_t)tok * width + col] = v;
             else ((bf16*)out)[(size_t)tok * width + col] = __float2bfloat16_rn(v);
@@ -355,7 +357,7 @@ static int skinny_product(void* out, int out_f32, const void* x, const void* w, 
     if (m < 0 || m > most) HB_REFUSE("gemm_bf16_skinny: %d rows; this kernel takes 1 to %d", m, most);
     if (k < 8 || k % 8) HB_REFUSE("gemm_bf16_skinny: k = %d is no multiple of 8", k);
     if ((((uintptr_t)out | (uintptr_t)x | (uintptr_t)w) % 16) != 0) HB_REFUSE("gemm_bf16_skinny: pointers must be 16-byte aligned");
-    if (mode != 0 && mode != 1 && mode != 3 && mode != 4) HB_REFUSE("gemm_bf16_skinny: mode %d", mode);
+    if (mode != 0 && mode != 1 && mode != 3 && mode != 4 && mode != 5) HB_REFUSE("gemm_bf16_skinny: mode %d", mode);
     if (mode == 4 && (!h || !post || !post[0] || !post[1] || !post[2] || out_f32 || (out && (!pre || !pre[0] || !pre[1] || !pre[2]))))
         HB_REFUSE("gemm_bf16_skinny: mode 4 needs h and the norm the product passes, with an output also the norm of the new stream, and writes bfloat16");
     if (mode == 3 && (!h || !next_weight || !ss_out || out_f32)) HB_REFUSE("gemm_bf16_skinny: mode 3 needs h, the next norm's weight and ss_out, and writes bfloat16");
@@ -389,10 +391,10 @@ static int skinny_product(void* out, int out_f32, const void* x, const void* w, 
         else gemm_skinny_kernel<2, 2, 4, 2><<<grid, SK_WARPS * 32, 0, s>>>(HB_SK_ARGS(1, inter));
     } else {
         if (n < 1) HB_REFUSE("gemm_bf16_skinny: n = %d", n);
-        const bool wide = mode == 0 && n >= 32 * 2 * sms;    // enough rows to give every SM two CTAs of 32 rows
+        const bool wide = (mode == 0 || mode == 5) && n >= 32 * 2 * sms;    // enough rows to give every SM two CTAs of 32 rows
         const int grid = wide ? (n + 31) / 32 : (n + 15) / 16;
-        if (wide && nt == 1) gemm_skinny_kernel<2, 1, 4, 2><<<grid, SK_WARPS * 32, 0, s>>>(HB_SK_ARGS(0, 0));
-        else if (wide) gemm_skinny_kernel<2, 2, 4, 2><<<grid, SK_WARPS * 32, 0, s>>>(HB_SK_ARGS(0, 0));
+        if (wide && nt == 1) gemm_skinny_kernel<2, 1, 4, 2><<<grid, SK_WARPS * 32, 0, s>>>(HB_SK_ARGS(mode, 0));
+        else if (wide) gemm_skinny_kernel<2, 2, 4, 2><<<grid, SK_WARPS * 32, 0, s>>>(HB_SK_ARGS(mode, 0));
         else if (nt == 1 && grid > 2 * sms && grid <= 3 * sms)       // one wave of three CTAs per SM instead of one and a bit of two
             gemm_skinny_kernel<1, 1, 4, 3><<<grid, SK_WARPS * 32, 0, s>>>(HB_SK_ARGS(mode, 0));
         else if (nt == 1) gemm_skinny_kernel<1, 1, 8, 2><<<grid, SK_WARPS * 32, 0, s>>>(HB_SK_ARGS(mode, 0));

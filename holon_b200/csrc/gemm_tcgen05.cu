@@ -140,6 +140,10 @@ __global__ void __launch_bounds__(192, 1) gemm_tcgen05_kernel(const __grid_const
 #pragma unroll
                     for (int i = 0; i < 32; ++i) v[i] = v[i] / (1.f + __expf(-v[i])) * __uint_as_float(u[i]);
                 }
+                if (mode == 5) {                                      // a squared relu
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) { v[i] = fmaxf(v[i], 0.f); v[i] *= v[i]; }
+                }
                 if (c == chunks - 1) {                               // everything is in registers: hand the accumulator back
                     tc_fence_before();
                     __syncwarp();
@@ -214,7 +218,7 @@ extern "C" int hb_gemm_bf16_tcgen05(void* out, int out_f32, const void* x, const
     if (m == 0 || n == 0) return 0;
     if (k < 8 || k % 8) HB_REFUSE("gemm_tcgen05: k = %d is no multiple of 8", k);
     if ((((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) % 16) != 0) HB_REFUSE("gemm_tcgen05: pointers must be 16-byte aligned");
-    if (mode != 0 && mode != 1) HB_REFUSE("gemm_tcgen05: mode %d", mode);
+    if (mode != 0 && mode != 1 && mode != 5) HB_REFUSE("gemm_tcgen05: mode %d", mode);
     if (mode == 1 && (inter < 1 || n != 2 * inter)) HB_REFUSE("gemm_tcgen05: mode 1 needs n = 2 inter (n %d, inter %d)", n, inter);
     CUtensorMap map_x, map_w;
     int rc = encode_map(&map_x, x, m, k, TC_BM);

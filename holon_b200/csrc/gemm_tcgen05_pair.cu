@@ -187,6 +187,10 @@ gemm_tcgen05_pair_kernel(const __grid_constant__ CUtensorMap map_x, const __grid
 #pragma unroll
                     for (int i = 0; i < 32; ++i) v[i] = v[i] / (1.f + __expf(-v[i])) * __uint_as_float(u[i]);
                 }
+                if (mode == 5) {                                      // a squared relu
+#pragma unroll
+                    for (int i = 0; i < 32; ++i) { v[i] = fmaxf(v[i], 0.f); v[i] *= v[i]; }
+                }
                 if (c == chunks - 1) {                               // everything is in registers: hand the accumulator back
                     tc_fence_before();
                     __syncwarp();
@@ -266,7 +270,7 @@ extern "C" int hb_gemm_bf16_tcgen05_pair(void* out, int out_f32, const void* x, 
     if (m == 0 || n == 0) return 0;
     if (k < 8 || k % 8) HB_REFUSE("gemm_tcgen05_pair: k = %d is no multiple of 8", k);
     if ((((uintptr_t)x | (uintptr_t)w | (uintptr_t)out) % 16) != 0) HB_REFUSE("gemm_tcgen05_pair: pointers must be 16-byte aligned");
-    if (mode != 0 && mode != 1) HB_REFUSE("gemm_tcgen05_pair: mode %d", mode);
+    if (mode != 0 && mode != 1 && mode != 5) HB_REFUSE("gemm_tcgen05_pair: mode %d", mode);
     if (mode == 1 && (inter < 1 || n != 2 * inter)) HB_REFUSE("gemm_tcgen05_pair: mode 1 needs n = 2 inter (n %d, inter %d)", n, inter);
     static int sms = 0;
     if (sms == 0) {

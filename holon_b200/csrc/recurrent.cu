@@ -477,51 +477,88 @@ extern "C" int hb_delta_prepare(float* qk, float* v, float* beta, float* decay, 
 // A token's row of `first` holds, from column `at` on, [x (heads vdim) | B (groups n) | C (groups n) | dt (heads)]. x, B and C
 // pass a causal convolution over time with a bias (weights conv [channels, taps], the last tap the token's own; inputs before
 // the step's first token of the row come from conv_state [slots, taps - 1, channels], oldest first) and silu; x goes to v, C and
-// B to cb [token][C, B][groups n]. dt = softplus(. + dt_bias), decay = exp(-exp(rate_log) dt). grid (tokens, segments); a thread
-// owns W neighbouring channels, or one head's dt. The carried inputs of a row of one token move on here, those of longer rows in
-// hb_conv_carry (as above).
-template <typename T, int W>
+// B to cb [token][C, B][groups n]. dt = softplus(. + dt_bias), decay = exp(-exp(rate_log) dt). grid (runs of `run` tokens, segments);
+// a thread owns W neighbouring channels, or one head's dt. The carried inputs of a row of one token move on here, those of longer
+// rows in hb_conv_carry (as above). TAPS > 0: so many taps, whose weights and inputs wait in registers from token to token; 0: any.
+template <typename T, int W, int TAPS>
 __global__ void state_space_prepare_kernel(float* __restrict__ cb, float* __restrict__ v, float* __restrict__ dt,
                                            float* __restrict__ decay, const T* __restrict__ first, long ld, int at,
                                            const T* __restrict__ conv, const T* __restrict__ conv_bias, int taps, T* conv_state,
                                            const float* __restrict__ dt_bias, const float* __restrict__ rate_log,
                                            const int32_t* __restrict__ query_start, const int32_t* __restrict__ row_slot, int rows,
-                                           int heads, int inner, int gn) {
-    const int t = blockIdx.x, C = inner + 2 * gn, quads = C / W;
+                                           int tokens, int run, int heads, int inner, int gn) {
+    const int C = inner + 2 * gn, quads = C / W, begin = blockIdx.x * run, end = min(begin + run, tokens);
     int e = blockIdx.y * blockDim.x + threadIdx.x;
     if (e >= quads) {
         e -= quads;
         if (e >= heads) return;
-        const float d = softplus_f(to_f32(first[(size_t)t * ld + at + C + e]) + dt_bias[e]);
-        dt[(size_t)t * heads + e] = d;
-        decay[(size_t)t * heads + e] = expf(-expf(rate_log[e]) * d);
+        for (int t = begin; t < end; ++t) {
+            const float d = softplus_f(to_f32(first[(size_t)t * ld + at + C + e]) + dt_bias[e]);
+            dt[(size_t)t * heads + e] = d;
+            decay[(size_t)t * heads + e] = expf(-expf(rate_log[e]) * d);
+        }
         return;
     }
-    const int c = e * W, b = row_of_token(query_start, rows, t), t0 = query_start[b];
-    T* st = conv_state ? conv_state + (size_t)row_slot[b] * (taps - 1) * C + c : nullptr;
+    const int c = e * W;
     auto load = [&](const T* p, float* x) {
         if constexpr (W == 4) { float f[4]; Vec4<T>::load(p, f); x[0] = f[0]; x[1] = f[1]; x[2] = f[2]; x[3] = f[3]; }
         else x[0] = to_f32(p[0]);
     };
-    float acc[W], x[W];
-    load(conv_bias + c, acc);
-    for (int j = 0; j < taps; ++j) {
-        const int from = t - (taps - 1 - j);                             // the token this tap weighs
-        load(from >= t0 ? first + (size_t)from * ld + at + c : st + (size_t)(taps - 1 + (from - t0)) * C, x);
+    constexpr int KEEP = TAPS > 1 ? TAPS - 1 : 1;
+    float bias[W], w[TAPS > 0 ? TAPS : 1][W], before[KEEP][W];             // before: the inputs ahead of the token, oldest first
+    load(conv_bias + c, bias);
+    if (TAPS > 0)
 #pragma unroll
-        for (int i = 0; i < W; ++i) acc[i] = fmaf(to_f32(conv[(size_t)(c + i) * taps + j]), x[i], acc[i]);
+        for (int j = 0; j < TAPS; ++j)
+#pragma unroll
+            for (int i = 0; i < W; ++i) w[j][i] = to_f32(conv[(size_t)(c + i) * TAPS + j]);
+    int b = row_of_token(query_start, rows, begin);
+    for (int t = begin; t < end; ++t) {
+        while (t >= query_start[b + 1]) ++b;
+        const int t0 = query_start[b];
+        T* st = conv_state ? conv_state + (size_t)row_slot[b] * (taps - 1) * C + c : nullptr;
+        auto input = [&](int from, float* x) {                               // the channel inputs of token `from` of this row
+            load(from >= t0 ? first + (size_t)from * ld + at + c : st + (size_t)(taps - 1 + (from - t0)) * C, x);
+        };
+        float acc[W], x[W];
+#pragma unroll
+        for (int i = 0; i < W; ++i) acc[i] = bias[i];
+        if (TAPS > 0) {
+            if (t == begin || t == t0) {
+#pragma unroll
+                for (int j = 0; j + 1 < TAPS; ++j) input(t - (TAPS - 1) + j, before[j]);
+            }
+            input(t, x);
+#pragma unroll
+            for (int j = 0; j + 1 < TAPS; ++j)
+#pragma unroll
+                for (int i = 0; i < W; ++i) acc[i] = fmaf(w[j][i], before[j][i], acc[i]);
+#pragma unroll
+            for (int i = 0; i < W; ++i) {
+                acc[i] = fmaf(w[TAPS > 0 ? TAPS - 1 : 0][i], x[i], acc[i]);
+#pragma unroll
+                for (int j = 0; j + 2 < TAPS; ++j) before[j][i] = before[j + 1][i];
+                before[KEEP - 1][i] = x[i];
+            }
+        } else {
+            for (int j = 0; j < taps; ++j) {
+                input(t - (taps - 1 - j), x);
+#pragma unroll
+                for (int i = 0; i < W; ++i) acc[i] = fmaf(to_f32(conv[(size_t)(c + i) * taps + j]), x[i], acc[i]);
+            }
+        }
+        if (st && taps > 1 && query_start[b + 1] - t0 == 1) {                // a row of one token: its carried inputs move on
+            for (int i = 0; i + 1 < taps - 1; ++i)
+#pragma unroll
+                for (int k = 0; k < W; ++k) st[(size_t)i * C + k] = st[(size_t)(i + 1) * C + k];
+#pragma unroll
+            for (int k = 0; k < W; ++k) st[(size_t)(taps - 2) * C + k] = first[(size_t)t * ld + at + c + k];
+        }
+        float* dst = c < inner ? v + (size_t)t * inner + c
+                   : c < inner + gn ? cb + (size_t)t * 2 * gn + gn + (c - inner) : cb + (size_t)t * 2 * gn + (c - inner - gn);
+        if constexpr (W == 4) *(float4*)dst = make_float4(silu_f(acc[0]), silu_f(acc[1]), silu_f(acc[2]), silu_f(acc[3]));
+        else dst[0] = silu_f(acc[0]);
     }
-    if (st && taps > 1 && query_start[b + 1] - t0 == 1) {                // a row of one token: its carried inputs move on
-        for (int i = 0; i + 1 < taps - 1; ++i)
-#pragma unroll
-            for (int k = 0; k < W; ++k) st[(size_t)i * C + k] = st[(size_t)(i + 1) * C + k];
-#pragma unroll
-        for (int k = 0; k < W; ++k) st[(size_t)(taps - 2) * C + k] = first[(size_t)t * ld + at + c + k];
-    }
-    float* dst = c < inner ? v + (size_t)t * inner + c
-               : c < inner + gn ? cb + (size_t)t * 2 * gn + gn + (c - inner) : cb + (size_t)t * 2 * gn + (c - inner - gn);
-    if constexpr (W == 4) *(float4*)dst = make_float4(silu_f(acc[0]), silu_f(acc[1]), silu_f(acc[2]), silu_f(acc[3]));
-    else dst[0] = silu_f(acc[0]);
 }
 
 extern "C" int hb_state_space_prepare(float* cb, float* v, float* dt, float* decay, const void* first, int dtype, long ld, int at,
@@ -537,14 +574,18 @@ extern "C" int hb_state_space_prepare(float* cb, float* v, float* dt, float* dec
                      (((uintptr_t)first | (uintptr_t)conv_bias | (uintptr_t)conv_state) % four) == 0;
     const long elements = (inner + 2L * gn) / (vec ? 4 : 1) + heads, segments = (elements + 127) / 128;
     if (segments > 65535) HB_REFUSE("state_space_prepare: %ld segments a token are above 65535", segments);
-    const dim3 grid(tokens, (unsigned)segments);
+    const int run = tokens >= 1024 ? 8 : tokens >= 256 ? 2 : 1;                // tokens a thread takes in turn
+    const dim3 grid((tokens + run - 1) / run, (unsigned)segments);
     cudaStream_t s = (cudaStream_t)stream;
-#define HB_RUN(T, W) state_space_prepare_kernel<T, W><<<grid, 128, 0, s>>>(cb, v, dt, decay, (const T*)first, ld, at, (const T*)conv, \
-    (const T*)conv_bias, taps, (T*)conv_state, dt_bias, rate_log, query_start, row_slot, rows, heads, inner, gn)
+#define HB_TAPS(T, W, N) state_space_prepare_kernel<T, W, N><<<grid, 128, 0, s>>>(cb, v, dt, decay, (const T*)first, ld, at, (const T*)conv, \
+    (const T*)conv_bias, taps, (T*)conv_state, dt_bias, rate_log, query_start, row_slot, rows, tokens, run, heads, inner, gn)
+#define HB_RUN(T, W) do { if (taps == 4) HB_TAPS(T, W, 4); else if (taps == 3) HB_TAPS(T, W, 3); else if (taps == 2) HB_TAPS(T, W, 2); \
+                          else HB_TAPS(T, W, 0); } while (0)
     if (dtype == HB_F32) { if (vec) HB_RUN(float, 4); else HB_RUN(float, 1); }
     else if (dtype == HB_BF16) { if (vec) HB_RUN(bf16, 4); else HB_RUN(bf16, 1); }
     else HB_REFUSE("state_space_prepare: dtype %d", dtype);
 #undef HB_RUN
+#undef HB_TAPS
     HB_LAUNCH_CHECK("state_space_prepare");
     return 0;
 }

@@ -1,0 +1,269 @@
+// The state-space recurrence for rows of several tokens, in chunks of 64 (the form of Dao and Gu, Transformers are SSMs: Generalized
+// Models and Efficient Algorithms Through Structured State Space Duality), everything in 32-bit on CUDA cores:
+//     S_t = g_t S_(t-1) + dt_t B_t x_t^T,  y_t = S_t^T C_t + skip x_t,  g_t = exp(-exp(rate_log) dt_t)
+// With L_i the sum of the logarithms of g over a chunk's tokens up to i (kept as a pair of float32 whose sum is exact to double
+// precision: what the weights need are differences of such sums), a chunk with the state S_in before it gives
+//     y_i = sum_(j <= i) (C_i . B_j) exp(L_i - L_j) dt_j x_j + exp(L_i) S_in^T C_i + skip x_i
+//     S_out = exp(L_last) S_in + sum_j exp(L_last - L_j) dt_j B_j x_j^T.
+// Four kernels: the chunks' products C_i . B_j, per group; the chunks' own contributions to the state, per head; the walk over a
+// row's chunks, an element of the state a thread, which leaves every chunk's S_in behind and writes the row's state back; the
+// chunks' outputs, per head. Only the third is sequential, one multiply-add a chunk. Blocks find their (row, chunk) in the step's
+// rows; launches may have more tiles than the step has chunks. One-token rows: csrc/recurrent.cu.
+#include <type_traits>
+
+#include "common.cuh"
+
+#define SS_Q 64                          // tokens a chunk
+#define SS_T 64                          // rows and columns of an output tile
+#define SS_K 32                          // depth of a staged slice
+#define SS_PAD 4
+#define SS_THREADS 128                   // a thread: 8 rows x 4 columns of a tile
+
+struct Chunk { int row, t0, n, first_tile; };              // the batch row, first token, tokens, the row's first tile
+
+// Tile number -> chunk (row -1: there is none). Rows row0 .. rows - 1 in order, each ceil(tokens / 64) tiles.
+__device__ __forceinline__ Chunk find_chunk(const int32_t* __restrict__ query_start, int row0, int rows, int tile) {
+    int left = tile;
+    for (int b = row0; b < rows; ++b) {
+        const int n = query_start[b + 1] - query_start[b], tiles = (n + SS_Q - 1) / SS_Q;
+        if (left < tiles) return {b, query_start[b] + left * SS_Q, min(SS_Q, n - left * SS_Q), tile - left};
+        left -= tiles;
+    }
+    return {-1, 0, 0, 0};
+}
+
+// A slice of both operands in shared memory, a[k][row], b[k][column]: acc += a^T b.
+__device__ __forceinline__ void tile_step(float (&acc)[8][4], const float (*a)[SS_T + SS_PAD], const float (*b)[SS_T + SS_PAD], int depth) {
+    const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+#pragma unroll 8
+    for (int k = 0; k < depth; ++k) {
+        const float4 r0 = *(const float4*)&a[k][ty * 8], r1 = *(const float4*)&a[k][ty * 8 + 4], c = *(const float4*)&b[k][tx * 4];
+        const float r[8] = {r0.x, r0.y, r0.z, r0.w, r1.x, r1.y, r1.z, r1.w};
+#pragma unroll
+        for (int i = 0; i < 8; ++i) {
+            acc[i][0] = fmaf(r[i], c.x, acc[i][0]); acc[i][1] = fmaf(r[i], c.y, acc[i][1]);
+            acc[i][2] = fmaf(r[i], c.z, acc[i][2]); acc[i][3] = fmaf(r[i], c.w, acc[i][3]);
+        }
+    }
+}
+
+// L_i of a chunk's tokens for one head, by warp 0: hi + lo in two floats; tokens past the chunk repeat the last.
+__device__ __forceinline__ void log_decays(float* hi, float* lo, float* steps, const float* __restrict__ dt, const Chunk& c, int heads,
+                                           int h, float rate) {
+    if (threadIdx.x < 32) {
+        const int lane = threadIdx.x;
+        const float d0 = 2 * lane < c.n ? dt[(size_t)(c.t0 + 2 * lane) * heads + h] : 0.f;
+        const float d1 = 2 * lane + 1 < c.n ? dt[(size_t)(c.t0 + 2 * lane + 1) * heads + h] : 0.f;
+        const double a0 = -(double)rate * d0, a1 = -(double)rate * d1;
+        double s = a0 + a1;
+#pragma unroll
+        for (int o = 1; o < 32; o <<= 1) {
+            const double up = __shfl_up_sync(0xffffffffu, s, o);
+            if (lane >= o) s += up;
+        }
+        const double l0 = s - a1;
+        steps[2 * lane] = d0; steps[2 * lane + 1] = d1;
+        hi[2 * lane] = (float)l0; lo[2 * lane] = (float)(l0 - (double)(float)l0);
+        hi[2 * lane + 1] = (float)s; lo[2 * lane + 1] = (float)(s - (double)(float)s);
+    }
+}
+
+// ---- products[tile][group][i][j] = C_i . B_j, [64][64] each. grid (tiles, groups)
+__global__ void __launch_bounds__(SS_THREADS) ss_products_kernel(float* __restrict__ products, const float* __restrict__ cb,
+                                                                 const int32_t* __restrict__ query_start, int row0, int rows, int groups, int n) {
+    __shared__ __align__(16) float a[SS_K][SS_T + SS_PAD], b[SS_K][SS_T + SS_PAD];
+    const Chunk c = find_chunk(query_start, row0, rows, blockIdx.x);
+    if (c.row < 0) return;
+    const int g = blockIdx.y;
+    float acc[8][4] = {};
+    for (int k0 = 0; k0 < n; k0 += SS_K) {
+        const int depth = min(SS_K, n - k0);
+        for (int e = threadIdx.x; e < SS_T * SS_K; e += SS_THREADS) {
+            const int i = e / SS_K, k = e % SS_K;
+            const bool in = i < c.n && k < depth;
+            const float* src = cb + ((size_t)(c.t0 + i) * 2 * groups + g) * n + k0 + k;
+            a[k][i] = in ? src[0] : 0.f;
+            b[k][i] = in ? src[(size_t)groups * n] : 0.f;
+        }
+        __syncthreads();
+        tile_step(acc, a, b, depth);
+        __syncthreads();
+    }
+    const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+    float* out = products + ((size_t)blockIdx.x * groups + g) * SS_Q * SS_Q;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) *(float4*)(out + (ty * 8 + i) * SS_Q + tx * 4) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+}
+
+// ---- own[tile][head][p][n] = sum_j exp(L_last - L_j) dt_j x_j[p] B_j[n]; last[tile][head] = exp(L_last). grid (tiles, heads, tiles of
+// p times tiles of n)
+__global__ void __launch_bounds__(SS_THREADS) ss_own_kernel(float* __restrict__ own, float* __restrict__ last, const float* __restrict__ cb,
+                                                            const float* __restrict__ x, const float* __restrict__ dt,
+                                                            const float* __restrict__ rate_log, const int32_t* __restrict__ query_start,
+                                                            int row0, int rows, int heads, int groups, int n, int vdim, int n_tiles) {
+    __shared__ __align__(16) float a[SS_K][SS_T + SS_PAD], b[SS_K][SS_T + SS_PAD];
+    __shared__ float hi[SS_Q], lo[SS_Q], steps[SS_Q], w[SS_Q];
+    const Chunk c = find_chunk(query_start, row0, rows, blockIdx.x);
+    if (c.row < 0) return;
+    const int h = blockIdx.y, g = h / (heads / groups);
+    const int p0 = ((int)blockIdx.z / n_tiles) * SS_T, n0 = ((int)blockIdx.z % n_tiles) * SS_T;
+    log_decays(hi, lo, steps, dt, c, heads, h, expf(rate_log[h]));
+    __syncthreads();
+    if (threadIdx.x < SS_Q) {
+        const int j = threadIdx.x;
+        w[j] = expf((hi[SS_Q - 1] - hi[j]) + (lo[SS_Q - 1] - lo[j])) * steps[j];
+        if (j == 0 && blockIdx.z == 0) last[(size_t)blockIdx.x * heads + h] = expf(hi[SS_Q - 1] + lo[SS_Q - 1]);
+    }
+    __syncthreads();
+    float acc[8][4] = {};
+    for (int k0 = 0; k0 < c.n; k0 += SS_K) {
+        const int depth = min(SS_K, c.n - k0);
+        for (int e = threadIdx.x; e < SS_K * SS_T; e += SS_THREADS) {
+            const int k = e / SS_T, i = e % SS_T;
+            const size_t t = (size_t)(c.t0 + k0 + k);
+            a[k][i] = k < depth && p0 + i < vdim ? x[(t * heads + h) * vdim + p0 + i] * w[k0 + k] : 0.f;
+            b[k][i] = k < depth && n0 + i < n ? cb[((t * 2 + 1) * groups + g) * n + n0 + i] : 0.f;
+        }
+        __syncthreads();
+        tile_step(acc, a, b, depth);
+        __syncthreads();
+    }
+    const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+    float* out = own + ((size_t)blockIdx.x * heads + h) * vdim * n;
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        const int p = p0 + ty * 8 + i, col = n0 + tx * 4;
+        if (p >= vdim) break;
+        if ((n & 3) == 0 && col + 3 < n) *(float4*)(out + (size_t)p * n + col) = make_float4(acc[i][0], acc[i][1], acc[i][2], acc[i][3]);
+        else
+#pragma unroll
+            for (int k = 0; k < 4; ++k) if (col + k < n) out[(size_t)p * n + col + k] = acc[i][k];
+    }
+}
+
+// ---- a row's chunks in order: own[tile] <- the state before the chunk, state <- the state behind the last. grid (rows - row0, heads,
+// slices of the state), an element (V: four) a thread.
+template <bool V>
+__global__ void ss_walk_kernel(float* __restrict__ own, const float* __restrict__ last, float* __restrict__ state,
+                               const int32_t* __restrict__ query_start, const int32_t* __restrict__ row_slot, int row0, int heads, int size) {
+    typedef typename std::conditional<V, float4, float>::type E;
+    const int b = row0 + (int)blockIdx.x, h = blockIdx.y, e = blockIdx.z * blockDim.x + threadIdx.x;
+    int first = 0;
+    for (int r = row0; r < b; ++r) first += (query_start[r + 1] - query_start[r] + SS_Q - 1) / SS_Q;
+    const int tiles = (query_start[b + 1] - query_start[b] + SS_Q - 1) / SS_Q;
+    if (e >= (V ? size >> 2 : size) || tiles == 0) return;
+    E* st = (E*)(state + ((size_t)row_slot[b] * heads + h) * size) + e;
+    const size_t stride = (size_t)heads * size / (V ? 4 : 1);
+    E* p = (E*)(own + ((size_t)first * heads + h) * size) + e;
+    const float* f = last + (size_t)first * heads + h;
+    E s = *st;
+    auto step = [&](float d, const E& v) {
+        if constexpr (V) { s.x = fmaf(d, s.x, v.x); s.y = fmaf(d, s.y, v.y); s.z = fmaf(d, s.z, v.z); s.w = fmaf(d, s.w, v.w); }
+        else s = fmaf(d, s, v);
+    };
+    int i = 0;
+    for (; i + 4 <= tiles; i += 4, p += 4 * stride, f += 4 * (size_t)heads) {        // (four chunks' loads fly together)
+        const E v0 = p[0], v1 = p[stride], v2 = p[2 * stride], v3 = p[3 * stride];
+        const float d0 = f[0], d1 = f[heads], d2 = f[2 * (size_t)heads], d3 = f[3 * (size_t)heads];
+        p[0] = s; step(d0, v0);
+        p[stride] = s; step(d1, v1);
+        p[2 * stride] = s; step(d2, v2);
+        p[3 * stride] = s; step(d3, v3);
+    }
+    for (; i < tiles; ++i, p += stride, f += heads) {
+        const E v = p[0];
+        p[0] = s;
+        step(f[0], v);
+    }
+    *st = s;
+}
+
+// ---- y_i[p] of a chunk: the products' part over its own tokens, the state's part over n, the skip. grid (tiles, heads, tiles of p)
+__global__ void __launch_bounds__(SS_THREADS) ss_out_kernel(float* __restrict__ y, const float* __restrict__ products,
+                                                            const float* __restrict__ before, const float* __restrict__ cb,
+                                                            const float* __restrict__ x, const float* __restrict__ dt,
+                                                            const float* __restrict__ rate_log, const float* __restrict__ skip,
+                                                            const int32_t* __restrict__ query_start, int row0, int rows, int heads,
+                                                            int groups, int n, int vdim) {
+    __shared__ __align__(16) float a[SS_K][SS_T + SS_PAD], b[SS_K][SS_T + SS_PAD];
+    __shared__ float hi[SS_Q], lo[SS_Q], steps[SS_Q], w[SS_Q];
+    const Chunk c = find_chunk(query_start, row0, rows, blockIdx.x);
+    if (c.row < 0) return;
+    const int h = blockIdx.y, g = h / (heads / groups), p0 = (int)blockIdx.z * SS_T;
+    log_decays(hi, lo, steps, dt, c, heads, h, expf(rate_log[h]));
+    __syncthreads();
+    if (threadIdx.x < SS_Q) w[threadIdx.x] = expf(hi[threadIdx.x] + lo[threadIdx.x]);
+    __syncthreads();
+    float acc[8][4] = {};
+    const float* cbp = products + ((size_t)blockIdx.x * groups + g) * SS_Q * SS_Q;
+    for (int k0 = 0; k0 < c.n; k0 += SS_K) {                       // over the chunk's tokens j
+        const int depth = min(SS_K, c.n - k0);
+        for (int e = threadIdx.x; e < SS_K * SS_T; e += SS_THREADS) {
+            const int i = e / SS_K, k = e % SS_K, j = k0 + k;       // weight of token j in row i
+            a[k][i] = j <= i && j < c.n ? cbp[i * SS_Q + j] * expf((hi[i] - hi[j]) + (lo[i] - lo[j])) * steps[j] : 0.f;
+        }
+        for (int e = threadIdx.x; e < SS_K * SS_T; e += SS_THREADS) {
+            const int k = e / SS_T, i = e % SS_T;
+            b[k][i] = k < depth && p0 + i < vdim ? x[((size_t)(c.t0 + k0 + k) * heads + h) * vdim + p0 + i] : 0.f;
+        }
+        __syncthreads();
+        tile_step(acc, a, b, depth);
+        __syncthreads();
+    }
+    const float* S = before + ((size_t)blockIdx.x * heads + h) * vdim * n;
+    for (int k0 = 0; k0 < n; k0 += SS_K) {                         // over the state's channels
+        const int depth = min(SS_K, n - k0);
+        for (int e = threadIdx.x; e < SS_K * SS_T; e += SS_THREADS) {
+            const int i = e / SS_K, k = e % SS_K;
+            a[k][i] = k < depth && i < c.n ? cb[((size_t)(c.t0 + i) * 2 * groups + g) * n + k0 + k] * w[i] : 0.f;
+            b[k][i] = k < depth && p0 + i < vdim ? S[(size_t)(p0 + i) * n + k0 + k] : 0.f;
+        }
+        __syncthreads();
+        tile_step(acc, a, b, depth);
+        __syncthreads();
+    }
+    const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+    const float d = skip[h];
+#pragma unroll
+    for (int i = 0; i < 8; ++i) {
+        const int r = ty * 8 + i;
+        if (r >= c.n) break;
+        const size_t at = ((size_t)(c.t0 + r) * heads + h) * vdim + p0 + tx * 4;
+#pragma unroll
+        for (int k = 0; k < 4; ++k) if (p0 + tx * 4 + k < vdim) y[at + k] = fmaf(d, x[at + k], acc[i][k]);
+    }
+}
+
+extern "C" size_t hb_state_space_prompt_scratch_floats(int tiles, int heads, int groups, int n, int vdim) {
+    return (size_t)tiles * ((size_t)heads * vdim * n + (size_t)groups * SS_Q * SS_Q + heads);
+}
+
+extern "C" int hb_state_space_prompt(float* y, const float* cb, const float* x, const float* dt, const float* rate_log, const float* skip,
+                                     float* state, float* scratch, const int32_t* query_start, const int32_t* row_slot, int row0,
+                                     int rows, int tiles, int heads, int groups, int n, int vdim, hb_stream stream) {
+    if (rows <= row0 || tiles == 0) return 0;
+    if (groups < 1 || heads % groups || n < 1 || vdim < 1) HB_REFUSE("state_space_prompt: %d heads of %d, %d groups of %d", heads, vdim, groups, n);
+    if (!scratch || ((uintptr_t)scratch & 15) || ((uintptr_t)state & 15)) HB_REFUSE("state_space_prompt: scratch and state must lie on 16-byte boundaries");
+    const int p_tiles = (vdim + SS_T - 1) / SS_T, n_tiles = (n + SS_T - 1) / SS_T;
+    if (heads > 65535 || (long)p_tiles * n_tiles > 65535) HB_REFUSE("state_space_prompt: %d heads of %d x %d", heads, vdim, n);
+    const int size = vdim * n;
+    float* products = scratch;                                     // [tiles][groups][64][64]
+    float* own = products + (size_t)tiles * groups * SS_Q * SS_Q;  // [tiles][heads][vdim][n]
+    float* last = own + (size_t)tiles * heads * size;              // [tiles][heads]
+    cudaStream_t s = (cudaStream_t)stream;
+    ss_products_kernel<<<dim3(tiles, groups), SS_THREADS, 0, s>>>(products, cb, query_start, row0, rows, groups, n);
+    HB_LAUNCH_CHECK("state_space_products");
+    ss_own_kernel<<<dim3(tiles, heads, p_tiles * n_tiles), SS_THREADS, 0, s>>>(own, last, cb, x, dt, rate_log, query_start, row0, rows, heads,
+                                                                               groups, n, vdim, n_tiles);
+    HB_LAUNCH_CHECK("state_space_own");
+    const bool vec = size % 4 == 0;
+    const int elements = vec ? size / 4 : size, slices = (elements + 127) / 128;
+    if (slices > 65535) HB_REFUSE("state_space_prompt: states of %d numbers", size);
+    if (vec) ss_walk_kernel<true><<<dim3(rows - row0, heads, slices), 128, 0, s>>>(own, last, state, query_start, row_slot, row0, heads, size);
+    else ss_walk_kernel<false><<<dim3(rows - row0, heads, slices), 128, 0, s>>>(own, last, state, query_start, row_slot, row0, heads, size);
+    HB_LAUNCH_CHECK("state_space_walk");
+    ss_out_kernel<<<dim3(tiles, heads, p_tiles), SS_THREADS, 0, s>>>(y, products, own, cb, x, dt, rate_log, skip, query_start, row0, rows, heads,
+                                                                     groups, n, vdim);
+    HB_LAUNCH_CHECK("state_space_out");
+    return 0;
+}

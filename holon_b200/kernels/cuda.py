@@ -721,6 +721,29 @@ class CudaKernels:
         else:
             torch.mm(x, weight.t(), out=out)
 
+    def linear_relu2(self, out, x, weight) -> bool:
+        """out = max(x · weightᵀ, 0)² in one kernel where the product runs on one of the library's own (a decode step's few rows, prompts
+        of the row counts at which SwiGLU's product stays here too); False, with nothing done, elsewhere."""
+        m, k = x.shape
+        n = weight.shape[0]
+        if x.dtype != torch.bfloat16 or k % 8 or self.gemm == "cublas" or m == 0 or self._pending:
+            return False
+        self._check(out, x, weight)
+        if weight.shape != (n, k) or out.shape != (m, n) or not (x.dtype == weight.dtype == out.dtype):
+            raise KernelError(f"linear_relu2: x {tuple(x.shape)} · w {tuple(weight.shape)}ᵀ -> out {tuple(out.shape)} do not fit")
+        args = (self._p(out), 0, self._p(x), self._p(weight), m, n, k, 5, 0)
+        if m <= self.SKINNY_ROWS:
+            self._call("hb_gemm_bf16_skinny", *args)
+        elif self._wide_takes(m, weight):
+            self._call("hb_gemm_bf16_skinny32", *args, None, None, 0, ctypes.c_float(0.0), None, None, 0, ctypes.c_float(0.0), 0)
+        elif self.gemm == "tcgen05" or 192 < m <= 6144:
+            self._call("hb_gemm_bf16_tcgen05_pair" if self.gemm_pair else "hb_gemm_bf16_tcgen05", *args)
+        elif 96 < m <= 192:
+            self._call("hb_gemm_bf16_tcgen05", *args)
+        else:
+            return False
+        return True
+
     SKINNY_ROWS = 16
     MID_ROWS = 64                             # rows the clustered tcgen05 products take (csrc/gemm_mid.cu)
 
@@ -1185,6 +1208,29 @@ class CudaKernels:
                    ctypes.c_long(first.shape[1]), int(at), self._p(conv), self._p(conv_bias), taps, self._p(conv_state),
                    self._p(dt_bias), self._p(rate_log), self._i32(rows.query_start, "query_start"),
                    self._i32(rows.row_slot, "row_slot"), rows.n_rows, t, heads, vdim, groups, n)
+
+    def state_space_scan(self, out, cb, v, dt, decay, rate_log, skip, state, rows) -> None:
+        """S ← decay · S + dt · B vᵀ, out = Sᵀ C + skip · v per head, cb [tokens, 2, groups, n] = (C, B), decay = exp(−exp(rate_log) dt):
+        rows of one token by the scan, rows of several in chunks (csrc/state_space.cu)."""
+        ones, portions = rows.n_decode, rows.n_rows > rows.n_decode
+        self._check(out, cb, v, dt, decay, rate_log, skip, state, rows.query_start, rows.row_slot)
+        self._f32("state_space_scan", out, cb, v, dt, decay, rate_log, skip, state)
+        t, heads, vdim = v.shape
+        groups, n = cb.shape[2], cb.shape[3]
+        if cb.shape != (t, 2, groups, n) or out.shape != v.shape or state.shape[1:] != (heads, vdim, n) or dt.shape != (t, heads) \
+                or decay.shape != (t, heads) or rate_log.shape != (heads,) or skip.shape != (heads,):
+            raise KernelError("state_space_scan: cb [tokens, 2, groups, n], v and out [tokens, heads, vdim], dt and decay [tokens, heads], "
+                              "rate_log and skip [heads], state [slots, heads, vdim, n]")
+        if ones:
+            self._call("hb_recurrent_scan", self._p(out), self._p(cb), self._p(v), None, None, self._p(decay), None, None, self._p(dt),
+                       self._p(skip), self._p(state), self._i32(rows.query_start, "query_start"), self._i32(rows.row_slot, "row_slot"),
+                       ones, heads, groups, n, vdim, 1)
+        if portions:
+            tiles = self._query_tiles(rows, 64)
+            scratch = torch.empty(tiles * (heads * vdim * n + groups * 64 * 64 + heads), dtype=torch.float32, device=self.device)
+            self._call("hb_state_space_prompt", self._p(out), self._p(cb), self._p(v), self._p(dt), self._p(rate_log), self._p(skip),
+                       self._p(state), self._p(scratch), self._i32(rows.query_start, "query_start"),
+                       self._i32(rows.row_slot, "row_slot"), ones, rows.n_rows, tiles, heads, groups, n, vdim)
 
     def retention_prepare(self, qk, v, first, positions, table, rot_dims, k_scale, silu=False) -> None:
         """`silu`: q, k and v pass silu before anything else (csrc/api.h: hb_retention_prepare)."""

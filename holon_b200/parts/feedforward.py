@@ -4,7 +4,8 @@
 ClampedGLU: a gated unit whose inputs are clamped, with a bias on every projection: g = min(W_gate x + b, limit),
 u = clamp(W_up x + b, −limit, limit), y = g · sigmoid(alpha · g) · (u + 1), output W_down y + b.
 
-MLP: W_down act(W_up x), no gate and no bias; `activation` as the experts name theirs ("gelu_tanh": the tanh form of
+MLP: W_down act(W_up x), no gate and no bias; `activation` as the experts name theirs ("relu2": the squared relu, which may ride in
+the first product's epilogue; "gelu_tanh": the tanh form of
 gelu, 0.5 z (1 + tanh(√(2/π) (z + 0.044715 z³))); "xielu": with two stored numbers p, q (`act`), softplus(p) z² + z/2 for
 z > 0 and (1/2 + softplus(q)) (exp(z) − 1 − z) + z/2 otherwise)."""
 from __future__ import annotations
@@ -71,7 +72,7 @@ class MLP(Part):
         from .experts import ACTIVATIONS
         if activation not in ACTIVATIONS:
             raise ValueError(f"mlp: activation {activation!r}; known: {sorted(ACTIVATIONS)}")
-        self.ctx, self.inter, self.act = ctx, inter, ACTIVATIONS[activation]
+        self.ctx, self.inter, self.act, self.squared_relu = ctx, inter, ACTIVATIONS[activation], activation == "relu2"
         self.numbers = self.add_param("act", (2,), "coef") if activation == "xielu" else None
         self.up = self.add_child("up_proj", Linear(ctx, "weight", hidden, {"up": inter}))
         self.down = self.add_child("down_proj", Linear(ctx, "weight", inter, {"down": hidden}))
@@ -84,6 +85,11 @@ class MLP(Part):
             yield name, p, rows
 
     def forward(self, x: torch.Tensor, step) -> torch.Tensor:
+        fused = getattr(self.ctx.kernels, "linear_relu2", None) if self.squared_relu else None
+        if fused is not None:                                            # a kernel table may do product and activation in one
+            z = self.ctx.empty(x.shape[0], self.inter)
+            if fused(z, x, self.up.weight.tensor):
+                return self.down.forward(z)
         z = self.up.forward(x)
         if self.numbers is not None:
             self.ctx.kernels.activation(z, self.act, self.numbers.tensor)

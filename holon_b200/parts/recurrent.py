@@ -43,7 +43,8 @@ dt = softplus(its projection + dt_bias) per token, and B, C [state] shared by th
 
 x, B and C pass one short causal convolution over time with a bias (its last taps − 1 inputs are carried per request) and silu;
 all heads' y times silu(z), then an RMS norm over each of `norm_groups` equal parts of the row with a weight over the whole of
-it, then W_o. dt is a factor on what the scan writes (`recurrent_scan(take=)`), D a skip in its read-out.
+it, then W_o. Rows of one token run on the scan (dt a factor on what it writes, D a skip in its read-out), rows of several in chunks
+of 64 tokens, whose outputs are products over the chunk and over the state before it.
 
 Everything that enters the recurrence is 32-bit (the scan's inputs are made in 32-bit from the first product's rows);
 the products themselves are the engine's. All first projections of a mixer are one merged product.
@@ -330,8 +331,7 @@ class StateSpace(_MatrixState):
         if step.rows.n_rows > step.rows.n_decode:                        # (rows of one token: moved on by the kernel above)
             k.conv_carry(carried, first, self.channels, self.taps, step.rows, least=2, at=inner)
         y = ctx.empty(t, heads, vdim, dtype=f32)
-        k.recurrent_scan(y, cb, v, None, None, None, cache.slots["state"], step.rows, token_decay=decay, take=dt,
-                         skip=self.skip.tensor)
+        k.state_space_scan(y, cb, v, dt, decay, self.rate_log.tensor, self.skip.tensor, cache.slots["state"], step.rows)
         n = self.norm_groups
         out = ctx.empty(t, n, inner // n)
         k.head_norm_gate(out, y.view(t, n, inner // n), self.gain.tensor, None, first[:, :inner], self.eps, gate_first=True)

@@ -230,6 +230,9 @@ class RefKernels:
         dt.copy_(torch.nn.functional.softplus(first[:, at + channels:].float() + dt_bias))
         decay.copy_(torch.exp(-torch.exp(rate_log) * dt))
 
+    def state_space_scan(self, out, cb, v, dt, decay, rate_log, skip, state, rows):
+        self.recurrent_scan(out, cb, v, None, None, None, state, rows, token_decay=decay, take=dt, skip=skip)
+
     def conv_carry(self, conv_state, first, channels, taps, rows, least=0, at=0):
         if taps <= 1:
             return

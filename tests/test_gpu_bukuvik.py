@@ -84,6 +84,23 @@ def test_norm_of_a_pair_and_of_one_output(K, dtype, rows, dim, weight32):
     close(dst, src.to(F64) + unit(z, 1e-6) * (w.to(F64) + 0.25), torch.float32)
 
 
+# ---------------------------------------------------------------- the squared relu in the first product
+@pytest.mark.parametrize("m,n,k", [(1, 96, 64), (8, 20000, 64), (9, 330, 256), (16, 48, 40), (20, 520, 128), (32, 100, 72), (100, 256, 64), (150, 1000, 320),
+                                   (300, 513, 128), (2048, 640, 512), (7000, 64, 64), (40, 64, 64), (5, 50, 33)])
+@pytest.mark.parametrize("pair", [True, False])
+def test_squared_relu_in_the_product(K, m, n, k, pair, monkeypatch):
+    monkeypatch.setattr(K, "gemm_pair", pair)
+    x, w = rand(m, k, dtype=torch.bfloat16, seed=1), rand(n, k, dtype=torch.bfloat16, seed=2, scale=k ** -0.5)
+    out = torch.full((m, n), float("nan"), dtype=torch.bfloat16, device=DEV)
+    took = K.linear_relu2(out, x.to(DEV), w.to(DEV))
+    assert took == (k % 8 == 0 and (m <= 32 or 96 < m <= 6144))
+    if took:
+        want = torch.relu(x.to(F64) @ w.to(F64).T) ** 2
+        d = (out.cpu().to(F64) - want).abs()
+        assert bool((d <= 2 ** -8 * want + 1e-4).all())
+        assert K.tcgen05_status() == 0
+
+
 # ---------------------------------------------------------------- state space
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("heads,groups,n,vdim,taps", [(6, 2, 48, 20, 3), (4, 4, 16, 8, 4), (3, 1, 7, 5, 1), (5, 5, 3, 2, 6), (8, 1, 128, 64, 4), (2, 1, 130, 33, 2)])
@@ -113,9 +130,9 @@ def test_state_space_inputs_and_carried_rows(K, dtype, heads, groups, n, vdim, t
 
 
 @pytest.mark.parametrize("heads,groups,n,vdim", [(4, 2, 16, 12), (3, 1, 7, 5), (8, 2, 128, 64), (2, 2, 1, 3), (2, 1, 96, 40), (4, 1, 256, 128), (2, 1, 300, 17)])
-@pytest.mark.parametrize("counts,lens", [([1, 1, 1], None), ([37], None), ([1, 1, 5, 200], None), ([64, 129], None), ([2, 63, 65, 300], None)])
-def test_scan_with_step_sizes_and_skips(K, heads, groups, n, vdim, counts, lens):
-    """The scan against the rule in 64-bit: step sizes from 1e-4 to several units, rates that forget at once and rates that keep
+@pytest.mark.parametrize("counts", [[1, 1, 1], [37], [1, 1, 5, 200], [64, 129], [2, 63, 65, 300], [1, 513]])
+def test_scan_with_step_sizes_and_skips(K, heads, groups, n, vdim, counts):
+    """The scan and its form in chunks against the rule in 64-bit: step sizes from 1e-4 to several units, rates that forget at once and rates that keep
     hundreds of tokens, states that are not empty at the start."""
     t, slots = sum(counts), [4, 1, 3, 0][:len(counts)]
     cb, v = rand(t, 2, groups, n, seed=1), rand(t, heads, vdim, seed=2)
@@ -133,13 +150,16 @@ def test_scan_with_step_sizes_and_skips(K, heads, groups, n, vdim, counts, lens)
             S = decay[i].to(F64)[:, None, None] * S + (dt[i].to(F64)[:, None] * x)[:, :, None] * B[:, None, :]
             want[i] = (S * C[:, None, :]).sum(-1) + skip.to(F64)[:, None] * x
         after[slot], at = S, at + count
-    out = torch.full((t, heads, vdim), float("nan"), device=DEV)
-    state = state0.to(DEV)
-    K.recurrent_scan(out, cb.to(DEV), v.to(DEV), None, None, None, state, rows_of(counts, slots), token_decay=decay.to(DEV),
-                     take=dt.to(DEV), skip=skip.to(DEV))
-    scale = 1.0 + float(want.abs().max())
-    close(out, want, torch.float32, scale=scale)
-    close(state, after, torch.float32, scale=1.0 + float(after.abs().max()))
+    for chunks in (False, True):
+        out = torch.full((t, heads, vdim), float("nan"), device=DEV)
+        state = state0.to(DEV)
+        if chunks:
+            K.state_space_scan(out, cb.to(DEV), v.to(DEV), dt.to(DEV), decay.to(DEV), rate_log.to(DEV), skip.to(DEV), state, rows_of(counts, slots))
+        else:
+            K.recurrent_scan(out, cb.to(DEV), v.to(DEV), None, None, None, state, rows_of(counts, slots), token_decay=decay.to(DEV),
+                             take=dt.to(DEV), skip=skip.to(DEV))
+        close(out, want, torch.float32, scale=0.2 * (1.0 + float(want.abs().max())))
+        close(state, after, torch.float32, scale=0.2 * (1.0 + float(after.abs().max())))
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
