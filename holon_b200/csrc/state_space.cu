@@ -47,6 +47,38 @@ __device__ __forceinline__ void tile_step(float (&acc)[8][4], const float (*a)[S
     }
 }
 
+// Slices travel through registers (the next one is on its way while the current one is multiplied), 16 bytes a load: four quads a
+// thread and operand. `along`: the operand's memory runs along k (element (row i, k) at p[i * stride + k]); a thread then holds quads
+// of one row, and the stores to [k][i] go to neighbouring banks. Else it runs along the tile's rows (element (k, i) at p[k * stride + i]).
+struct Quads { float4 v[4]; };
+__device__ __forceinline__ float4 load_quad(const float* p, int left, bool vec) {        // zeros from `left` on
+    if (vec && left >= 4) return *(const float4*)p;
+    return make_float4(left > 0 ? p[0] : 0.f, left > 1 ? p[1] : 0.f, left > 2 ? p[2] : 0.f, left > 3 ? p[3] : 0.f);
+}
+__device__ __forceinline__ void fetch_along(Quads& q, const float* p, size_t stride, int rows, int depth, bool vec) {
+    const int i = threadIdx.x & 63, k = (threadIdx.x >> 6) * 4;
+#pragma unroll
+    for (int r = 0; r < 4; ++r) q.v[r] = load_quad(p + i * stride + k + 8 * r, i < rows ? depth - k - 8 * r : 0, vec);
+}
+__device__ __forceinline__ void store_along(float (*a)[SS_T + SS_PAD], const Quads& q) {
+    const int i = threadIdx.x & 63, k = (threadIdx.x >> 6) * 4;
+#pragma unroll
+    for (int r = 0; r < 4; ++r) {
+        a[k + 8 * r][i] = q.v[r].x; a[k + 8 * r + 1][i] = q.v[r].y; a[k + 8 * r + 2][i] = q.v[r].z; a[k + 8 * r + 3][i] = q.v[r].w;
+    }
+}
+__device__ __forceinline__ void fetch_across(Quads& q, const float* p, size_t stride, int rows, int depth, bool vec) {
+    const int i = (threadIdx.x & 15) * 4, k = threadIdx.x >> 4;
+#pragma unroll
+    for (int r = 0; r < 4; ++r) q.v[r] = load_quad(p + (k + 8 * r) * stride + i, k + 8 * r < depth ? rows - i : 0, vec);
+}
+__device__ __forceinline__ void store_across(float (*a)[SS_T + SS_PAD], const Quads& q) {
+    const int i = (threadIdx.x & 15) * 4, k = threadIdx.x >> 4;
+#pragma unroll
+    for (int r = 0; r < 4; ++r) *(float4*)&a[k + 8 * r][i] = q.v[r];
+}
+__device__ __forceinline__ void scale_quad(float4& v, float f) { v.x *= f; v.y *= f; v.z *= f; v.w *= f; }
+
 // L_i of a chunk's tokens for one head, by warp 0: hi + lo in two floats; tokens past the chunk repeat the last.
 __device__ __forceinline__ void log_decays(float* hi, float* lo, float* steps, const float* __restrict__ dt, const Chunk& c, int heads,
                                            int h, float rate) {
@@ -76,17 +108,21 @@ __global__ void __launch_bounds__(SS_THREADS) ss_products_kernel(float* __restri
     if (c.row < 0) return;
     const int g = blockIdx.y;
     float acc[8][4] = {};
+    Quads qa, qb;
+    const float* src = cb + ((size_t)c.t0 * 2 * groups + g) * n;
+    const size_t stride = (size_t)2 * groups * n;
+    const bool vec = (n & 3) == 0;
+    fetch_along(qa, src, stride, c.n, n, vec);
+    fetch_along(qb, src + (size_t)groups * n, stride, c.n, n, vec);
     for (int k0 = 0; k0 < n; k0 += SS_K) {
-        const int depth = min(SS_K, n - k0);
-        for (int e = threadIdx.x; e < SS_T * SS_K; e += SS_THREADS) {
-            const int i = e / SS_K, k = e % SS_K;
-            const bool in = i < c.n && k < depth;
-            const float* src = cb + ((size_t)(c.t0 + i) * 2 * groups + g) * n + k0 + k;
-            a[k][i] = in ? src[0] : 0.f;
-            b[k][i] = in ? src[(size_t)groups * n] : 0.f;
-        }
+        store_along(a, qa);
+        store_along(b, qb);
         __syncthreads();
-        tile_step(acc, a, b, depth);
+        if (k0 + SS_K < n) {
+            fetch_along(qa, src + k0 + SS_K, stride, c.n, n - k0 - SS_K, vec);
+            fetch_along(qb, src + (size_t)groups * n + k0 + SS_K, stride, c.n, n - k0 - SS_K, vec);
+        }
+        tile_step(acc, a, b, min(SS_K, n - k0));
         __syncthreads();
     }
     const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
@@ -116,16 +152,24 @@ __global__ void __launch_bounds__(SS_THREADS) ss_own_kernel(float* __restrict__ 
     }
     __syncthreads();
     float acc[8][4] = {};
+    Quads qa, qb;
+    const size_t xs = (size_t)heads * vdim, bs = (size_t)2 * groups * n;
+    const float* xp = x + ((size_t)c.t0 * heads + h) * vdim + p0;
+    const float* bp = cb + (((size_t)c.t0 * 2 + 1) * groups + g) * n + n0;
+    const bool vx = (vdim & 3) == 0, vb = (n & 3) == 0;
+    fetch_across(qa, xp, xs, vdim - p0, c.n, vx);
+    fetch_across(qb, bp, bs, n - n0, c.n, vb);
     for (int k0 = 0; k0 < c.n; k0 += SS_K) {
-        const int depth = min(SS_K, c.n - k0);
-        for (int e = threadIdx.x; e < SS_K * SS_T; e += SS_THREADS) {
-            const int k = e / SS_T, i = e % SS_T;
-            const size_t t = (size_t)(c.t0 + k0 + k);
-            a[k][i] = k < depth && p0 + i < vdim ? x[(t * heads + h) * vdim + p0 + i] * w[k0 + k] : 0.f;
-            b[k][i] = k < depth && n0 + i < n ? cb[((t * 2 + 1) * groups + g) * n + n0 + i] : 0.f;
-        }
+#pragma unroll
+        for (int r = 0; r < 4; ++r) scale_quad(qa.v[r], w[min(k0 + ((int)threadIdx.x >> 4) + 8 * r, SS_Q - 1)]);
+        store_across(a, qa);
+        store_across(b, qb);
         __syncthreads();
-        tile_step(acc, a, b, depth);
+        if (k0 + SS_K < c.n) {
+            fetch_across(qa, xp + (k0 + SS_K) * xs, xs, vdim - p0, c.n - k0 - SS_K, vx);
+            fetch_across(qb, bp + (k0 + SS_K) * bs, bs, n - n0, c.n - k0 - SS_K, vb);
+        }
+        tile_step(acc, a, b, min(SS_K, c.n - k0));
         __syncthreads();
     }
     const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
@@ -196,30 +240,47 @@ __global__ void __launch_bounds__(SS_THREADS) ss_out_kernel(float* __restrict__ 
     __syncthreads();
     float acc[8][4] = {};
     const float* cbp = products + ((size_t)blockIdx.x * groups + g) * SS_Q * SS_Q;
-    for (int k0 = 0; k0 < c.n; k0 += SS_K) {                       // over the chunk's tokens j
-        const int depth = min(SS_K, c.n - k0);
-        for (int e = threadIdx.x; e < SS_K * SS_T; e += SS_THREADS) {
-            const int i = e / SS_K, k = e % SS_K, j = k0 + k;       // weight of token j in row i
-            a[k][i] = j <= i && j < c.n ? cbp[i * SS_Q + j] * expf((hi[i] - hi[j]) + (lo[i] - lo[j])) * steps[j] : 0.f;
+    const float* xp = x + ((size_t)c.t0 * heads + h) * vdim + p0;
+    const float* cp = cb + ((size_t)c.t0 * 2 * groups + g) * n;
+    const float* sp = before + (((size_t)blockIdx.x * heads + h) * vdim + p0) * n;
+    const size_t xs = (size_t)heads * vdim, cs = (size_t)2 * groups * n;
+    const bool vx = (vdim & 3) == 0, vn = (n & 3) == 0;
+    const int own_slices = (c.n + SS_K - 1) / SS_K, slices = own_slices + (n + SS_K - 1) / SS_K;
+    Quads qa, qb;
+    auto fetch = [&](int s) {
+        if (s < own_slices) {                                       // over the chunk's tokens j
+            const int k0 = s * SS_K;
+            fetch_along(qa, cbp + k0, SS_Q, SS_Q, SS_K, true);
+            fetch_across(qb, xp + k0 * xs, xs, vdim - p0, c.n - k0, vx);
+        } else {                                                    // over the state's channels
+            const int k0 = (s - own_slices) * SS_K;
+            fetch_along(qa, cp + k0, cs, c.n, n - k0, vn);
+            fetch_along(qb, sp + k0, n, vdim - p0, n - k0, vn);
         }
-        for (int e = threadIdx.x; e < SS_K * SS_T; e += SS_THREADS) {
-            const int k = e / SS_T, i = e % SS_T;
-            b[k][i] = k < depth && p0 + i < vdim ? x[((size_t)(c.t0 + k0 + k) * heads + h) * vdim + p0 + i] : 0.f;
+    };
+    fetch(0);
+    const int row = threadIdx.x & 63, kq = (threadIdx.x >> 6) * 4;
+    for (int s = 0; s < slices; ++s) {
+        if (s < own_slices) {                                       // weight of token j in row i: C_i . B_j exp(L_i - L_j) dt_j, j <= i
+            const float hr = hi[row], lr = lo[row];
+#pragma unroll
+            for (int r = 0; r < 4; ++r) {
+                const int j = s * SS_K + kq + 8 * r;
+                auto weight = [&](int jj, float v) -> float { return jj <= row && jj < c.n ? v * expf((hr - hi[jj]) + (lr - lo[jj])) * steps[jj] : 0.f; };
+                qa.v[r].x = weight(j, qa.v[r].x); qa.v[r].y = weight(j + 1, qa.v[r].y);
+                qa.v[r].z = weight(j + 2, qa.v[r].z); qa.v[r].w = weight(j + 3, qa.v[r].w);
+            }
+        } else {
+            const float f = w[row];
+#pragma unroll
+            for (int r = 0; r < 4; ++r) scale_quad(qa.v[r], f);
         }
+        store_along(a, qa);
+        if (s < own_slices) store_across(b, qb); else store_along(b, qb);
         __syncthreads();
-        tile_step(acc, a, b, depth);
-        __syncthreads();
-    }
-    const float* S = before + ((size_t)blockIdx.x * heads + h) * vdim * n;
-    for (int k0 = 0; k0 < n; k0 += SS_K) {                         // over the state's channels
-        const int depth = min(SS_K, n - k0);
-        for (int e = threadIdx.x; e < SS_K * SS_T; e += SS_THREADS) {
-            const int i = e / SS_K, k = e % SS_K;
-            a[k][i] = k < depth && i < c.n ? cb[((size_t)(c.t0 + i) * 2 * groups + g) * n + k0 + k] * w[i] : 0.f;
-            b[k][i] = k < depth && p0 + i < vdim ? S[(size_t)(p0 + i) * n + k0 + k] : 0.f;
-        }
-        __syncthreads();
-        tile_step(acc, a, b, depth);
+        if (s + 1 < slices) fetch(s + 1);
+        // (the second half of a chunk's tokens weighs nothing in its first half's rows)
+        if (s >= own_slices || s == 0 || (int)(threadIdx.x >> 5) * 16 + 15 >= s * SS_K) tile_step(acc, a, b, SS_K);
         __syncthreads();
     }
     const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;

@@ -4,6 +4,9 @@
     python -m holon_b200.kernels.microbench gemm [--rows 2048] [--shapes qkv o gate_up down]
     python -m holon_b200.kernels.microbench prefill_attention [--rows 2048] [--context 2048]
     python -m holon_b200.kernels.microbench layer [--rows 8 1 16 64] [--context 8192]
+    python -m holon_b200.kernels.microbench maps [--rows 2048 1] [--heads 16 --kv-heads 4 --window 1024 --context 2048]
+    python -m holon_b200.kernels.microbench state_space [--rows 2048 1] [--heads 32 --kv-heads 4 --dim 128 --vdim 64]
+    python -m holon_b200.kernels.microbench out_norm [--rows 8 2048 8192] [--hidden 2048]
     python -m holon_b200.kernels.microbench scan [--rows 2048 256 1] [--heads 16 --kv-heads 4 --dim 128 --vdim 128]
 
 `layer` times the kernels of a decode layer the way a step runs them: back to back inside a CUDA graph, each launch
@@ -434,6 +437,103 @@ def layernorm(k, args) -> None:
             print(f"layernorm {t:6d} rows of {dim}, {name:18s}: {us:7.1f} us  ({moved / us / 1e3:7.0f} GB/s)")
 
 
+def _rows_on(dev, counts, lens) -> Rows:
+    starts = [sum(counts[:i]) for i in range(len(counts) + 1)]
+    t = lambda v: torch.tensor(v, device=dev, dtype=torch.int32)          # noqa: E731
+    return Rows(t(list(range(len(counts)))), t(starts), t(lens), len(counts), starts[-1], sum(1 for n in counts if n == 1), max(counts),
+                max(lens), starts, lens)
+
+
+def maps(k, args) -> None:
+    """Attention with maps (`attention_maps`, `qkv_maps_prepare`): two maps of 64 over values of 128 under a cap, one map of 128 with
+    16 kept tokens, and beside them `paged_attention` with heads of 128 and a sink; a window of `--window`. `--rows` 1: eight rows of
+    one token over `--context` tokens each, on caches in turn that are larger than the L2; else one prompt of that many tokens."""
+    dev, heads, kvh, page, w = k.device, args.heads, args.kv_heads, 64, args.window
+    bf = dict(device=dev, dtype=torch.bfloat16)
+    for tokens in args.rows:
+        counts, n = ([1] * 8, args.context) if tokens == 1 else ([tokens], tokens)
+        t, per = sum(counts), -(-n // page)
+        batch = _rows_on(dev, counts, [n] * len(counts))
+        table = torch.arange(len(counts) * per, device=dev, dtype=torch.int32).view(len(counts), per).contiguous()
+        sets = 8 if tokens == 1 else 2
+        gate = torch.randn(t, heads * 128, **bf)
+        sink = torch.zeros(heads, device=dev)
+        out = torch.empty(t, heads, 128, **bf)
+        seen = sum(min(i + 1, w) for i in range(n)) if tokens > 1 else t * min(n, w)
+        for name, m, d in (("two maps of 64, cap", 2, 64), ("one map of 128, kept", 1, 128), ("paged_attention", 0, 128)):
+            shape = (len(counts) * per + 1, kvh, page, m * d + 128) if m else (len(counts) * per + 1, 2, kvh, page, 128)
+            caches = [torch.randn(*shape, **bf) for _ in range(sets)]
+            q = torch.randn(t, heads, m, d, **bf) if m else torch.randn(t, heads, d, **bf)
+            def call(kv):                                                 # noqa: E306
+                if m:
+                    k.attention_maps(out, q, kv, table, batch, d ** -0.5, 50.0 if m == 2 else None, w, 16 if m == 1 else 0,
+                                     (0.5, 0.5) if m == 2 else None, 1e-6, gate)
+                else:
+                    k.paged_attention(out, q, kv, table, batch, d ** -0.5, w, sink)
+            us = in_graph([lambda kv=kv: call(kv) for kv in caches])
+            flops = 2 * seen * heads * ((m or 1) * d + (m or 1) * 128)
+            moved = 2 * (seen * kvh * ((m or 1) * d + 128) if tokens == 1 else n * kvh * ((m or 1) * d + 128) + t * heads * ((m or 1) * d + 256))
+            print(f"{name:22s} {len(counts)} row(s) of {counts[0]:5d}, {n} keys, window {w}: {us:8.1f} us  {flops / us / 1e6:7.1f} TFLOP/s  {moved / us / 1e3:7.0f} GB/s")
+            if not m:
+                continue
+            first = torch.randn(t, heads * m * d + kvh * (m * d + 128) + heads * 128, **bf)
+            rot = torch.randn(n + 1, d, device=dev)
+            pos, write = torch.arange(t, device=dev, dtype=torch.int32) % n, torch.arange(t, device=dev, dtype=torch.int32)
+            gain = torch.ones(d, device=dev)
+            us = in_graph([lambda kv=kv: k.qkv_maps_prepare(q, kv, first, gain if m == 2 else None, gain if m == 2 else None, 1e-6,
+                                                           "before" if m == 2 else "after", pos, rot, d, write, kvh, 128) for kv in caches])
+            moved = 4 * t * (heads * m * d + kvh * (m * d + 128))
+            print(f"{name:22s} preparation: {us:8.1f} us  {moved / us / 1e3:7.0f} GB/s")
+    print("tcgen05 status", k.tcgen05_status())
+
+
+def state_space(k, args) -> None:
+    """A state space's kernels: heads of `--vdim` over a state of `--dim`, `--kv-heads` groups; one prompt of `--rows` tokens (1: eight
+    rows of one token): preparation, recurrence (and the scan token by token), gate and norm."""
+    dev, heads, groups, n, vdim, taps = k.device, args.heads, args.kv_heads, args.dim, args.vdim, 4
+    for tokens in args.rows:
+        counts = [1] * 8 if tokens == 1 else [tokens]
+        t, inner, channels = sum(counts), heads * vdim, heads * vdim + 2 * groups * n
+        batch = _rows_on(dev, counts, counts)
+        first = torch.randn(t, inner + channels + heads, device=dev, dtype=torch.bfloat16)
+        conv, bias = torch.randn(channels, taps, device=dev).bfloat16(), torch.randn(channels, device=dev).bfloat16()
+        carried = torch.zeros(len(counts), taps - 1, channels, device=dev, dtype=torch.bfloat16)
+        f = lambda *s: torch.empty(*s, device=dev)                        # noqa: E731
+        cb, v, dt, decay, y = f(t, 2, groups, n), f(t, heads, vdim), f(t, heads), f(t, heads), f(t, heads, vdim)
+        bias_dt, rate, skip = torch.randn(heads, device=dev), torch.randn(heads, device=dev), torch.ones(heads, device=dev)
+        state = torch.zeros(len(counts), heads, vdim, n, device=dev)
+        out, gain = torch.empty(t, groups, inner // groups, device=dev, dtype=torch.bfloat16), torch.ones(inner, device=dev)
+        cases = (("preparation", t * (2 * (channels + heads) + 4 * (channels + 2 * heads)),
+                  lambda: k.state_space_prepare(cb, v, dt, decay, first, inner, conv, bias, carried, bias_dt, rate, batch)),
+                 ("recurrence", 4 * (t * (channels + inner) + 2 * state.numel()), lambda: k.state_space_scan(y, cb, v, dt, decay, rate, skip, state, batch)),
+                 ("scan by token", 4 * (t * (channels + inner) + 2 * state.numel()),
+                  lambda: k.recurrent_scan(y, cb, v, None, None, None, state, batch, token_decay=decay, take=dt, skip=skip)),
+                 ("gate and norm", t * inner * 8, lambda: k.head_norm_gate(out, y.view(out.shape), gain, None, first[:, :inner], 1e-6, gate_first=True)))
+        for name, moved, fn in cases:
+            us = in_graph([fn], 4)
+            print(f"state space {len(counts)} row(s) of {counts[0]:5d} tokens, {heads} heads of {n} x {vdim}, {name:14s}: {us:8.1f} us  ({moved / us / 1e3:7.0f} GB/s)")
+
+
+def out_norm(k, args) -> None:
+    """The norm on an output that is added to the stream (`out_norm_add`), and on a pair of outputs (`out_norm_pair_add`), beside
+    `add_rmsnorm`, over rows of `--hidden`. Two sets of buffers alternate; many rows are larger than the L2."""
+    from ..parts.base import NormedPair
+    dev, dim = k.device, args.hidden
+    for t in args.rows:
+        sets = []
+        for _ in range(2):
+            a, b = torch.randn(t, dim, device=dev).bfloat16(), torch.randn(t, dim, device=dev).bfloat16()
+            sets.append((torch.randn(t, dim, device=dev), a, b, torch.empty(t, dim, device=dev, dtype=torch.bfloat16)))
+        w, gain = torch.ones(dim, device=dev, dtype=torch.bfloat16), torch.ones(dim, device=dev)
+        base = t * dim * (4 + 4 + 2)                                     # the stream in and out, its rows in 16 bits
+        cases = (("one output", base + 2 * t * dim, lambda h, a, b, out: k.out_norm_add(h, h, a, None, gain, 1e-6, 0.0, cast=out)),
+                 ("a pair", base + 4 * t * dim, lambda h, a, b, out: k.out_norm_pair_add(h, h, NormedPair(a, w, b, w, 1e-6, 0.5), gain, 1e-6, 0.0, cast=out)),
+                 ("add_rmsnorm", base + 2 * t * dim, lambda h, a, b, out: k.add_rmsnorm(out, h, a, w, 1e-6, 0.0, None)))
+        for name, moved, fn in cases:
+            us = in_graph([lambda s=s, fn=fn: fn(*s) for s in sets])
+            print(f"out_norm {t:6d} rows of {dim}, {name:12s}: {us:7.1f} us  ({moved / us / 1e3:7.0f} GB/s)")
+
+
 def expert_glu(k, args) -> None:
     """The clamped unit of routed experts (`expert_glu`: 32 experts, 4 a token, experts of three eighths of twice the width)
     beside the product with the unit in a kernel of its own."""
@@ -465,12 +565,13 @@ def expert_glu(k, args) -> None:
 
 def main() -> None:
     ap = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
-    ap.add_argument("what", choices=("decode_attention", "gemm", "prefill_attention", "chain", "layer", "scan", "layernorm", "expert_glu"))
+    ap.add_argument("what", choices=("decode_attention", "gemm", "prefill_attention", "chain", "layer", "scan", "layernorm", "expert_glu", "maps", "state_space", "out_norm"))
     ap.add_argument("--heads", type=int, default=16, help="scan: value heads")
     ap.add_argument("--kv-heads", type=int, default=4, help="scan: query/key heads of the delta rule")
     ap.add_argument("--dim", type=int, default=128, help="scan: key size")
     ap.add_argument("--vdim", type=int, default=128, help="scan: value size")
-    ap.add_argument("--hidden", type=int, default=2048, help="layernorm, expert_glu: the width")
+    ap.add_argument("--hidden", type=int, default=2048, help="layernorm, expert_glu, out_norm: the width")
+    ap.add_argument("--window", type=int, default=1024, help="maps: the window")
     ap.add_argument("--rows", type=int, nargs="*", default=None)
     ap.add_argument("--context", type=int, default=8192)
     ap.add_argument("--splits", type=int, nargs="*", default=None)
@@ -498,6 +599,15 @@ def main() -> None:
         elif args.what == "expert_glu":
             args.rows = args.rows or [1, 8, 2048]
             expert_glu(k, args)
+        elif args.what == "maps":
+            args.rows = args.rows or [2048, 1]
+            maps(k, args)
+        elif args.what == "state_space":
+            args.rows = args.rows or [2048, 1]
+            state_space(k, args)
+        elif args.what == "out_norm":
+            args.rows = args.rows or [8, 2048, 8192]
+            out_norm(k, args)
         elif args.what == "scan":
             args.rows = args.rows or [2048, 256, 1]
             scan(k, args)
