@@ -353,7 +353,7 @@ __device__ __forceinline__ void load_maps_tile(uint32_t k_s, uint32_t v_s, const
 }
 
 template <int KP, int VP, int STAGES>
-__global__ void __launch_bounds__(128) maps_decode_kernel(const MapsArgs a) {
+__global__ void __launch_bounds__(128, (KP + VP <= 256 ? 3 : 1)) maps_decode_kernel(const MapsArgs a) {
     extern __shared__ __align__(128) unsigned char smem_raw[];
     __shared__ float scratch[33];
     constexpr uint32_t K_BYTES = TILE_N * KP * 2, V_BYTES = TILE_N * VP * 2;
@@ -426,16 +426,37 @@ __global__ void __launch_bounds__(128) maps_decode_kernel(const MapsArgs a) {
                 mma_bf16(s[1], Q_IN_REGS ? qf[Q_IN_REGS ? ks : 0] : qa, kb[2], kb[3]);
             }
         }
-        const bool inside = key0 >= lo && key0 + 16 <= n;
+        if (a.cap > 0.f) {
+            const float to_x = a.scale / a.cap, from_x = a.cap * LOG2E;
+            float top = 0.f;
 #pragma unroll
-        for (int nt = 0; nt < 2; ++nt)
+            for (int nt = 0; nt < 2; ++nt)
 #pragma unroll
-            for (int e = 0; e < 4; ++e) {
-                float u = s[nt][e] * a.scale;
-                if (a.cap > 0.f) u = a.cap * tanhf(u / a.cap);
-                const int j = key0 + nt * 8 + (lane & 3) * 2 + (e & 1);
-                s[nt][e] = inside || (j < n && (j >= lo || j < a.keep)) ? u * LOG2E : -INFINITY;
-            }
+                for (int e = 0; e < 4; ++e) { s[nt][e] *= to_x; top = fmaxf(top, fabsf(s[nt][e])); }
+            const bool small = __all_sync(0xffffffffu, top <= 0.25f);
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const float x = s[nt][e], y = x * x;              // (the polynomial's error is below 3e-7 of the value here)
+                    s[nt][e] = from_x * (small ? x * fmaf(y, fmaf(y, fmaf(y, -17.f / 315.f, 2.f / 15.f), -1.f / 3.f), 1.f) : tanhf(x));
+                }
+        } else {
+            const float f = a.scale * LOG2E;
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) s[nt][e] *= f;
+        }
+        if (!(key0 >= lo && key0 + 16 <= n)) {                       // only tiles at an edge need the mask
+#pragma unroll
+            for (int nt = 0; nt < 2; ++nt)
+#pragma unroll
+                for (int e = 0; e < 4; ++e) {
+                    const int j = key0 + nt * 8 + (lane & 3) * 2 + (e & 1);
+                    if (!(j < n && (j >= lo || j < a.keep))) s[nt][e] = -INFINITY;
+                }
+        }
         float c0, c1;
         softmax_step<2>(s, m0, m1, l0, l1, 1.f, c0, c1);
         uint32_t p[4] = {pack_bf16(s[0][0], s[0][1]), pack_bf16(s[0][2], s[0][3]), pack_bf16(s[1][0], s[1][1]), pack_bf16(s[1][2], s[1][3])};
@@ -464,19 +485,22 @@ __global__ void __launch_bounds__(128) maps_decode_kernel(const MapsArgs a) {
     float* part_o = wml + 4 * 16 * 2;
     float* part_ml = part_o + 16 * VP;
     const int r0 = lane >> 2, cq = (lane & 3) * 2;
+    const bool up = r0 % hpm < g, down = (r0 + 8) % hpm < g;         // rows that hold a head
 #pragma unroll
     for (int i = 0; i < VP / 8; ++i) {
-        *(float2*)(wo + (warp * 16 + r0) * VP + i * 8 + cq) = make_float2(o[i][0], o[i][1]);
-        *(float2*)(wo + (warp * 16 + r0 + 8) * VP + i * 8 + cq) = make_float2(o[i][2], o[i][3]);
+        if (i * 8 < a.vdim) {
+            if (up) *(float2*)(wo + (warp * 16 + r0) * VP + i * 8 + cq) = make_float2(o[i][0], o[i][1]);
+            if (down) *(float2*)(wo + (warp * 16 + r0 + 8) * VP + i * 8 + cq) = make_float2(o[i][2], o[i][3]);
+        }
     }
     if ((lane & 3) == 0) {
         wml[(warp * 16 + r0) * 2] = m0; wml[(warp * 16 + r0) * 2 + 1] = l0;
         wml[(warp * 16 + r0 + 8) * 2] = m1; wml[(warp * 16 + r0 + 8) * 2 + 1] = l1;
     }
     __syncthreads();
-    for (int i = threadIdx.x; i < 16 * VP; i += 128) {
-        const int r = i / VP, d = i % VP;
-        if (r % hpm >= g || d >= a.vdim) continue;
+    for (int i = threadIdx.x; i < a.maps * g * VP; i += 128) {
+        const int d = i % VP, x = i / VP, r = x < g ? x : hpm + x - g;   // (map, head) pairs in a row
+        if (d >= a.vdim) continue;
         float mm = -INFINITY;
 #pragma unroll
         for (int w = 0; w < 4; ++w) mm = fmaxf(mm, wml[(w * 16 + r) * 2]);

@@ -14,7 +14,9 @@
 // their shares of the sum of squares through shared memory, scale, gate and store.
 //
 // The cap c tanh(s / c): where every |s / c| of a warp's tile is at most 1/4 a polynomial of degree 7 on packed pairs (its error is
-// below 3e-7 of the value there), else 1 - 2 / (1 + e^(2x)) on the special-function unit.
+// below 3e-7 of the value there), else 1 - 2 / (1 + e^(2x)) on the special-function unit. Capped scores lie between -c and c, so
+// with c up to 55 the weights need no maximum at all: 2^(c log2 e) stays below 2^80, far inside the range of float32 and bfloat16,
+// and neither the search for a row's maximum nor any rescaling is left (CAP 1; larger caps keep the running maximum, CAP 2).
 // Keys past a row's length are masked; they are read (a page is loaded whole), which is safe because cache pools start as zeros
 // and only ever hold finite values. Every mbarrier wait is bounded (tcgen05.cuh).
 #include "tcgen05.cuh"
@@ -50,13 +52,13 @@ __device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
 }
 __device__ __forceinline__ float am_sigmoid(float x) { return 1.f / (1.f + __expf(-x)); }
 
-template <int MAPS, bool CAP>
+template <int MAPS, int CAP, int QB, int VB>
 __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid_constant__ CUtensorMap map_q,
                                                                     const __grid_constant__ CUtensorMap map_kv, const MapsPrompt a) {
     extern __shared__ unsigned char smem_raw[];
-    const int qb = (a.dim + 63) >> 6, vb = (a.vdim + 63) >> 6;          // 64-channel blocks of a key and of a value
-    const uint32_t k_bytes = MAPS * qb * AM_KV_BLOCK, stage_bytes = k_bytes + vb * AM_KV_BLOCK;
-    const uint32_t q_bytes = qb * AM_Q_BLOCK;                            // a group's queries
+    constexpr int qb = QB, vb = VB;                                      // 64-channel blocks of a key and of a value
+    constexpr uint32_t k_bytes = MAPS * qb * AM_KV_BLOCK, stage_bytes = k_bytes + vb * AM_KV_BLOCK;
+    constexpr uint32_t q_bytes = qb * AM_Q_BLOCK;                        // a group's queries
     const uint32_t base = (smem_addr(smem_raw) + 1023u) & ~1023u;
     const uint32_t q_s = base, kv_s = q_s + AM_GROUPS * q_bytes;
     const uint32_t bars = kv_s + AM_STAGES * stage_bytes;
@@ -160,7 +162,9 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
                         tc_fence_after();
                         const uint32_t s_t = tmem + g * 256 + (j & 1) * AM_BN;
                         const uint32_t k_src = kv_s + s * stage_bytes + (MAPS == 2 ? g * qb * AM_KV_BLOCK : 0);
-                        for (int kk = 0; kk < ksteps; ++kk) {
+#pragma unroll
+                        for (int kk = 0; kk < QB * 4; ++kk) {
+                            if (kk >= ksteps) break;
                             const uint32_t blk = kk >> 2, within = (kk & 3) * 2;
                             tc_mma(s_t, tc_smem_desc(q_s + g * q_bytes + blk * AM_Q_BLOCK) + within,
                                    tc_smem_desc(k_src + blk * AM_KV_BLOCK) + within, idesc_qk, kk != 0);
@@ -202,6 +206,11 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
         const uint32_t o_t = lane_t + 2 * AM_BN;
         const float scale_log2 = CAP ? 1.f : a.scale * AM_LOG2E;         // capped scores are already in log2 units
         const float to_x = CAP ? a.scale / a.cap : 0.f, from_x = CAP ? a.cap * AM_LOG2E : 0.f;
+        const float t2 = to_x * to_x;
+        // c log2(e) tanh(s t) = s (scale log2 e) (1 + s^2 (-t^2/3 + s^2 (2 t^4/15 - s^2 17 t^6/315))), t = scale / c
+        const uint64_t c7 = pack2(-17.f / 315.f * t2 * t2 * t2, -17.f / 315.f * t2 * t2 * t2), c5 = pack2(2.f / 15.f * t2 * t2, 2.f / 15.f * t2 * t2);
+        const uint64_t c3 = pack2(-1.f / 3.f * t2, -1.f / 3.f * t2), one = pack2(1.f, 1.f);
+        const uint64_t fx = pack2(a.scale * AM_LOG2E, a.scale * AM_LOG2E);
         float m_used = -INFINITY, l = 0.f;                               // in log2 units; the maximum may lag by AM_RESCALE
         bool ok = true;
         for (int j = 0; j < my_tiles && ok; ++j) {
@@ -221,14 +230,11 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
                     for (int i = 0; i < 32; ++i) top4[i & 3] = fmaxf(top4[i & 3], fabsf(__uint_as_float(sr[c][i])));
                 const float top = fmaxf(fmaxf(top4[0], top4[1]), fmaxf(top4[2], top4[3])) * to_x;
                 if (__all_sync(0xffffffffu, top <= 0.25f)) {
-                    const uint64_t tx = pack2(to_x, to_x), fx = pack2(from_x, from_x);
-                    const uint64_t c7 = pack2(-17.f / 315.f, -17.f / 315.f), c5 = pack2(2.f / 15.f, 2.f / 15.f);
-                    const uint64_t c3 = pack2(-1.f / 3.f, -1.f / 3.f), one = pack2(1.f, 1.f);
 #pragma unroll
                     for (int c = 0; c < 2; ++c)
 #pragma unroll
                         for (int i = 0; i < 32; i += 2) {
-                            const uint64_t x = mul2(pack2(__uint_as_float(sr[c][i]), __uint_as_float(sr[c][i + 1])), tx), y = mul2(x, x);
+                            const uint64_t x = pack2(__uint_as_float(sr[c][i]), __uint_as_float(sr[c][i + 1])), y = mul2(x, x);
                             const uint64_t w = fma2(y, fma2(y, fma2(y, c7, c5), c3), one);
                             float u, v;
                             unpack2(mul2(mul2(x, fx), w), u, v);
@@ -256,33 +262,35 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
                         if (!(key <= pos && key < hi && (a.window <= 0 || pos - key < a.window || key < a.keep))) sr[c][i] = 0xff800000u;
                     }
             }
-            float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY}; // four chains instead of one of 64
+            if constexpr (CAP != 1) {
+                float mx4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY}; // four chains instead of one of 64
 #pragma unroll
-            for (int c = 0; c < 2; ++c)
+                for (int c = 0; c < 2; ++c)
 #pragma unroll
-                for (int i = 0; i < 32; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(sr[c][i]));
-            const float mt = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2;
-            const bool grow = mt > m_used + AM_RESCALE || (m_used == -INFINITY && mt > -INFINITY);
-            if (__any_sync(0xffffffffu, grow)) {                         // rescale what is summed (whole warp: the TMEM ops are collective)
-                const float m_new = grow ? mt : m_used;
-                const float f = m_used == -INFINITY ? 0.f : at_ex2(m_used - m_new);
-                if (j > 0) {
-                    ok = mbar_wait(p_empty0 + 8 * (g * 2 + ((j - 1) & 1)), ((j - 1) >> 1) & 1, 7);   // O holds every tile before j
-                    tc_fence_after();
-                    if (ok) {
-                        for (int c = 0; c < (a.vdim + 31) >> 5; ++c) {
-                            uint32_t o[32];
-                            tc_ld32(o_t + c * 32, o);
+                    for (int i = 0; i < 32; ++i) mx4[i & 3] = fmaxf(mx4[i & 3], __uint_as_float(sr[c][i]));
+                const float mt = fmaxf(fmaxf(mx4[0], mx4[1]), fmaxf(mx4[2], mx4[3])) * scale_log2;
+                const bool grow = mt > m_used + AM_RESCALE || (m_used == -INFINITY && mt > -INFINITY);
+                if (__any_sync(0xffffffffu, grow)) {                         // rescale what is summed (whole warp: the TMEM ops are collective)
+                    const float m_new = grow ? mt : m_used;
+                    const float f = m_used == -INFINITY ? 0.f : at_ex2(m_used - m_new);
+                    if (j > 0) {
+                        ok = mbar_wait(p_empty0 + 8 * (g * 2 + ((j - 1) & 1)), ((j - 1) >> 1) & 1, 7);   // O holds every tile before j
+                        tc_fence_after();
+                        if (ok) {
+                            for (int c = 0; c < (a.vdim + 31) >> 5; ++c) {
+                                uint32_t o[32];
+                                tc_ld32(o_t + c * 32, o);
 #pragma unroll
-                            for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * f);
-                            tc_st32(o_t + c * 32, o);
+                                for (int i = 0; i < 32; ++i) o[i] = __float_as_uint(__uint_as_float(o[i]) * f);
+                                tc_st32(o_t + c * 32, o);
+                            }
                         }
                     }
+                    l *= f;
+                    m_used = m_new;
                 }
-                l *= f;
-                m_used = m_new;
             }
-            const float off = m_used == -INFINITY ? 0.f : -m_used;
+            const float off = CAP == 1 || m_used == -INFINITY ? 0.f : -m_used;
             const uint64_t scale2 = pack2(scale_log2, scale_log2), off2 = pack2(off, off);
             uint64_t sum2[4] = {0ull, 0ull, 0ull, 0ull};                 // four chains of packed sums
             uint32_t pk[32];                                             // 64 weights as bfloat16 pairs
@@ -291,7 +299,8 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
 #pragma unroll
                 for (int i = 0; i < 32; i += 2) {
                     float x, y;
-                    unpack2(fma2(pack2(__uint_as_float(sr[c][i]), __uint_as_float(sr[c][i + 1])), scale2, off2), x, y);
+                    if constexpr (CAP == 1) { x = __uint_as_float(sr[c][i]); y = __uint_as_float(sr[c][i + 1]); }
+                    else unpack2(fma2(pack2(__uint_as_float(sr[c][i]), __uint_as_float(sr[c][i + 1])), scale2, off2), x, y);
                     x = at_ex2(x);
                     y = at_ex2(y);
                     sum2[(i >> 1) & 3] = add2(sum2[(i >> 1) & 3], pack2(x, y));
@@ -455,8 +464,12 @@ extern "C" int hb_attention_maps_prefill(void* out, const void* q, const void* k
     const size_t smem = AM_GROUPS * (size_t)qb * AM_Q_BLOCK + AM_STAGES * (size_t)(maps * qb + vb) * AM_KV_BLOCK + 1024 + 256;
     const MapsPrompt p{(bf16*)out, block_table, row_slot, query_start, kv_len, (const bf16*)gate, gate_ld, table_stride, row0, rows,
                        heads, kv_heads, dim, vdim, pages, page_size, window, window > 0 ? keep : 0, tile_q, scale, cap, lam, factor, eps};
-    auto kernel = maps == 2 ? (cap > 0.f ? maps_prompt_kernel<2, true> : maps_prompt_kernel<2, false>)
-                            : (cap > 0.f ? maps_prompt_kernel<1, true> : maps_prompt_kernel<1, false>);
+    void (*kernel)(const CUtensorMap, const CUtensorMap, const MapsPrompt) = nullptr;
+    const int kind = cap <= 0.f ? 0 : cap <= 55.f ? 1 : 2;
+#define HB_PICK(M, C) if (maps == M && kind == C) kernel = qb == 1 ? (vb == 1 ? maps_prompt_kernel<M, C, 1, 1> : maps_prompt_kernel<M, C, 1, 2>) \
+                                                                   : (vb == 1 ? maps_prompt_kernel<M, C, 2, 1> : maps_prompt_kernel<M, C, 2, 2>)
+    HB_PICK(1, 0); HB_PICK(1, 1); HB_PICK(1, 2); HB_PICK(2, 0); HB_PICK(2, 1); HB_PICK(2, 2);
+#undef HB_PICK
     HB_CUDA(cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)smem));
     kernel<<<dim3(heads, q_tiles), AM_THREADS, smem, (cudaStream_t)stream>>>(map_q, map_kv, p);
     HB_LAUNCH_CHECK("attention_maps_prefill");

@@ -16,7 +16,6 @@
 #define SS_Q 64                          // tokens a chunk
 #define SS_T 64                          // rows and columns of an output tile
 #define SS_K 32                          // depth of a staged slice
-#define SS_PAD 4
 #define SS_THREADS 128                   // a thread: 8 rows x 4 columns of a tile
 
 struct Chunk { int row, t0, n, first_tile; };              // the batch row, first token, tokens, the row's first tile
@@ -32,12 +31,18 @@ __device__ __forceinline__ Chunk find_chunk(const int32_t* __restrict__ query_st
     return {-1, 0, 0, 0};
 }
 
-// A slice of both operands in shared memory, a[k][row], b[k][column]: acc += a^T b.
-__device__ __forceinline__ void tile_step(float (&acc)[8][4], const float (*a)[SS_T + SS_PAD], const float (*b)[SS_T + SS_PAD], int depth) {
+// A slice of an operand in shared memory: element (k, i) in the group of four floats at(k, i / 4). The groups of a row of k are
+// permuted by k / 4, so that stores of four k's of one i by eight neighbouring lanes, and of four i's by four, hit different banks.
+__device__ __forceinline__ int group_at(int k, int g) { return k * (SS_T / 4) + (g ^ ((k >> 2) & 7)); }
+
+// acc += a^T b over a slice.
+__device__ __forceinline__ void tile_step(float (&acc)[8][4], const float* a, const float* b, int depth) {
     const int ty = threadIdx.x >> 4, tx = threadIdx.x & 15;
+    const float4* a4 = (const float4*)a;
+    const float4* b4 = (const float4*)b;
 #pragma unroll 8
     for (int k = 0; k < depth; ++k) {
-        const float4 r0 = *(const float4*)&a[k][ty * 8], r1 = *(const float4*)&a[k][ty * 8 + 4], c = *(const float4*)&b[k][tx * 4];
+        const float4 r0 = a4[group_at(k, ty * 2)], r1 = a4[group_at(k, ty * 2 + 1)], c = b4[group_at(k, tx)];
         const float r[8] = {r0.x, r0.y, r0.z, r0.w, r1.x, r1.y, r1.z, r1.w};
 #pragma unroll
         for (int i = 0; i < 8; ++i) {
@@ -48,23 +53,25 @@ __device__ __forceinline__ void tile_step(float (&acc)[8][4], const float (*a)[S
 }
 
 // Slices travel through registers (the next one is on its way while the current one is multiplied), 16 bytes a load: four quads a
-// thread and operand. `along`: the operand's memory runs along k (element (row i, k) at p[i * stride + k]); a thread then holds quads
-// of one row, and the stores to [k][i] go to neighbouring banks. Else it runs along the tile's rows (element (k, i) at p[k * stride + i]).
+// thread and operand. `along`: the operand's memory runs along k (element (row i, k) at p[i * stride + k]); eight neighbouring lanes
+// load 128 bytes of one row. `across`: it runs along the tile's rows (element (k, i) at p[k * stride + i]).
 struct Quads { float4 v[4]; };
 __device__ __forceinline__ float4 load_quad(const float* p, int left, bool vec) {        // zeros from `left` on
     if (vec && left >= 4) return *(const float4*)p;
     return make_float4(left > 0 ? p[0] : 0.f, left > 1 ? p[1] : 0.f, left > 2 ? p[2] : 0.f, left > 3 ? p[3] : 0.f);
 }
 __device__ __forceinline__ void fetch_along(Quads& q, const float* p, size_t stride, int rows, int depth, bool vec) {
-    const int i = threadIdx.x & 63, k = (threadIdx.x >> 6) * 4;
+    const int i = threadIdx.x >> 3, k = (threadIdx.x & 7) * 4;
 #pragma unroll
-    for (int r = 0; r < 4; ++r) q.v[r] = load_quad(p + i * stride + k + 8 * r, i < rows ? depth - k - 8 * r : 0, vec);
+    for (int r = 0; r < 4; ++r) q.v[r] = load_quad(p + (i + 16 * r) * stride + k, i + 16 * r < rows ? depth - k : 0, vec);
 }
-__device__ __forceinline__ void store_along(float (*a)[SS_T + SS_PAD], const Quads& q) {
-    const int i = threadIdx.x & 63, k = (threadIdx.x >> 6) * 4;
+__device__ __forceinline__ void store_along(float* a, const Quads& q) {
+    const int k = (threadIdx.x & 7) * 4;
 #pragma unroll
     for (int r = 0; r < 4; ++r) {
-        a[k + 8 * r][i] = q.v[r].x; a[k + 8 * r + 1][i] = q.v[r].y; a[k + 8 * r + 2][i] = q.v[r].z; a[k + 8 * r + 3][i] = q.v[r].w;
+        const int i = (threadIdx.x >> 3) + 16 * r, g = i >> 2, e = i & 3;      // (k .. k + 3 share their permutation)
+        a[group_at(k, g) * 4 + e] = q.v[r].x; a[group_at(k + 1, g) * 4 + e] = q.v[r].y;
+        a[group_at(k + 2, g) * 4 + e] = q.v[r].z; a[group_at(k + 3, g) * 4 + e] = q.v[r].w;
     }
 }
 __device__ __forceinline__ void fetch_across(Quads& q, const float* p, size_t stride, int rows, int depth, bool vec) {
@@ -72,10 +79,10 @@ __device__ __forceinline__ void fetch_across(Quads& q, const float* p, size_t st
 #pragma unroll
     for (int r = 0; r < 4; ++r) q.v[r] = load_quad(p + (k + 8 * r) * stride + i, k + 8 * r < depth ? rows - i : 0, vec);
 }
-__device__ __forceinline__ void store_across(float (*a)[SS_T + SS_PAD], const Quads& q) {
-    const int i = (threadIdx.x & 15) * 4, k = threadIdx.x >> 4;
+__device__ __forceinline__ void store_across(float* a, const Quads& q) {
+    const int k = threadIdx.x >> 4;
 #pragma unroll
-    for (int r = 0; r < 4; ++r) *(float4*)&a[k + 8 * r][i] = q.v[r];
+    for (int r = 0; r < 4; ++r) ((float4*)a)[group_at(k + 8 * r, threadIdx.x & 15)] = q.v[r];
 }
 __device__ __forceinline__ void scale_quad(float4& v, float f) { v.x *= f; v.y *= f; v.z *= f; v.w *= f; }
 
@@ -101,9 +108,9 @@ __device__ __forceinline__ void log_decays(float* hi, float* lo, float* steps, c
 }
 
 // ---- products[tile][group][i][j] = C_i . B_j, [64][64] each. grid (tiles, groups)
-__global__ void __launch_bounds__(SS_THREADS) ss_products_kernel(float* __restrict__ products, const float* __restrict__ cb,
+__global__ void __launch_bounds__(SS_THREADS, 4) ss_products_kernel(float* __restrict__ products, const float* __restrict__ cb,
                                                                  const int32_t* __restrict__ query_start, int row0, int rows, int groups, int n) {
-    __shared__ __align__(16) float a[SS_K][SS_T + SS_PAD], b[SS_K][SS_T + SS_PAD];
+    __shared__ __align__(16) float a[SS_K * SS_T], b[SS_K * SS_T];
     const Chunk c = find_chunk(query_start, row0, rows, blockIdx.x);
     if (c.row < 0) return;
     const int g = blockIdx.y;
@@ -133,11 +140,11 @@ __global__ void __launch_bounds__(SS_THREADS) ss_products_kernel(float* __restri
 
 // ---- own[tile][head][p][n] = sum_j exp(L_last - L_j) dt_j x_j[p] B_j[n]; last[tile][head] = exp(L_last). grid (tiles, heads, tiles of
 // p times tiles of n)
-__global__ void __launch_bounds__(SS_THREADS) ss_own_kernel(float* __restrict__ own, float* __restrict__ last, const float* __restrict__ cb,
+__global__ void __launch_bounds__(SS_THREADS, 4) ss_own_kernel(float* __restrict__ own, float* __restrict__ last, const float* __restrict__ cb,
                                                             const float* __restrict__ x, const float* __restrict__ dt,
                                                             const float* __restrict__ rate_log, const int32_t* __restrict__ query_start,
                                                             int row0, int rows, int heads, int groups, int n, int vdim, int n_tiles) {
-    __shared__ __align__(16) float a[SS_K][SS_T + SS_PAD], b[SS_K][SS_T + SS_PAD];
+    __shared__ __align__(16) float a[SS_K * SS_T], b[SS_K * SS_T];
     __shared__ float hi[SS_Q], lo[SS_Q], steps[SS_Q], w[SS_Q];
     const Chunk c = find_chunk(query_start, row0, rows, blockIdx.x);
     if (c.row < 0) return;
@@ -223,13 +230,13 @@ __global__ void ss_walk_kernel(float* __restrict__ own, const float* __restrict_
 }
 
 // ---- y_i[p] of a chunk: the products' part over its own tokens, the state's part over n, the skip. grid (tiles, heads, tiles of p)
-__global__ void __launch_bounds__(SS_THREADS) ss_out_kernel(float* __restrict__ y, const float* __restrict__ products,
+__global__ void __launch_bounds__(SS_THREADS, 4) ss_out_kernel(float* __restrict__ y, const float* __restrict__ products,
                                                             const float* __restrict__ before, const float* __restrict__ cb,
                                                             const float* __restrict__ x, const float* __restrict__ dt,
                                                             const float* __restrict__ rate_log, const float* __restrict__ skip,
                                                             const int32_t* __restrict__ query_start, int row0, int rows, int heads,
                                                             int groups, int n, int vdim) {
-    __shared__ __align__(16) float a[SS_K][SS_T + SS_PAD], b[SS_K][SS_T + SS_PAD];
+    __shared__ __align__(16) float a[SS_K * SS_T], b[SS_K * SS_T];
     __shared__ float hi[SS_Q], lo[SS_Q], steps[SS_Q], w[SS_Q];
     const Chunk c = find_chunk(query_start, row0, rows, blockIdx.x);
     if (c.row < 0) return;
@@ -259,21 +266,20 @@ __global__ void __launch_bounds__(SS_THREADS) ss_out_kernel(float* __restrict__ 
         }
     };
     fetch(0);
-    const int row = threadIdx.x & 63, kq = (threadIdx.x >> 6) * 4;
     for (int s = 0; s < slices; ++s) {
         if (s < own_slices) {                                       // weight of token j in row i: C_i . B_j exp(L_i - L_j) dt_j, j <= i
-            const float hr = hi[row], lr = lo[row];
+            const int j = s * SS_K + ((int)threadIdx.x & 7) * 4;
 #pragma unroll
             for (int r = 0; r < 4; ++r) {
-                const int j = s * SS_K + kq + 8 * r;
+                const int row = ((int)threadIdx.x >> 3) + 16 * r;
+                const float hr = hi[row], lr = lo[row];
                 auto weight = [&](int jj, float v) -> float { return jj <= row && jj < c.n ? v * expf((hr - hi[jj]) + (lr - lo[jj])) * steps[jj] : 0.f; };
                 qa.v[r].x = weight(j, qa.v[r].x); qa.v[r].y = weight(j + 1, qa.v[r].y);
                 qa.v[r].z = weight(j + 2, qa.v[r].z); qa.v[r].w = weight(j + 3, qa.v[r].w);
             }
         } else {
-            const float f = w[row];
 #pragma unroll
-            for (int r = 0; r < 4; ++r) scale_quad(qa.v[r], f);
+            for (int r = 0; r < 4; ++r) scale_quad(qa.v[r], w[((int)threadIdx.x >> 3) + 16 * r]);
         }
         store_along(a, qa);
         if (s < own_slices) store_across(b, qb); else store_along(b, qb);
