@@ -596,7 +596,7 @@ class TimedKernels:
     def __getattr__(self, name):
         import torch
         value = getattr(self._k, name)
-        if not callable(value) or name.startswith("_") or name in ("attention_capture_plan", "can_link", "flush", "status"):
+        if not callable(value) or name.startswith("_") or name in ("attention_capture_plan", "branch", "can_link", "flush", "status"):
             return value
 
         def timed(*a, **kw):

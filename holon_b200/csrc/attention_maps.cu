@@ -21,7 +21,7 @@
 __device__ __forceinline__ float mp_sigmoid(float x) { return 1.f / (1.f + expf(-x)); }
 
 // ---------------------------------------------------------------- from the first product to q rows and cache rows
-// One warp per (token, slot): heads * maps queries, kv_heads * maps keys, kv_heads values. norm 1: x / rms(x) * weight, then
+// One warp per token and SL slots: heads * maps queries, kv_heads * maps keys, kv_heads values. norm 1: x / rms(x) * weight, then
 // the rotation; norm 2: the rotation, then x / rms(x); 0: no norm. The first rot_dims channels turn in half-split pairs;
 // `table` holds, per position, the rot_dims / 2 cosines and then the sines. One rounding, at the end. PAIR: a lane owns runs of
 // two neighbouring channels (dim, vdim, the rows and the cache even), else every 32nd channel.
@@ -37,7 +37,7 @@ template <> struct Two<bf16> {
     static __device__ __forceinline__ void store(bf16* p, float a, float b) { *(__nv_bfloat162*)p = __floats2bfloat162_rn(a, b); }
 };
 
-template <typename T, bool PAIR, int PL>
+template <typename T, bool PAIR, int PL, int SL>
 __global__ void maps_prepare_kernel(T* __restrict__ q_out, T* __restrict__ kv, const T* __restrict__ first, long ld,
                                     const float* __restrict__ q_weight, const float* __restrict__ k_weight, float eps, int norm,
                                     const int32_t* __restrict__ positions, const float* __restrict__ table, int rot_dims,
@@ -47,86 +47,104 @@ __global__ void maps_prepare_kernel(T* __restrict__ q_out, T* __restrict__ kv, c
     const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
     const int nq = heads * maps, nk = kv_heads * maps, slots = nq + nk + kv_heads;
     const long t = blockIdx.x;
-    const int slot = (int)blockIdx.y * MP_WARPS + warp;
-    if (slot >= slots) return;
-    const int rowlen = maps * dim + vdim;
+    const int slot0 = ((int)blockIdx.y * MP_WARPS + warp) * SL;
+    if (slot0 >= slots) return;
+    const int rowlen = maps * dim + vdim, last = min(slots, slot0 + SL);
     const long w = write_index ? write_index[t] : -1;
     const bool stored = w >= 0 && w < (long)pages * page_size;
     const long page = stored ? w / page_size : 0, off = stored ? w - page * page_size : 0;
     const T* row = first + t * ld;
-    if (slot >= nq + nk) {                                            // a value head: copied
-        if (!stored) return;
-        const int c = slot - nq - nk;
-        const T* src = row + (long)(nq + nk) * dim + (long)c * vdim;
-        T* dst = kv + ((page * kv_heads + c) * page_size + off) * rowlen + maps * dim;
-        if (PAIR) {
-            for (int d = 2 * lane; d < vdim; d += 64) { const float2 v = Two<T>::load(src + d); Two<T>::store(dst + d, v.x, v.y); }
-        } else {
-            for (int d = lane; d < vdim; d += 32) dst[d] = src[d];
-        }
-        return;
-    }
-    const bool is_q = slot < nq;
-    const T* src = row + (long)slot * dim;                            // (queries, then keys, map by map: one numbering)
-    T* dst = nullptr;
-    if (is_q) dst = q_out + (t * nq + slot) * dim;
-    else if (stored) {
-        const int c = (slot - nq) / maps, m = (slot - nq) - c * maps;
-        dst = kv + ((page * kv_heads + c) * page_size + off) * rowlen + m * dim;
-    }
-    if (!dst) return;
-    const float* weight = is_q ? q_weight : k_weight;
     float* ys = mp_smem + (size_t)warp * ((dim + 3) & ~3);
-    float x[PL];
     auto at = [&](int i) -> int { return PAIR ? 2 * lane + 64 * (i >> 1) + (i & 1) : lane + 32 * i; };
-    float ss = 0.f;
+    float x[SL][PL];                                                  // every slot's numbers are asked for before any is worked on
 #pragma unroll
-    for (int i = 0; i < PL; i += PAIR ? 2 : 1) {
-        const int d = at(i);
-        if (PAIR) {
-            const float2 v = d < dim ? Two<T>::load(src + d) : make_float2(0.f, 0.f);
-            x[i] = v.x; x[i + 1] = v.y;
-            ss += v.x * v.x + v.y * v.y;
-        } else {
-            x[i] = d < dim ? to_f32(src[d]) : 0.f;
-            ss += x[i] * x[i];
+    for (int s = 0; s < SL; ++s) {
+        const T* src = row + (long)(slot0 + s) * dim;                 // (queries, then keys, map by map: one numbering)
+        const bool mine = slot0 + s < nq + nk;
+#pragma unroll
+        for (int i = 0; i < PL; i += PAIR ? 2 : 1) {
+            const int d = at(i);
+            if (PAIR) {
+                const float2 v = mine && d < dim ? Two<T>::load(src + d) : make_float2(0.f, 0.f);
+                x[s][i] = v.x; x[s][i + 1] = v.y;
+            } else {
+                x[s][i] = mine && d < dim ? to_f32(src[d]) : 0.f;
+            }
         }
     }
-    if (norm == 1) {
-        const float r = rsqrtf(warp_sum(ss) / (float)dim + eps);
-#pragma unroll
-        for (int i = 0; i < PL; ++i) { const int d = at(i); if (d < dim) x[i] *= r * weight[d]; }
-    }
+    const int half = rot_dims >> 1;
+    float co[PL], si[PL];                                             // the token's angles, for all its slots
     if (rot_dims) {
         int pos = positions[t];
         pos = pos < 0 ? 0 : (pos >= table_rows ? table_rows - 1 : pos);
         const float* cs = table + (size_t)pos * rot_dims;
-        const int half = rot_dims >> 1;
-#pragma unroll
-        for (int i = 0; i < PL; ++i) { const int d = at(i); if (d < rot_dims) ys[d] = x[i]; }
-        __syncwarp();
-        ss = 0.f;
 #pragma unroll
         for (int i = 0; i < PL; ++i) {
-            const int d = at(i);
-            if (d < rot_dims) {
-                const bool lead = d < half;                           // u of the pair (u, v), or v
-                const int c = lead ? d : d - half;
-                const float o = ys[lead ? d + half : c], co = cs[c], si = cs[half + c];
-                x[i] = lead ? x[i] * co - o * si : x[i] * co + o * si;
-            }
-            if (d < dim) ss += x[i] * x[i];
+            const int d = at(i), c = d < half ? d : d - half;
+            co[i] = d < rot_dims ? cs[c] : 1.f;
+            si[i] = d < rot_dims ? cs[half + c] : 0.f;
         }
     }
-    if (norm == 2) {
-        const float r = rsqrtf(warp_sum(ss) / (float)dim + eps);
 #pragma unroll
-        for (int i = 0; i < PL; ++i) x[i] *= r;
-    }
+    for (int s = 0; s < SL; ++s) {
+        const int slot = slot0 + s;
+        if (slot >= last) break;
+        if (slot >= nq + nk) {                                        // a value head: copied
+            if (!stored) continue;
+            const int c = slot - nq - nk;
+            const T* src = row + (long)(nq + nk) * dim + (long)c * vdim;
+            T* dst = kv + ((page * kv_heads + c) * page_size + off) * rowlen + maps * dim;
+            if (PAIR) {
+                for (int d = 2 * lane; d < vdim; d += 64) { const float2 v = Two<T>::load(src + d); Two<T>::store(dst + d, v.x, v.y); }
+            } else {
+                for (int d = lane; d < vdim; d += 32) dst[d] = src[d];
+            }
+            continue;
+        }
+        const bool is_q = slot < nq;
+        T* dst = nullptr;
+        if (is_q) dst = q_out + (t * nq + slot) * dim;
+        else if (stored) {
+            const int c = (slot - nq) / maps, m = (slot - nq) - c * maps;
+            dst = kv + ((page * kv_heads + c) * page_size + off) * rowlen + m * dim;
+        }
+        if (!dst) continue;
+        float ss = 0.f;
+        if (norm == 1) {
+            const float* weight = is_q ? q_weight : k_weight;
 #pragma unroll
-    for (int i = 0; i < PL; i += PAIR ? 2 : 1) {
-        const int d = at(i);
-        if (d < dim) { if (PAIR) Two<T>::store(dst + d, x[i], x[i + 1]); else dst[d] = from_f32<T>(x[i]); }
+            for (int i = 0; i < PL; ++i) ss += x[s][i] * x[s][i];
+            const float r = rsqrtf(warp_sum(ss) / (float)dim + eps);
+#pragma unroll
+            for (int i = 0; i < PL; ++i) { const int d = at(i); if (d < dim) x[s][i] *= r * weight[d]; }
+        }
+        if (rot_dims) {
+            __syncwarp();                                             // (the slot before has read its numbers)
+#pragma unroll
+            for (int i = 0; i < PL; ++i) { const int d = at(i); if (d < rot_dims) ys[d] = x[s][i]; }
+            __syncwarp();
+#pragma unroll
+            for (int i = 0; i < PL; ++i) {
+                const int d = at(i);
+                if (d < rot_dims) {                                   // u of the pair (u, v), or v
+                    const float o = ys[d < half ? d + half : d - half];
+                    x[s][i] = d < half ? x[s][i] * co[i] - o * si[i] : x[s][i] * co[i] + o * si[i];
+                }
+            }
+        }
+        if (norm == 2) {
+            ss = 0.f;
+#pragma unroll
+            for (int i = 0; i < PL; ++i) ss += x[s][i] * x[s][i];
+            const float r = rsqrtf(warp_sum(ss) / (float)dim + eps);
+#pragma unroll
+            for (int i = 0; i < PL; ++i) x[s][i] *= r;
+        }
+#pragma unroll
+        for (int i = 0; i < PL; i += PAIR ? 2 : 1) {
+            const int d = at(i);
+            if (d < dim) { if (PAIR) Two<T>::store(dst + d, x[s][i], x[s][i + 1]); else dst[d] = from_f32<T>(x[s][i]); }
+        }
     }
 }
 
@@ -142,15 +160,17 @@ extern "C" int hb_qkv_maps_prepare(void* q_out, void* kv, const void* first, int
     if (maps < 1 || kv_heads < 1 || heads % kv_heads) HB_REFUSE("qkv_maps_prepare: %d heads, %d kv heads, %d maps", heads, kv_heads, maps);
     const long slots = (long)heads * maps + (long)kv_heads * maps + kv_heads;
     if (slots > 65535L * MP_WARPS) HB_REFUSE("qkv_maps_prepare: %ld heads a token", slots);
-    const dim3 grid(tokens, (unsigned)((slots + MP_WARPS - 1) / MP_WARPS));
+    const int sl = dim <= 128 && tokens >= 64 ? 4 : 1;                // slots a warp takes in turn
+    const dim3 grid(tokens, (unsigned)((slots + MP_WARPS * sl - 1) / (MP_WARPS * sl)));
     const size_t smem = (size_t)MP_WARPS * ((dim + 3) & ~3) * sizeof(float);
     cudaStream_t s = (cudaStream_t)stream;
     const size_t two = dtype == HB_F32 ? 8 : 4;
     const bool pair = dim % 2 == 0 && vdim % 2 == 0 && ld % 2 == 0 && (((uintptr_t)q_out | (uintptr_t)kv | (uintptr_t)first) % two) == 0;
 #define HB_ARGS(T) (T*)q_out, (T*)kv, (const T*)first, ld, q_weight, k_weight, eps, norm, positions, table, rot_dims, table_rows, \
     write_index, pages, page_size, heads, kv_heads, maps, dim, vdim
-#define HB_RUN(T, P) do { if (dim <= 128) maps_prepare_kernel<T, P, 4><<<grid, MP_WARPS * 32, smem, s>>>(HB_ARGS(T)); \
-                          else maps_prepare_kernel<T, P, MP_PER_LANE><<<grid, MP_WARPS * 32, smem, s>>>(HB_ARGS(T)); } while (0)
+#define HB_RUN(T, P) do { if (sl == 4) maps_prepare_kernel<T, P, 4, 4><<<grid, MP_WARPS * 32, smem, s>>>(HB_ARGS(T)); \
+                          else if (dim <= 128) maps_prepare_kernel<T, P, 4, 1><<<grid, MP_WARPS * 32, smem, s>>>(HB_ARGS(T)); \
+                          else maps_prepare_kernel<T, P, MP_PER_LANE, 1><<<grid, MP_WARPS * 32, smem, s>>>(HB_ARGS(T)); } while (0)
     if (dtype == HB_F32) { if (pair) HB_RUN(float, true); else HB_RUN(float, false); }
     else if (dtype == HB_BF16) { if (pair) HB_RUN(bf16, true); else HB_RUN(bf16, false); }
     else HB_REFUSE("qkv_maps_prepare: dtype %d", dtype);

@@ -318,15 +318,25 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
             __syncwarp();
             if (lane == 0) mbar_arrive(p_full0 + 8 * gb);
         }
-        if (ok) ok = mbar_wait(o_full0 + 8 * g, 0, 9);
-        tc_fence_after();
-        const float inv = ok && my_tiles > 0 && l > 0.f ? 1.f / l : 0.f;
+        constexpr int CHUNKS = VB * 2, MINE = MAPS == 1 ? CHUNKS : VB;   // chunks of 32 channels; this thread's (two maps: g, g + 2)
         const int chunks = (a.vdim + 31) >> 5;
         const size_t token = (size_t)(t0 + (MAPS == 1 ? g * AM_BM : 0) + (r < qn ? r : 0));
         bf16* o_row = a.out + (token * a.heads + h) * a.vdim;
         const bf16* g_row = a.gate ? a.gate + token * a.gate_ld + (size_t)h * a.vdim : nullptr;
         const bool g_vec = (((uintptr_t)a.gate | (uintptr_t)(a.gate_ld * 2)) & 15) == 0;      // (vdim is a multiple of 16)
-        auto store = [&](const float (&v)[32], int c) {                  // a chunk of 32 channels of this thread's row, gated
+        uint4 gq[MINE][4];                                               // the row's gates, asked for ahead of the last products
+#pragma unroll
+        for (int k = 0; k < MINE; ++k)
+#pragma unroll
+            for (int i = 0; i < 4; ++i) {
+                const int d = (MAPS == 1 ? k : g + 2 * k) * 32 + i * 8;
+                gq[k][i] = make_uint4(0u, 0u, 0u, 0u);
+                if (g_row && g_vec && r < qn && d < a.vdim) gq[k][i] = *(const uint4*)(g_row + d);
+            }
+        if (ok) ok = mbar_wait(o_full0 + 8 * g, 0, 9);
+        tc_fence_after();
+        const float inv = ok && my_tiles > 0 && l > 0.f ? 1.f / l : 0.f;
+        auto store = [&](const float (&v)[32], int c, const uint4 (&gz)[4]) {                  // a chunk of 32 channels of this thread's row, gated
             const int live = min(32, a.vdim - c * 32);                   // 32 or 16
 #pragma unroll
             for (int i = 0; i < 32; i += 8) {
@@ -337,7 +347,7 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
                 if (g_row) {
                     float z[8];
                     if (g_vec) {
-                        const uint4 w = *(const uint4*)(g_row + c * 32 + i);
+                        const uint4 w = gz[i / 8];
                         const uint32_t u[4] = {w.x, w.y, w.z, w.w};
 #pragma unroll
                         for (int e = 0; e < 4; ++e) { z[2 * e] = __uint_as_float(u[e] << 16); z[2 * e + 1] = __uint_as_float(u[e] & 0xffff0000u); }
@@ -357,13 +367,15 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
         };
         if (MAPS == 1) {
             if (ok && qn > 0) {                                          // (the tensor-memory loads are warp-collective: no lane skips them)
-                for (int c = 0; c < chunks; ++c) {
+#pragma unroll
+                for (int c = 0; c < CHUNKS; ++c) {
+                    if (c >= chunks) break;
                     uint32_t o[32];
                     tc_ld32(o_t + c * 32, o);
                     float v[32];
 #pragma unroll
                     for (int i = 0; i < 32; ++i) v[i] = inv > 0.f ? __uint_as_float(o[i]) * inv : 0.f;
-                    if (r < qn) store(v, c);
+                    if (r < qn) store(v, c, gq[c < MINE ? c : 0]);
                 }
             }
         } else {
@@ -373,9 +385,9 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
             tc_fence_after();
             const float i1 = s_inv[0][r], i2 = s_inv[1][r] * a.lam;
             const uint32_t row_t = tmem + ((uint32_t)(q * 32) << 16) + 2 * AM_BN;
-            float v[2][32], ss = 0.f;                                    // channels of chunks g, g + 2
+            float v[VB][32], ss = 0.f;                                   // channels of chunks g, g + 2
 #pragma unroll
-            for (int k = 0; k < 2; ++k) {
+            for (int k = 0; k < VB; ++k) {
                 const int c = g + 2 * k;
 #pragma unroll
                 for (int i = 0; i < 32; ++i) v[k][i] = 0.f;
@@ -397,12 +409,12 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
             asm volatile("bar.sync 1, 256;\n" ::: "memory");
             const float f = rsqrtf((s_ss[0][r] + s_ss[1][r]) / (float)a.vdim + a.eps) * a.factor;
 #pragma unroll
-            for (int k = 0; k < 2; ++k) {
+            for (int k = 0; k < VB; ++k) {
                 const int c = g + 2 * k;
                 if (c < chunks && r < qn) {
 #pragma unroll
                     for (int i = 0; i < 32; ++i) v[k][i] *= f;
-                    store(v[k], c);
+                    store(v[k], c, gq[k]);
                 }
             }
         }

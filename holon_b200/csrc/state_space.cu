@@ -150,6 +150,13 @@ __global__ void __launch_bounds__(SS_THREADS, 4) ss_own_kernel(float* __restrict
     if (c.row < 0) return;
     const int h = blockIdx.y, g = h / (heads / groups);
     const int p0 = ((int)blockIdx.z / n_tiles) * SS_T, n0 = ((int)blockIdx.z % n_tiles) * SS_T;
+    Quads qa, qb;
+    const size_t xs = (size_t)heads * vdim, bs = (size_t)2 * groups * n;
+    const float* xp = x + ((size_t)c.t0 * heads + h) * vdim + p0;
+    const float* bp = cb + (((size_t)c.t0 * 2 + 1) * groups + g) * n + n0;
+    const bool vx = (vdim & 3) == 0, vb = (n & 3) == 0;
+    fetch_across(qa, xp, xs, vdim - p0, c.n, vx);                   // (on its way while the decays are added up)
+    fetch_across(qb, bp, bs, n - n0, c.n, vb);
     log_decays(hi, lo, steps, dt, c, heads, h, expf(rate_log[h]));
     __syncthreads();
     if (threadIdx.x < SS_Q) {
@@ -159,13 +166,6 @@ __global__ void __launch_bounds__(SS_THREADS, 4) ss_own_kernel(float* __restrict
     }
     __syncthreads();
     float acc[8][4] = {};
-    Quads qa, qb;
-    const size_t xs = (size_t)heads * vdim, bs = (size_t)2 * groups * n;
-    const float* xp = x + ((size_t)c.t0 * heads + h) * vdim + p0;
-    const float* bp = cb + (((size_t)c.t0 * 2 + 1) * groups + g) * n + n0;
-    const bool vx = (vdim & 3) == 0, vb = (n & 3) == 0;
-    fetch_across(qa, xp, xs, vdim - p0, c.n, vx);
-    fetch_across(qb, bp, bs, n - n0, c.n, vb);
     for (int k0 = 0; k0 < c.n; k0 += SS_K) {
 #pragma unroll
         for (int r = 0; r < 4; ++r) scale_quad(qa.v[r], w[min(k0 + ((int)threadIdx.x >> 4) + 8 * r, SS_Q - 1)]);
@@ -213,13 +213,13 @@ __global__ void ss_walk_kernel(float* __restrict__ own, const float* __restrict_
         else s = fmaf(d, s, v);
     };
     int i = 0;
-    for (; i + 4 <= tiles; i += 4, p += 4 * stride, f += 4 * (size_t)heads) {        // (four chunks' loads fly together)
-        const E v0 = p[0], v1 = p[stride], v2 = p[2 * stride], v3 = p[3 * stride];
-        const float d0 = f[0], d1 = f[heads], d2 = f[2 * (size_t)heads], d3 = f[3 * (size_t)heads];
-        p[0] = s; step(d0, v0);
-        p[stride] = s; step(d1, v1);
-        p[2 * stride] = s; step(d2, v2);
-        p[3 * stride] = s; step(d3, v3);
+    for (; i + 8 <= tiles; i += 8, p += 8 * stride, f += 8 * (size_t)heads) {        // (eight chunks' loads fly together)
+        E v[8];
+        float d[8];
+#pragma unroll
+        for (int k = 0; k < 8; ++k) { v[k] = p[k * stride]; d[k] = f[k * (size_t)heads]; }
+#pragma unroll
+        for (int k = 0; k < 8; ++k) { p[k * stride] = s; step(d[k], v[k]); }
     }
     for (; i < tiles; ++i, p += stride, f += heads) {
         const E v = p[0];
@@ -241,11 +241,6 @@ __global__ void __launch_bounds__(SS_THREADS, 4) ss_out_kernel(float* __restrict
     const Chunk c = find_chunk(query_start, row0, rows, blockIdx.x);
     if (c.row < 0) return;
     const int h = blockIdx.y, g = h / (heads / groups), p0 = (int)blockIdx.z * SS_T;
-    log_decays(hi, lo, steps, dt, c, heads, h, expf(rate_log[h]));
-    __syncthreads();
-    if (threadIdx.x < SS_Q) w[threadIdx.x] = expf(hi[threadIdx.x] + lo[threadIdx.x]);
-    __syncthreads();
-    float acc[8][4] = {};
     const float* cbp = products + ((size_t)blockIdx.x * groups + g) * SS_Q * SS_Q;
     const float* xp = x + ((size_t)c.t0 * heads + h) * vdim + p0;
     const float* cp = cb + ((size_t)c.t0 * 2 * groups + g) * n;
@@ -265,7 +260,12 @@ __global__ void __launch_bounds__(SS_THREADS, 4) ss_out_kernel(float* __restrict
             fetch_along(qb, sp + k0, n, vdim - p0, n - k0, vn);
         }
     };
-    fetch(0);
+    fetch(0);                                                       // (on its way while the decays are added up)
+    log_decays(hi, lo, steps, dt, c, heads, h, expf(rate_log[h]));
+    __syncthreads();
+    if (threadIdx.x < SS_Q) w[threadIdx.x] = expf(hi[threadIdx.x] + lo[threadIdx.x]);
+    __syncthreads();
+    float acc[8][4] = {};
     for (int s = 0; s < slices; ++s) {
         if (s < own_slices) {                                       // weight of token j in row i: C_i . B_j exp(L_i - L_j) dt_j, j <= i
             const int j = s * SS_K + ((int)threadIdx.x & 7) * 4;

@@ -58,6 +58,26 @@ class Extension:
         self.kernels._call_in(self.lib, self._fn, fn, *args)
 
 
+class Branch:
+    """A second stream beside the current one (`CudaKernels.branch`): what is enqueued inside `with branch:` starts behind all that the
+    current stream holds and runs beside what is enqueued on it until `join()`, from where on the current stream waits for it."""
+
+    def __init__(self, main, side) -> None:
+        self.main, self.side = main, side
+        self._inside = torch.cuda.stream(side)
+
+    def __enter__(self):
+        self.side.wait_stream(self.main)
+        self._inside.__enter__()
+        return self
+
+    def __exit__(self, *exc):
+        return self._inside.__exit__(*exc)
+
+    def join(self) -> None:
+        self.main.wait_stream(self.side)
+
+
 class CudaKernels:
     name = "cuda sm_100a"
 
@@ -154,6 +174,9 @@ class CudaKernels:
         self._chain_flags = torch.zeros(self._chain_slots, dtype=torch.int32, device=self.device)
         self._chain_scratch = torch.empty(self._chain_slots * 512, dtype=torch.float32, device=self.device)
         self._ticket_state = torch.zeros(8, dtype=torch.int32, device=self.device)
+        # Two mixers that read the same input run as two branches of a step's graph (HOLON_B200_BRANCHES=0: one after the other).
+        self.branches = os.environ.get("HOLON_B200_BRANCHES", "1") != "0"
+        self._side = None
         # One word of page-locked host memory that a kernel's bounded wait writes when it gives up (csrc/status.cu)
         word = ctypes.POINTER(ctypes.c_uint)()
         with torch.cuda.device(self.device):
@@ -272,6 +295,16 @@ class CudaKernels:
         """Whether a product of `m` rows over `k` columns of these bfloat16 tensors may be queued."""
         return bool(self.chain) and 0 < m <= self.SKINNY_ROWS and k % 8 == 0 \
             and all(t.dtype == torch.bfloat16 and t.data_ptr() % 16 == 0 for t in tensors)
+
+    def branch(self) -> Branch | None:
+        """A branch for work that may run beside what follows on the current stream, while a graph is captured: a decode step's
+        kernels leave most of the GPU idle, and two chains of them side by side take the time of the longer one. None otherwise (in an
+        eager step the host is what a second stream would wait for)."""
+        if not self.branches or self.chain or not torch.cuda.is_current_stream_capturing():
+            return None
+        if self._side is None:
+            self._side = torch.cuda.Stream(self.device)
+        return Branch(torch.cuda.current_stream(self.device), self._side)
 
     def _stream(self) -> int:
         """The handle of torch's current stream on the device (a few hundred kernels a step ask for it)."""

@@ -5,7 +5,7 @@ ffn(h). The residual sum is one kernel over all terms, in 32-bit, straight into 
 next is a parallel block too, the same kernel leaves that block's normed rows behind (`Residual.normed`), so a layer
 has one launch for its sum and the next layer's norm.
 
-`SideBySide`: a mixer made of two mixers that read the same input, result = left_scale · left + right_scale · right.
+`SideBySide`: a mixer made of two mixers that read the same input (in a step's graph two branches), result = left_scale · left + right_scale · right.
 At most one of the two may ask for a paged cache; their fixed-size states are kept under `left.` and `right.` names.
 Inside a `ParallelBlock` its two outputs go into the block's one sum as terms of their own. With `out_eps` each output first
 passes an RMS norm over its row with a weight of its own (stored `left.out`, `right.out`), and the two scales are equal; an
@@ -67,13 +67,21 @@ class SideBySide(Part):
         return NormedPair(a, self.out_gain[0].tensor, b, self.out_gain[1].tensor, self.out_eps, scale)
 
     def _run(self, x: torch.Tensor, step, cache) -> list:
-        out = []
-        for (side, part), scale in zip(self._sides(), self.scales):
+        def run(side, part):
             slots = {name[len(side) + 1:]: t for name, t in cache.slots.items() if name.startswith(side + ".")}
             paged = part.cache() is not None
             own = LayerCache(cache.kv if paged else None, cache.group if paged else None, cache.fills, slots)
-            out.append((part.forward(x, step, own), scale))
-        return out
+            return part.forward(x, step, own)
+
+        branch = getattr(self.ctx.kernels, "branch", None)           # a kernel table may run the two side by side
+        aside = branch() if branch is not None else None
+        if aside is None:
+            return [(run(side, part), scale) for (side, part), scale in zip(self._sides(), self.scales)]
+        with aside:
+            right = run("right", self.right)
+        left = run("left", self.left)
+        aside.join()
+        return [(left, self.scales[0]), (right, self.scales[1])]
 
     def forward(self, x: torch.Tensor, step, cache) -> torch.Tensor:
         if self.out_eps is not None:
