@@ -497,7 +497,7 @@ int hb_attention_maps_decode(void* out, const void* q, const void* kv, const int
                              const int32_t* row_slot, const int32_t* query_start, const int32_t* kv_len, int rows, int heads,
                              int kv_heads, int maps, int dim, int vdim, int pages, int page_size, float scale, float cap, int window,
                              int keep, float lam, float factor, float eps, const void* gate, long gate_ld, int splits, hb_stream stream);
-// bfloat16, rows row0 .. rows - 1 of any number of tokens on tcgen05 tensor cores: dim and vdim multiples of 16 up to 128, pages of a
+// bfloat16, rows row0 .. rows - 1 of any number of tokens on tcgen05 tensor cores: dim and vdim multiples of 8 up to 128, pages of a
 // multiple of 64 tokens. q_tiles: the sum over the rows of ceil(tokens / tile_q), tile_q 128 or, with one map, 256; tokens: all
 // tokens of the step. hb_attention_maps_status synchronises the device and returns (and clears) the kernel's status word.
 int hb_attention_maps_prefill(void* out, const void* q, const void* kv, const int32_t* block_table, int table_stride,

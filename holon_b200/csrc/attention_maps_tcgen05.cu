@@ -1,5 +1,6 @@
 // bfloat16 prompt attention with one or two maps a head on tcgen05 tensor cores (the rules: csrc/attention_maps.cu): key sizes
-// that are multiples of 16 up to 128, value sizes likewise, pages of a multiple of 64 tokens.
+// that are multiples of 8 up to 128, value sizes likewise, pages of a multiple of 64 tokens. (Queries are loaded through a map of
+// [token, head and map, channel], so that channels past a key's size are zeros whatever lies behind the key in its row.)
 //
 // A CTA carries two groups of 128 query rows that share its value tiles: with one map two groups of queries of one head, with two
 // maps the two maps of the same 128 queries (each with its own keys, in the same cache rows). It walks the 64-key tiles that some
@@ -50,7 +51,7 @@ __device__ __forceinline__ uint64_t mul2(uint64_t a, uint64_t b) {
     asm("mul.rn.f32x2 %0, %1, %2;\n" : "=l"(d) : "l"(a), "l"(b));
     return d;
 }
-__device__ __forceinline__ float am_sigmoid(float x) { return 1.f / (1.f + __expf(-x)); }
+__device__ __forceinline__ float am_sigmoid(float x) { return __fdividef(1.f, 1.f + __expf(-x)); }
 
 template <int MAPS, int CAP, int QB, int VB>
 __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid_constant__ CUtensorMap map_q,
@@ -123,7 +124,7 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
             mbar_expect_tx(q_full, AM_GROUPS * q_bytes);
             for (int g = 0; g < AM_GROUPS; ++g)                          // (a group without queries loads rows it never uses)
                 for (int c = 0; c < qb; ++c)
-                    tma_load_2d(q_s + g * q_bytes + c * AM_Q_BLOCK, &map_q, q_full, (MAPS == 1 ? h : h * 2 + g) * a.dim + c * 64,
+                    tma_load_3d(q_s + g * q_bytes + c * AM_Q_BLOCK, &map_q, q_full, c * 64, MAPS == 1 ? h : h * 2 + g,
                                 t0 + (MAPS == 1 ? g * AM_BM : 0));
             const int32_t* table = a.block_table + (size_t)a.row_slot[b] * a.table_stride;
             for (int j = 0; j < tiles; ++j) {
@@ -146,9 +147,8 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
         if (lane == 0) {
             // kind::f16, D float32, A and B bfloat16; N / 8 at bit 17, M / 16 at bit 24; bit 16: B is MN-major
             const uint32_t idesc_qk = (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)(AM_BN >> 3) << 17) | ((uint32_t)(AM_BM >> 4) << 24);
-            const uint32_t idesc_pv = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)(a.vdim >> 3) << 17) | ((uint32_t)(AM_BM >> 4) << 24);
+            const uint32_t idesc_pv = (1u << 4) | (1u << 7) | (1u << 10) | (1u << 16) | ((uint32_t)((a.vdim + 15) >> 4) << 18) | ((uint32_t)(AM_BM >> 4) << 24);
             if (warp == 1) {
-                const int ksteps = a.dim >> 4;
                 bool ok = mbar_wait(q_full, 0, 2);
                 for (int j = 0; j < tiles && ok; ++j) {
                     const int s = j % AM_STAGES;
@@ -164,7 +164,6 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
                         const uint32_t k_src = kv_s + s * stage_bytes + (MAPS == 2 ? g * qb * AM_KV_BLOCK : 0);
 #pragma unroll
                         for (int kk = 0; kk < QB * 4; ++kk) {
-                            if (kk >= ksteps) break;
                             const uint32_t blk = kk >> 2, within = (kk & 3) * 2;
                             tc_mma(s_t, tc_smem_desc(q_s + g * q_bytes + blk * AM_Q_BLOCK) + within,
                                    tc_smem_desc(k_src + blk * AM_KV_BLOCK) + within, idesc_qk, kk != 0);
@@ -323,7 +322,7 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
         const size_t token = (size_t)(t0 + (MAPS == 1 ? g * AM_BM : 0) + (r < qn ? r : 0));
         bf16* o_row = a.out + (token * a.heads + h) * a.vdim;
         const bf16* g_row = a.gate ? a.gate + token * a.gate_ld + (size_t)h * a.vdim : nullptr;
-        const bool g_vec = (((uintptr_t)a.gate | (uintptr_t)(a.gate_ld * 2)) & 15) == 0;      // (vdim is a multiple of 16)
+        const bool g_vec = (((uintptr_t)a.gate | (uintptr_t)(a.gate_ld * 2)) & 15) == 0;      // (vdim is a multiple of 8)
         uint4 gq[MINE][4];                                               // the row's gates, asked for ahead of the last products
 #pragma unroll
         for (int k = 0; k < MINE; ++k)
@@ -337,7 +336,7 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
         tc_fence_after();
         const float inv = ok && my_tiles > 0 && l > 0.f ? 1.f / l : 0.f;
         auto store = [&](const float (&v)[32], int c, const uint4 (&gz)[4]) {                  // a chunk of 32 channels of this thread's row, gated
-            const int live = min(32, a.vdim - c * 32);                   // 32 or 16
+            const int live = min(32, a.vdim - c * 32);                   // a multiple of 8
 #pragma unroll
             for (int i = 0; i < 32; i += 8) {
                 if (i >= live) break;
@@ -398,7 +397,7 @@ __global__ void __launch_bounds__(AM_THREADS, 1) maps_prompt_kernel(const __grid
                     tc_ld_wait();
 #pragma unroll
                     for (int i = 0; i < 32; ++i) {
-                        if (i < 16 || a.vdim - c * 32 > 16) {            // (a row's last chunk may be half a chunk)
+                        if (i < a.vdim - c * 32) {                       // (a row's last chunk may be a part of a chunk)
                             v[k][i] = (i1 > 0.f ? __uint_as_float(o1[i]) * i1 : 0.f) - (s_inv[1][r] > 0.f ? __uint_as_float(o2[i]) * i2 : 0.f);
                             ss = fmaf(v[k][i], v[k][i], ss);
                         }
@@ -457,8 +456,8 @@ extern "C" int hb_attention_maps_prefill(void* out, const void* q, const void* k
                                          float factor, float eps, const void* gate, long gate_ld, int tile_q, hb_stream stream) {
     if (rows <= row0 || q_tiles == 0) return 0;
     if (maps != 1 && maps != 2) HB_REFUSE("attention_maps_prefill: %d maps (1 or 2)", maps);
-    if (dim % 16 || dim < 16 || dim > 128 || vdim % 16 || vdim < 16 || vdim > 128)
-        HB_REFUSE("attention_maps_prefill: keys of %d and values of %d: multiples of 16 up to 128", dim, vdim);
+    if (dim % 8 || dim < 8 || dim > 128 || vdim % 8 || vdim < 8 || vdim > 128)
+        HB_REFUSE("attention_maps_prefill: keys of %d and values of %d: multiples of 8 up to 128", dim, vdim);
     if (tile_q != AM_BM && (maps == 2 || tile_q != AM_GROUPS * AM_BM)) HB_REFUSE("attention_maps_prefill: query tiles of %d", tile_q);
     if (page_size % AM_BN) HB_REFUSE("attention_maps_prefill: page size %d is no multiple of %d", page_size, AM_BN);
     if (kv_heads < 1 || heads % kv_heads) HB_REFUSE("attention_maps_prefill: %d heads, %d kv heads", heads, kv_heads);
@@ -468,9 +467,16 @@ extern "C" int hb_attention_maps_prefill(void* out, const void* q, const void* k
     const uint64_t kv_rows = (uint64_t)pages * kv_heads * page_size;
     if (kv_rows > 0x7fffffffull) HB_REFUSE("attention_maps_prefill: the cache has %llu rows, above 2^31", (unsigned long long)kv_rows);
     CUtensorMap map_q, map_kv;
-    int rc = encode_rows(&map_q, q, (uint64_t)heads * maps * dim, (uint64_t)tokens, AM_BM, "q");
-    if (rc) return rc;
-    rc = encode_rows(&map_kv, kv, (uint64_t)maps * dim + vdim, kv_rows, AM_BN, "the cache");
+    {
+        const cuuint64_t dims[3] = {(cuuint64_t)dim, (cuuint64_t)heads * maps, (cuuint64_t)tokens};
+        const cuuint64_t strides[2] = {(cuuint64_t)dim * 2, (cuuint64_t)heads * maps * dim * 2};
+        const cuuint32_t box[3] = {64, 1, AM_BM}, elem[3] = {1, 1, 1};
+        const CUresult r = cuTensorMapEncodeTiled(&map_q, CU_TENSOR_MAP_DATA_TYPE_BFLOAT16, 3, const_cast<void*>(q), dims, strides, box, elem,
+                                                  CU_TENSOR_MAP_INTERLEAVE_NONE, CU_TENSOR_MAP_SWIZZLE_128B,
+                                                  CU_TENSOR_MAP_L2_PROMOTION_L2_256B, CU_TENSOR_MAP_FLOAT_OOB_FILL_NONE);
+        if (r != CUDA_SUCCESS) HB_REFUSE("attention_maps_prefill: cuTensorMapEncodeTiled failed with %d for q", (int)r);
+    }
+    int rc = encode_rows(&map_kv, kv, (uint64_t)maps * dim + vdim, kv_rows, AM_BN, "the cache");
     if (rc) return rc;
     const int qb = (dim + 63) / 64, vb = (vdim + 63) / 64;
     const size_t smem = AM_GROUPS * (size_t)qb * AM_Q_BLOCK + AM_STAGES * (size_t)(maps * qb + vb) * AM_KV_BLOCK + 1024 + 256;

@@ -42,6 +42,17 @@ __device__ __forceinline__ float block_sum(float v, float* scratch) {
     __syncthreads();
     return scratch[32];
 }
+// Two sums at once (`scratch` holds 66 floats): x and y become the block's sums.
+__device__ __forceinline__ void block_sum2(float& x, float& y, float* scratch) {
+    const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = (blockDim.x + 31) >> 5;
+    x = warp_sum(x);
+    y = warp_sum(y);
+    __syncthreads();
+    if (lane == 0) { scratch[warp] = x; scratch[33 + warp] = y; }
+    __syncthreads();
+    x = warp_sum(lane < warps ? scratch[lane] : 0.f);             // (every warp adds the warps' sums up in the same order)
+    y = warp_sum(lane < warps ? scratch[33 + lane] : 0.f);
+}
 __device__ __forceinline__ float block_max(float v, float* scratch) {
     const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5, warps = (blockDim.x + 31) >> 5;
     v = warp_max(v);

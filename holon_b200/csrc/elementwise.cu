@@ -271,6 +271,17 @@ __global__ void embed_pair_kernel(float* __restrict__ out, const T* __restrict__
         extra = pair + (size_t)r * hidden;
     }
     float* o = out + (size_t)t * hidden;
+    if ((hidden & 3) == 0 && (((uintptr_t)out | (uintptr_t)table | (uintptr_t)pair) & 15) == 0) {      // four numbers a thread
+        for (int i = threadIdx.x * 4; i < hidden; i += blockDim.x * 4) {
+            float x[4] = {0.f, 0.f, 0.f, 0.f}, y[4] = {0.f, 0.f, 0.f, 0.f};
+            if (ok) Vec4<T>::load(row + i, x);
+            if (extra) Vec4<T>::load(extra + i, y);
+#pragma unroll
+            for (int e = 0; e < 4; ++e) x[e] = ok ? x[e] * scale + y[e] : 0.f;
+            Vec4<float>::store(o + i, x);
+        }
+        return;
+    }
     for (int i = threadIdx.x; i < hidden; i += blockDim.x)
         o[i] = ok ? to_f32(row[i]) * scale + (extra ? to_f32(extra[i]) : 0.f) : 0.f;
 }

@@ -13,7 +13,7 @@ __global__ void out_norm_rows_kernel(float* dst, const float* src, const T* __re
                                      const TW* __restrict__ a_weight, const TW* __restrict__ b_weight, float pair_eps, float scale,
                                      const void* __restrict__ weight, int weight_f32, float eps, float offset, T* cast, int dim) {
     extern __shared__ float on_rows[];
-    __shared__ float scratch[33];
+    __shared__ float scratch[66];
     const size_t at = (size_t)blockIdx.x * dim;
     auto w1 = [&](int d) -> float { return (weight_f32 ? ((const float*)weight)[d] : to_f32(((const bf16*)weight)[d])) + offset; };
     if constexpr (NV > 0) {
@@ -36,8 +36,8 @@ __global__ void out_norm_rows_kernel(float* dst, const float* src, const T* __re
             }
         }
         if (PAIR) {
-            const float fa = rsqrtf(block_sum(sa, scratch) / (float)dim + pair_eps) * scale;
-            const float fb = rsqrtf(block_sum(sb, scratch) / (float)dim + pair_eps) * scale;
+            block_sum2(sa, sb, scratch);
+            const float fa = rsqrtf(sa / (float)dim + pair_eps) * scale, fb = rsqrtf(sb / (float)dim + pair_eps) * scale;
             sa = 0.f;
 #pragma unroll
             for (int n = 0; n < NV; ++n) {
@@ -77,8 +77,8 @@ __global__ void out_norm_rows_kernel(float* dst, const float* src, const T* __re
             on_rows[d] = z;
         }
         if (PAIR) {
-            const float fa = rsqrtf(block_sum(sa, scratch) / (float)dim + pair_eps) * scale;
-            const float fb = rsqrtf(block_sum(sb, scratch) / (float)dim + pair_eps) * scale;
+            block_sum2(sa, sb, scratch);
+            const float fa = rsqrtf(sa / (float)dim + pair_eps) * scale, fb = rsqrtf(sb / (float)dim + pair_eps) * scale;
             sa = 0.f;
             for (int d = threadIdx.x; d < dim; d += blockDim.x) {
                 const float z = on_rows[d] * fa * to_f32(a_weight[d]) + to_f32(b[at + d]) * fb * to_f32(b_weight[d]);

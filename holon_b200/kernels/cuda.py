@@ -1474,8 +1474,8 @@ class CudaKernels:
         head = (self._p(out), self._p(q), self._p(kv))
         fast = q.dtype == torch.bfloat16 and self.attention_bf16 == "fast"
         ones, portions = rows.n_decode, rows.n_rows > rows.n_decode
-        tiles16 = fast and self.prefill_attention == "tcgen05" and dim % 16 == 0 and vd % 16 == 0 and max(dim, vd) <= 128 and page % 64 == 0
-        if not (fast and dim % 8 == 0 and vd % 8 == 0 and max(maps * dim, vd) <= 256) or (portions and not tiles16):
+        fast = fast and dim % 8 == 0 and vd % 8 == 0
+        if not (fast and max(maps * dim, vd) <= 256) or (portions and not (self.prefill_attention == "tcgen05" and max(dim, vd) <= 128 and page % 64 == 0)):
             return self._call("hb_attention_maps", *head, _code(q), *common, rows.n_rows, t, *sizes, *rules)
         if ones:
             self._call("hb_attention_maps_decode", *head, *common, ones, *sizes, *rules,

@@ -231,7 +231,7 @@ def paged(lens, page, kv, rowlen, window, keep, dtype, seed, before=None):
 
 MAPS = [(4, 2, 2, 32, 64, 64, 20.0), (20, 1, 1, 48, 80, 64, 0.0), (2, 2, 2, 64, 128, 64, 3.0), (4, 1, 1, 128, 128, 128, 0.0), (24, 2, 2, 16, 48, 16, 5.0),
         (3, 3, 1, 11, 7, 4, 0.0), (3, 1, 2, 9, 13, 16, 2.0), (8, 2, 2, 128, 96, 64, 30.0), (2, 1, 1, 112, 16, 64, 0.5), (2, 1, 2, 40, 24, 64, 0.0), (1, 1, 1, 256, 256, 64, 0.0),
-        (34, 1, 2, 8, 8, 64, 9.0)]
+        (34, 1, 2, 8, 8, 64, 9.0), (4, 2, 2, 72, 104, 64, 60.0), (6, 2, 1, 24, 40, 64, 70.0)]
 
 
 @pytest.mark.parametrize("dtype", DTYPES)
