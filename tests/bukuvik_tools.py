@@ -58,9 +58,9 @@ BA = _model(64, 211, 1e-5, 0.7, 2.5, [
 # as many kept tokens as the window has, a model that starts with a parallel layer and multiplies nothing.
 BB = _model(70, 157, 1e-6, 1.0, 1.0, [
     _par(_att(3, 3, 11, 7, 3.0), _ssm(3, 1, 5, 9, 1, 1), 37),
-    _diff(_att(3, 1, 9, 13, 2.0, 6, diff=0.2), None),
+    _diff(_att(3, 1, 9, 29, 2.0, 6, diff=0.2), None),
     _par(_att(2, 1, 18, 5, 3.0, 8, 8, _rot(50.0, 2)), _ssm(5, 5, 1, 3, 2, 5), 21),
-    _diff(_att(2, 2, 7, 6, 2.0, rot=_rot(40.0, 6), diff=0.0), 33)])
+    _diff(_att(2, 2, 7, 22, 2.0, rot=_rot(40.0, 6), diff=0.0), 33)])
 # C: sizes the tensor cores take: maps of 32 and 16, values of 64 and 48, windows that end inside and past a page of 64, kept tokens
 # up to and over a page, heads of which sixteen or more read one key/value head, larger states.
 BC = _model(128, 300, 1e-5, 0.5, 4.0, [
@@ -103,18 +103,19 @@ def tensor_table(config):
 
 
 def make_weights(config, seed: int):
-    """Random weights, rounded to bfloat16 (so that both sides read the same numbers). Products' weights are N(0, 1/in) over a
-    stream of unit size; with the configurations' score scales the scores spread over several units, so a wrong key, page or
-    window edge moves the logits. Norm weights, layer scales, the two sides' weights and skips differ from one another visibly,
-    λ is far from 0 and from `diff`, biases of the convolution and of the step sizes are of their inputs' size, rates spread so
-    that some heads forget within a few tokens and others keep what the first tokens wrote."""
+    """Random weights, rounded to bfloat16 (so that both sides read the same numbers). Products' weights are N(0, 1/in); with the
+    configurations' score scales the scores spread over several units, so a wrong key, page or window edge moves the logits. The
+    embedding's rows are small beside what the layers add, so that the next token is not simply the last one again. Norm weights,
+    layer scales, the two sides' weights and skips differ from one another visibly, λ is far from 0 and from `diff`, biases of the
+    convolution and of the step sizes are of their inputs' size, rates spread so that some heads forget within a few tokens and
+    others keep what the first tokens wrote."""
     g = torch.Generator().manual_seed(seed)
     out = {}
     for name, shape in tensor_table(config):
         x = torch.randn(shape, generator=g, dtype=torch.float32)
         tail = name.split(".", 1)[1] if name.startswith("l") else name
         if name == "embed":
-            x = x / float(config["embedding"]["scale"])
+            x = 0.3 * x / float(config["embedding"]["scale"])
         elif tail.endswith(".conv"):
             x = 0.6 * x
         elif tail.endswith(".conv.b"):
