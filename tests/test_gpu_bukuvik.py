@@ -103,7 +103,7 @@ def test_squared_relu_in_the_product(K, m, n, k, pair, monkeypatch):
 
 # ---------------------------------------------------------------- state space
 @pytest.mark.parametrize("dtype", DTYPES)
-@pytest.mark.parametrize("heads,groups,n,vdim,taps", [(6, 2, 48, 20, 3), (4, 4, 16, 8, 4), (3, 1, 7, 5, 1), (5, 5, 3, 2, 6), (8, 1, 128, 64, 4), (2, 1, 130, 33, 2)])
+@pytest.mark.parametrize("heads,groups,n,vdim,taps", [(6, 3, 40, 20, 3), (4, 4, 16, 8, 4), (3, 1, 7, 5, 1), (5, 5, 3, 2, 6), (8, 1, 128, 64, 4), (2, 1, 130, 33, 2)])
 def test_state_space_inputs_and_carried_rows(K, dtype, heads, groups, n, vdim, taps):
     """Portions and one-token rows of three requests, twice in a row (the second step reads what the first carried)."""
     inner, channels = heads * vdim, heads * vdim + 2 * groups * n
@@ -186,7 +186,7 @@ def turn_table(dims, positions=512, base=300.0, size=1.2):
 
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("norm", [None, "before", "after"])
-@pytest.mark.parametrize("heads,kv,maps,dim,vdim,rot", [(4, 2, 2, 48, 96, 12), (6, 3, 1, 64, 64, 32), (3, 1, 2, 11, 7, 4), (2, 2, 1, 17, 5, 16), (1, 1, 2, 8, 3, 0),
+@pytest.mark.parametrize("heads,kv,maps,dim,vdim,rot", [(6, 2, 2, 56, 72, 24), (6, 3, 1, 96, 64, 48), (3, 1, 2, 11, 7, 4), (2, 2, 1, 17, 5, 16), (1, 1, 2, 8, 3, 0),
                                                        (32, 8, 1, 128, 128, 128), (2, 1, 2, 200, 150, 100), (2, 1, 1, 512, 64, 2)])
 def test_queries_and_cache_rows(K, dtype, norm, heads, kv, maps, dim, vdim, rot):
     t, page = 9, 4
